@@ -81,6 +81,10 @@ SIGNATURES = {
     "alice_model_kv_write": (C.c_int32, [_vp, C.c_uint32, C.c_uint32, C.c_uint32, _vp, _vp]),
     "alice_model_kv_read": (C.c_int32, [_vp, C.c_uint32, C.c_uint32, C.c_uint32, _vp, _vp]),
     "alice_model_set_position": (C.c_int32, [_vp, C.c_uint32]),
+    "alice_model_forward_rows": (C.c_int32, [_vp, _vp, C.c_uint32, _vp, C.c_uint32, _vp]),
+    "alice_stack_create": (C.c_int32, [_vp, _vp, _vp, _vp, _vp, _pp]),
+    "alice_stack_trace": (C.c_int32, [_vp, C.c_int32]),
+    "alice_stack_read_trace": (C.c_int32, [_vp, _vp, C.c_size_t, C.POINTER(C.c_uint32), C.POINTER(C.c_uint32)]),
     "alice_matvec_preq_noalloc": (C.c_int32, [_vp, _vp, _vp, _vp]),
     "alice_matvec_host": (C.c_int32, [C.c_uint32, _vp, C.c_size_t, C.c_uint32, C.c_uint32, _vp, _vp]),
     "alice_dequantize_host": (C.c_int32, [C.c_uint32, _vp, C.c_size_t, _vp, C.c_size_t]),
@@ -99,6 +103,21 @@ class LayerWeights(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("q", "k", "v", "o", "gate", "up", "down", "attn_norm", "ffn_norm")]
 
 
+class StackLayer(C.Structure):
+    """alice_stack_layer"""
+    _fields_ = [(n, C.c_uint32) for n in ("mixer", "heads", "kv_heads", "dim", "vdim", "q_rank", "kv_rank", "rot_dim", "rot_dims", "conv_taps",
+                                          "decay_rank", "gate_rank", "ff")] + \
+               [("scale", C.c_float), ("rot_base", C.c_double)] + \
+               [(n, C.c_void_p) for n in ("in_", "uq", "uk", "uv", "a2", "g2", "o", "gu", "down", "norm", "ls1", "ls2", "gate_bias", "up_bias",
+                                          "down_bias", "q_norm", "kv_norm", "sink", "conv", "a_log", "dt_bias", "head_norm")]
+
+
+class StackConfig(C.Structure):
+    """alice_stack_config"""
+    _fields_ = [(n, C.c_uint32) for n in ("num_layers", "width", "vocab_size", "max_seq_len", "loop_start", "loop_stop", "loop_times", "exact")] + \
+               [("eps", C.c_float), ("embed_scale", C.c_float), ("loop_step", C.c_void_p)]
+
+
 class AliceError(RuntimeError):
     def __init__(self, code: int, msg: str):
         super().__init__(f"alice_cuda error {code}: {msg}")
@@ -106,22 +125,43 @@ class AliceError(RuntimeError):
 
 
 _lib = None
+_part = "all"
 
 
 def lib_path() -> str:
     return _build.LIB
 
 
+def prefer(part: str) -> None:
+    """Which part of the library the process needs ("all", or "stack" for layer-stack models only), before anything loads it."""
+    global _part
+    _part = part
+
+
+def _missing(name):
+    def call(*_):
+        raise AliceError(E_UNSUPPORTED, f"{name}: this process loaded the part of the library for layer-stack models only")
+    return call
+
+
 def load():
-    """Load (building first if the .so is absent or older than its sources)."""
+    """Load (building first if the .so is absent; the stack part also when it is older than its sources)."""
     global _lib
     if _lib is None:
         path = _build.LIB
-        if not os.path.exists(path) or os.environ.get("ALICE_REBUILD") == "1":
+        if _part == "stack" and _build.stale(path):
+            path = _build.build(part=_part)
+        elif not os.path.exists(path) or os.environ.get("ALICE_REBUILD") == "1":
             path = _build.build()
         lib = C.CDLL(path)
         for name, (res, args) in SIGNATURES.items():
-            fn = getattr(lib, name)  # AttributeError if the library lacks a declared symbol
+            try:
+                fn = getattr(lib, name)
+            except AttributeError:
+                if path != _build.LIB_STACK:
+                    raise   # the library lacks a declared symbol
+                setattr(lib, name, _missing(name))
+                continue
             fn.restype = res
             fn.argtypes = args
         _lib = lib

@@ -13,7 +13,11 @@ import sys
 HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 LIB = os.path.join(HERE, "libalice_cuda.so")
-SOURCES = ["abi.cu", "gemv_launch.cu", "q8k.cu", "dequant.cu", "ternarize.cu", "glue.cu", "model.cu", "tp.cu"]
+# What a layer-stack model needs, as a library of its own; the whole library is these and the quantized-matvec path.
+LIB_STACK = os.path.join(HERE, "libalice_stack.so")
+STACK_SOURCES = ["engine.cu", "tp.cu", "step.cu", "model_api.cu", "stack_model.cu", "stack_ops.cu", "dense_rows.cu", "dense_gemm.cu", "delta.cu",
+                 "latent.cu"]
+SOURCES = STACK_SOURCES + ["abi.cu", "gemv_launch.cu", "q8k.cu", "dequant.cu", "ternarize.cu", "glue.cu", "model.cu"]
 # never --use_fast_math: dequantization and the Q8_K quantizer must round like the reference
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC", "-Xcompiler", "-fno-strict-aliasing"]
@@ -26,20 +30,34 @@ def _nvcc() -> str:
     raise RuntimeError("nvcc not found")
 
 
-def _stale() -> bool:
-    if not os.path.exists(LIB):
+def stale(lib: str) -> bool:
+    if not os.path.exists(lib):
         return True
-    t = os.path.getmtime(LIB)
-    deps = [os.path.join(CSRC, f) for f in os.listdir(CSRC)] + [os.path.join(HERE, "..", "include", "alice_cuda.h")]
+    t = os.path.getmtime(lib)
+    deps = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if not f.endswith(".o")] + [os.path.join(HERE, "..", "include", "alice_cuda.h")]
     return any(os.path.getmtime(d) > t for d in deps)
 
 
-def build(force: bool = False, verbose: bool = False) -> str:
-    if not force and not _stale():
-        return LIB
+def _object_stale(obj: str, src: str) -> bool:
+    """Objects of unchanged sources are kept; any header change rebuilds them all."""
+    if not os.path.exists(obj):
+        return True
+    t = os.path.getmtime(obj)
+    deps = [src] + [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith(".cuh")] + [os.path.join(HERE, "..", "include", "alice_cuda.h")]
+    return any(os.path.getmtime(d) > t for d in deps)
+
+
+def build(force: bool = False, verbose: bool = False, part: str = "all") -> str:
+    """part "all": the complete library; "stack": only what layer-stack models need."""
+    lib, sources = (LIB_STACK, STACK_SOURCES) if part == "stack" else (LIB, SOURCES)
+    if not force and not stale(lib):
+        return lib
+
     def compile_one(src):
-        obj = os.path.join(CSRC, src.replace(".cu", ".o"))
-        cmd = [_nvcc(), *NVCC_FLAGS, "-c", os.path.join(CSRC, src), "-o", obj]
+        path, obj = os.path.join(CSRC, src), os.path.join(CSRC, src.replace(".cu", ".o"))
+        if not force and not _object_stale(obj, path):
+            return obj
+        cmd = [_nvcc(), *NVCC_FLAGS, "-c", path, "-o", obj]
         if verbose:
             cmd.insert(1, "-Xptxas")
             cmd.insert(2, "-v")
@@ -47,11 +65,11 @@ def build(force: bool = False, verbose: bool = False) -> str:
         return obj
 
     # the translation units are independent: compile them side by side
-    with ThreadPoolExecutor(max_workers=min(len(SOURCES), os.cpu_count() or 1)) as pool:
-        objs = list(pool.map(compile_one, SOURCES))
-    subprocess.check_call([_nvcc(), "-shared", "-o", LIB, *objs, "-lcudart", "-ldl"])
-    return LIB
+    with ThreadPoolExecutor(max_workers=min(len(sources), os.cpu_count() or 1)) as pool:
+        objs = list(pool.map(compile_one, sources))
+    subprocess.check_call([_nvcc(), "-shared", "-o", lib, *objs, "-lcudart", "-ldl"])
+    return lib
 
 
 if __name__ == "__main__":
-    print(build(force="--force" in sys.argv, verbose="-v" in sys.argv))
+    print(build(force="--force" in sys.argv, verbose="-v" in sys.argv, part="stack" if "--stack" in sys.argv else "all"))

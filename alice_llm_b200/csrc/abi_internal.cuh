@@ -56,3 +56,4 @@ int alice_cuda_fail(cudaError_t err, const char* what);
 alice::LaunchCfg alice_cfg_of(const alice_engine* e);
 void alice_engine_retain(alice_engine* e);
 void alice_engine_release(alice_engine* e);
+void alice_quiesce(alice_engine* e);

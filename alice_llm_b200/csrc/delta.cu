@@ -1,0 +1,235 @@
+// Delta rule with one decay per key channel. Per head, with a state S [dim][vdim] kept in f32:
+//   S <- g * S (rows);  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q.
+// A column of S never meets another one, so the recurrence runs column-parallel: eight lanes hold one column in registers
+// for as long as the tokens last. Both products of a token are taken from the decayed column in one pass,
+//   o = (gS)^T q + (k.q) u,   with k.q prepared per token,
+// which leaves one eight-lane reduction on the token-to-token path.
+#include "dense_dev.cuh"
+#include "mixers.cuh"
+
+namespace alice {
+namespace {
+
+// Convolution input of channel c, `back` tokens before token t (the state holds the tokens before the first one).
+__device__ __forceinline__ float conv_in(const DeltaArgs& a, int t, int back, uint32_t c) {
+    const int s = t - back;
+    if (s >= 0) return a.y[(size_t)s * a.ldy + c];
+    return a.conv_state[(size_t)((int)a.s.taps - 1 + s) * a.s.conv_cols + c];
+}
+__device__ __forceinline__ float conv_silu(const DeltaArgs& a, int t, uint32_t c) {
+    const int taps = (int)a.s.taps;
+    const float* w = a.conv_w + (size_t)c * taps;
+    float v = 0.0f;
+    for (int j = 0; j < taps; j++) v = fmaf(w[j], conv_in(a, t, taps - 1 - j, c), v);
+    return silu_ref(v);
+}
+
+// One warp per (token, key head) or (token, value head).
+__global__ void __launch_bounds__(256) delta_prepare_kernel(const __grid_constant__ DeltaArgs a, uint32_t tokens) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const DeltaShape& s = a.s;
+    const uint32_t lane = threadIdx.x & 31, per = s.kv_heads + s.heads;
+    const size_t task = (size_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (task >= (size_t)tokens * per) return;
+    const uint32_t t = (uint32_t)(task / per), i = (uint32_t)(task % per);
+    if (i < s.kv_heads) {
+        constexpr int N = DELTA_MAX_DIM / 32;
+        float q[N], k[N], sq = 0.0f, sk = 0.0f;
+#pragma unroll
+        for (int j = 0; j < N; j++) {
+            const uint32_t d = lane + 32 * j;
+            q[j] = k[j] = 0.0f;
+            if (d < s.dim) {
+                q[j] = conv_silu(a, (int)t, s.off_q + i * s.dim + d);
+                k[j] = conv_silu(a, (int)t, s.off_k + i * s.dim + d);
+            }
+            sq = fmaf(q[j], q[j], sq); sk = fmaf(k[j], k[j], sk);
+        }
+        sq = warp_sum(sq); sk = warp_sum(sk);
+        const float iq = __frcp_rn(__fsqrt_rn(sq + 1e-6f)) * __frcp_rn(__fsqrt_rn((float)s.dim)), ik = __frcp_rn(__fsqrt_rn(sk + 1e-6f));
+        float dot = 0.0f;
+        const size_t o = ((size_t)t * s.kv_heads + i) * s.dp;
+#pragma unroll
+        for (int j = 0; j < N; j++) {
+            const uint32_t d = lane + 32 * j;
+            q[j] *= iq; k[j] *= ik;
+            dot = fmaf(q[j], k[j], dot);
+            if (d < s.dp) { a.qn[o + d] = q[j]; a.kn[o + d] = k[j]; }
+        }
+        dot = warp_sum(dot);
+        if (lane == 0) a.kq[(size_t)t * s.kv_heads + i] = dot;
+    } else {
+        const uint32_t h = i - s.kv_heads;
+        const size_t o = ((size_t)t * s.heads + h) * s.vp;
+        for (uint32_t d = lane; d < s.vp; d += 32) a.v[o + d] = d < s.vdim ? conv_silu(a, (int)t, s.off_v + h * s.vdim + d) : 0.0f;
+        if (lane == 0) a.beta[(size_t)t * s.heads + h] = sigmoid_f(a.y[(size_t)t * a.ldy + s.off_b + h]);
+    }
+}
+
+// The last taps - 1 inputs of every channel (ascending, so an entry is read before it is overwritten).
+__global__ void __launch_bounds__(256) conv_tail_kernel(const __grid_constant__ DeltaArgs a, uint32_t tokens) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const uint32_t c = blockIdx.x * 256 + threadIdx.x, keep = a.s.taps - 1;
+    if (c >= a.s.conv_cols) return;
+    for (uint32_t j = 0; j < keep; j++) {
+        const uint32_t i = tokens + j;      // index into [state; new tokens]
+        a.conv_state[(size_t)j * a.s.conv_cols + c] =
+            i < keep ? a.conv_state[(size_t)i * a.s.conv_cols + c] : a.y[(size_t)(i - keep) * a.ldy + c];
+    }
+}
+
+constexpr int SCAN_COLS = 32, SCAN_CHUNK = 8;   // columns per CTA, tokens per staged chunk
+
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// E elements of a column per lane: element e of lane l is dim (e / 4) * 32 + l * 4 + e % 4.
+template <int E>
+struct ScanStage {
+    float k[SCAN_CHUNK][8 * E], q[SCAN_CHUNK][8 * E], g[SCAN_CHUNK][8 * E], v[SCAN_CHUNK][SCAN_COLS];
+    float beta[SCAN_CHUNK], kq[SCAN_CHUNK];
+};
+
+template <int E>
+__device__ __forceinline__ void scan_fetch(ScanStage<E>& st, const DeltaArgs& a, uint32_t t0, uint32_t n, uint32_t h, uint32_t kh, uint32_t c0) {
+    const DeltaShape& s = a.s;
+    constexpr uint32_t P = 8 * E / 4;
+    for (uint32_t i = threadIdx.x; i < n * P; i += 256) {
+        const uint32_t j = i / P, d = i % P * 4;
+        const size_t ko = ((size_t)(t0 + j) * s.kv_heads + kh) * s.dp + d;
+        cp_async16(&st.k[j][d], a.kn + ko);
+        cp_async16(&st.q[j][d], a.qn + ko);
+        cp_async16(&st.g[j][d], a.g + ((size_t)(t0 + j) * s.heads + h) * s.dp + d);
+    }
+    for (uint32_t i = threadIdx.x; i < n * (SCAN_COLS / 4); i += 256) {
+        const uint32_t j = i / (SCAN_COLS / 4), d = i % (SCAN_COLS / 4) * 4;
+        cp_async16(&st.v[j][d], a.v + ((size_t)(t0 + j) * s.heads + h) * s.vp + c0 + d);
+    }
+    if (threadIdx.x < n) {
+        st.beta[threadIdx.x] = a.beta[(size_t)(t0 + threadIdx.x) * s.heads + h];
+        st.kq[threadIdx.x] = a.kq[(size_t)(t0 + threadIdx.x) * s.kv_heads + kh];
+    }
+}
+
+template <int E>
+__global__ void __launch_bounds__(256) delta_scan_kernel(const __grid_constant__ DeltaArgs a, uint32_t tokens) {
+    extern __shared__ __align__(16) uint8_t smem[];
+    auto* stage = reinterpret_cast<ScanStage<E>*>(smem);   // two
+    __shared__ float os[SCAN_CHUNK][SCAN_COLS];
+    const DeltaShape& s = a.s;
+    const uint32_t h = blockIdx.y, kh = h / (s.heads / s.kv_heads), c0 = blockIdx.x * SCAN_COLS;
+    const uint32_t lane = threadIdx.x & 31, l = lane & 7, col = (threadIdx.x >> 5) * 4 + (lane >> 3);
+    float* sp = a.state + ((size_t)h * s.vp + c0 + col) * s.dp + l * 4;
+    pdl_launch_dependents();
+    pdl_wait();
+    float S[E];
+#pragma unroll
+    for (int e = 0; e < E; e += 4) {
+        const float4 f = *reinterpret_cast<const float4*>(sp + e * 8);
+        S[e] = f.x; S[e + 1] = f.y; S[e + 2] = f.z; S[e + 3] = f.w;
+    }
+    scan_fetch<E>(stage[0], a, 0, min(tokens, (uint32_t)SCAN_CHUNK), h, kh, c0);
+    cp_commit();
+    for (uint32_t t0 = 0, b = 0; t0 < tokens; t0 += SCAN_CHUNK, b ^= 1) {
+        const uint32_t n = min(tokens - t0, (uint32_t)SCAN_CHUNK);
+        if (t0 + SCAN_CHUNK < tokens) scan_fetch<E>(stage[b ^ 1], a, t0 + SCAN_CHUNK, min(tokens - t0 - SCAN_CHUNK, (uint32_t)SCAN_CHUNK), h, kh, c0);
+        cp_commit();
+        cp_wait<1>();
+        __syncthreads();
+        const ScanStage<E>& st = stage[b];
+        for (uint32_t j = 0; j < n; j++) {
+            float k[E], dk = 0.0f, dq = 0.0f, dk2 = 0.0f, dq2 = 0.0f;
+#pragma unroll
+            for (int e = 0; e < E; e += 4) {
+                const float4 kk = *reinterpret_cast<const float4*>(&st.k[j][e * 8 + l * 4]), qq = *reinterpret_cast<const float4*>(&st.q[j][e * 8 + l * 4]),
+                             gg = *reinterpret_cast<const float4*>(&st.g[j][e * 8 + l * 4]);
+                S[e] *= gg.x; S[e + 1] *= gg.y; S[e + 2] *= gg.z; S[e + 3] *= gg.w;
+                dk = fmaf(S[e], kk.x, dk); dk2 = fmaf(S[e + 1], kk.y, dk2); dk = fmaf(S[e + 2], kk.z, dk); dk2 = fmaf(S[e + 3], kk.w, dk2);
+                dq = fmaf(S[e], qq.x, dq); dq2 = fmaf(S[e + 1], qq.y, dq2); dq = fmaf(S[e + 2], qq.z, dq); dq2 = fmaf(S[e + 3], qq.w, dq2);
+                k[e] = kk.x; k[e + 1] = kk.y; k[e + 2] = kk.z; k[e + 3] = kk.w;
+            }
+            dk += dk2; dq += dq2;
+#pragma unroll
+            for (int o = 4; o > 0; o >>= 1) {
+                dk += __shfl_xor_sync(0xffffffffu, dk, o);
+                dq += __shfl_xor_sync(0xffffffffu, dq, o);
+            }
+            const float u = st.beta[j] * (st.v[j][col] - dk);
+#pragma unroll
+            for (int e = 0; e < E; e++) S[e] = fmaf(k[e], u, S[e]);
+            if (l == 0) os[j][col] = fmaf(st.kq[j], u, dq);
+        }
+        __syncthreads();
+        for (uint32_t i = threadIdx.x; i < n * SCAN_COLS; i += 256) {
+            const uint32_t j = i / SCAN_COLS, c = i % SCAN_COLS;
+            if (c0 + c < s.vdim) a.o[((size_t)(t0 + j) * s.heads + h) * s.vdim + c0 + c] = os[j][c];
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int e = 0; e < E; e += 4) *reinterpret_cast<float4*>(sp + e * 8) = make_float4(S[e], S[e + 1], S[e + 2], S[e + 3]);
+}
+
+// One warp per (token, head): root-mean-square norm over vdim, weight, gate.
+template <class OT>
+__global__ void __launch_bounds__(256) delta_out_kernel(const __grid_constant__ DeltaArgs a, uint32_t tokens) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const DeltaShape& s = a.s;
+    const uint32_t lane = threadIdx.x & 31;
+    const size_t task = (size_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (task >= (size_t)tokens * s.heads) return;
+    const uint32_t t = (uint32_t)(task / s.heads), h = (uint32_t)(task % s.heads);
+    const float* o = a.o + task * s.vdim;
+    const float* gate = a.gate + task * s.vdim;
+    float q = 0.0f;
+    for (uint32_t d = lane; d < s.vdim; d += 32) q = fmaf(o[d], o[d], q);
+    q = warp_sum(q);
+    const float inv = __frcp_rn(__fsqrt_rn(q / (float)s.vdim + a.eps));
+    OT* out = static_cast<OT*>(a.out) + (size_t)t * a.ldo + (size_t)h * s.vdim;
+    for (uint32_t d = lane; d < s.vdim; d += 32) put(out + d, o[d] * inv * a.norm_w[d] * gate[d]);
+    if (h + 1 == s.heads)   // padding up to the stride
+        for (uint32_t d = s.vdim + lane; d < a.ldo - h * s.vdim; d += 32) put(out + d, 0.0f);
+}
+
+template <int E>
+cudaError_t scan_e(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
+    static bool done[64] = {};
+    constexpr size_t smem = 2 * sizeof(ScanStage<E>);
+    const cudaError_t err = allow_smem(delta_scan_kernel<E>, smem, done);
+    if (err != cudaSuccess) return err;
+    return launch_pdl(delta_scan_kernel<E>, dim3(a.s.vp / SCAN_COLS, a.s.heads), dim3(256), smem, st, pdl, a, tokens);
+}
+
+}  // namespace
+
+cudaError_t launch_delta_prepare(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
+    const size_t tasks = (size_t)tokens * (a.s.kv_heads + a.s.heads);
+    cudaError_t err = launch_pdl(delta_prepare_kernel, dim3((unsigned)((tasks + 7) / 8)), dim3(256), 0, st, pdl, a, tokens);
+    if (err != cudaSuccess || a.s.taps <= 1) return err;
+    return launch_pdl(conv_tail_kernel, dim3((a.s.conv_cols + 255) / 256), dim3(256), 0, st, pdl, a, tokens);
+}
+
+cudaError_t launch_delta_scan(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
+    switch (a.s.dp) {
+        case 32: return scan_e<4>(a, tokens, st, pdl);
+        case 64: return scan_e<8>(a, tokens, st, pdl);
+        case 128: return scan_e<16>(a, tokens, st, pdl);
+        case 256: return scan_e<32>(a, tokens, st, pdl);
+        default: return cudaErrorInvalidValue;
+    }
+}
+
+cudaError_t launch_delta_out(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
+    const unsigned grid = (unsigned)(((size_t)tokens * a.s.heads + 7) / 8);
+    return a.out_bf16 ? launch_pdl(delta_out_kernel<bf16>, dim3(grid), dim3(256), 0, st, pdl, a, tokens)
+                      : launch_pdl(delta_out_kernel<float>, dim3(grid), dim3(256), 0, st, pdl, a, tokens);
+}
+
+}  // namespace alice

@@ -1,0 +1,187 @@
+// One token against dense bfloat16 rows. A warp owns R consecutive rows at a time; every lane streams 16-byte pieces of
+// each (R * unroll loads in flight per lane), the input sits in shared memory as f32. The rows a warp starts with are
+// requested into L2 before the wait for the producing kernel, so under programmatic dependent launch the weights travel
+// while the input is still being made.
+#include "dense_dev.cuh"
+
+namespace alice {
+namespace {
+
+constexpr int RT = 256, RW = RT / 32;
+
+template <int R>
+__device__ __forceinline__ void dot_rows(const bf16* const (&w)[R], const float* xs, uint32_t k, uint32_t lane, float (&acc)[R]) {
+#pragma unroll
+    for (int r = 0; r < R; r++) acc[r] = 0.0f;
+#pragma unroll 4
+    for (uint32_t c = lane * 8; c < k; c += 256) {
+        uint4 v[R];
+#pragma unroll
+        for (int r = 0; r < R; r++) v[r] = __ldg(reinterpret_cast<const uint4*>(w[r] + c));
+        const float4 x0 = *reinterpret_cast<const float4*>(xs + c), x1 = *reinterpret_cast<const float4*>(xs + c + 4);
+#pragma unroll
+        for (int r = 0; r < R; r++) {
+            const float2 a = bf2(v[r].x), b = bf2(v[r].y), d = bf2(v[r].z), e = bf2(v[r].w);
+            acc[r] = fmaf(a.x, x0.x, acc[r]); acc[r] = fmaf(a.y, x0.y, acc[r]);
+            acc[r] = fmaf(b.x, x0.z, acc[r]); acc[r] = fmaf(b.y, x0.w, acc[r]);
+            acc[r] = fmaf(d.x, x1.x, acc[r]); acc[r] = fmaf(d.y, x1.y, acc[r]);
+            acc[r] = fmaf(e.x, x1.z, acc[r]); acc[r] = fmaf(e.y, x1.w, acc[r]);
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < R; r++) acc[r] = warp_sum(acc[r]);
+}
+
+__device__ __forceinline__ void prefetch_row(const bf16* w, uint32_t k, uint32_t lane) {
+    for (uint32_t c = lane * 64; c < k; c += 32 * 64) prefetch_l2(w + c);
+}
+
+// order-preserving image of a float, as the output head's argmax packs it
+__device__ __forceinline__ unsigned long long argmax_pack(float v, uint32_t row) {
+    uint32_t u = __float_as_uint(v);
+    u = (u & 0x80000000u) ? ~u : (u | 0x80000000u);
+    return ((unsigned long long)u << 32) | (0xFFFFFFFFu - row);
+}
+
+// Item i of the work list: R rows of w0, or R / 2 gate rows with their up rows.
+template <int R>
+__device__ __forceinline__ void item_rows(const RowsIn& op, uint32_t item, uint32_t items0, const bf16* (&w)[R], uint32_t& first, bool& pair) {
+    pair = item >= items0;
+    if (!pair) {
+        first = item * R;
+#pragma unroll
+        for (int r = 0; r < R; r++) w[r] = op.w0.w + (size_t)min(first + r, op.w0.n - 1) * op.w0.k;
+    } else {
+        first = (item - items0) * (R / 2);
+#pragma unroll
+        for (int r = 0; r < R / 2; r++) {
+            const uint32_t c = first + r, row = (c / 64) * 128 + c % 64;
+            w[r] = op.gu.w + (size_t)row * op.gu.k;
+            w[R / 2 + r] = w[r] + (size_t)64 * op.gu.k;
+        }
+    }
+}
+
+template <int R>
+__global__ void __launch_bounds__(RT, 3) rows_in_kernel(const __grid_constant__ RowsIn op) {
+    extern __shared__ __align__(16) float xs[];
+    __shared__ float red[RW];
+    const uint32_t lane = threadIdx.x & 31, warps = gridDim.x * RW;
+    const uint32_t items0 = (op.w0.n + R - 1) / R, items = items0 + op.gu.n / R;
+    const uint32_t w_id = blockIdx.x + (threadIdx.x >> 5) * gridDim.x;
+    const uint32_t k = op.w0.k;
+    const bf16* w[R];
+    uint32_t first;
+    bool pair;
+    pdl_launch_dependents();
+    if (w_id < items) {
+        item_rows<R>(op, w_id, items0, w, first, pair);
+#pragma unroll
+        for (int r = 0; r < R; r++) prefetch_row(w[r], k, lane);
+    }
+    pdl_wait();
+    load_normed<RW>(xs, op.x, op.n_x, k, op.norm, op.norm_w, op.eps, red);
+    unsigned long long best = 0ull;
+    for (uint32_t item = w_id; item < items; item += warps) {
+        item_rows<R>(op, item, items0, w, first, pair);
+        float acc[R];
+        dot_rows<R>(w, xs, k, lane, acc);
+        if (!pair) {
+#pragma unroll
+            for (int r = 0; r < R; r++) {
+                if (first + r >= op.w0.n) break;
+                if (lane == (uint32_t)r) op.y0[first + r] = acc[r];
+                if (op.argmax_key) { const unsigned long long key = argmax_pack(acc[r], first + r); best = key > best ? key : best; }
+            }
+        } else {
+#pragma unroll
+            for (int r = 0; r < R / 2; r++)
+                if (lane == (uint32_t)r) op.y1[first + r] = silu_ref(acc[r] + op.gate_b[first + r]) * (acc[R / 2 + r] + op.up_b[first + r]);
+        }
+    }
+    if (op.argmax_key && lane == 0 && best) atomicMax(op.argmax_key, best);
+}
+
+template <int R>
+__global__ void __launch_bounds__(RT, 2) rows_out_kernel(const __grid_constant__ RowsOut op) {
+    extern __shared__ __align__(16) float xs[];
+    const uint32_t lane = threadIdx.x & 31, warps = gridDim.x * RW;
+    const uint32_t n = op.w1.n, k1 = op.w1.k, k2 = op.w2.n ? op.w2.k : 0;
+    const uint32_t items = (n + R - 1) / R, w_id = blockIdx.x + (threadIdx.x >> 5) * gridDim.x;
+    const bf16 *u[R], *d[R];
+    auto rows_of = [&](uint32_t item) {
+#pragma unroll
+        for (int r = 0; r < R; r++) {
+            const uint32_t row = min(item * R + r, n - 1);
+            u[r] = op.w1.w + (size_t)row * k1;
+            d[r] = k2 ? op.w2.w + (size_t)row * k2 : nullptr;
+        }
+    };
+    pdl_launch_dependents();
+    if (w_id < items) {
+        rows_of(w_id);
+#pragma unroll
+        for (int r = 0; r < R; r++) {
+            prefetch_row(u[r], k1, lane);
+            if (k2) prefetch_row(d[r], k2, lane);
+        }
+    }
+    pdl_wait();
+    for (uint32_t i = threadIdx.x * 4; i < k1; i += RT * 4) *reinterpret_cast<float4*>(xs + i) = __ldcg(reinterpret_cast<const float4*>(op.a + i));
+    for (uint32_t i = threadIdx.x * 4; i < k2; i += RT * 4) *reinterpret_cast<float4*>(xs + k1 + i) = __ldcg(reinterpret_cast<const float4*>(op.f + i));
+    __syncthreads();
+    for (uint32_t item = w_id; item < items; item += warps) {
+        rows_of(item);
+        float acc1[R], acc2[R];
+        dot_rows<R>(u, xs, k1, lane, acc1);
+#pragma unroll
+        for (int r = 0; r < R; r++) acc2[r] = 0.0f;
+        if (k2) dot_rows<R>(d, xs + k1, k2, lane, acc2);
+#pragma unroll
+        for (int r = 0; r < R; r++) {
+            const uint32_t row = item * R + r;
+            if (lane == (uint32_t)r && row < n) {
+                float v = op.s1[row] * acc1[r];
+                if (k2) v += op.s2[row] * (acc2[r] + op.b2[row]);
+                op.x[row] += v;
+            }
+        }
+    }
+}
+
+template <int R>
+cudaError_t rows_in_r(const RowsIn& op, int num_sms, cudaStream_t st, bool pdl) {
+    static bool done[64] = {};
+    cudaError_t err = allow_smem(rows_in_kernel<R>, 224 * 1024, done);
+    if (err != cudaSuccess) return err;
+    const uint32_t items = (op.w0.n + R - 1) / R + op.gu.n / R;
+    const uint32_t grid = std::min<uint32_t>((items + RW - 1) / RW, (uint32_t)num_sms * 3);
+    return launch_pdl(rows_in_kernel<R>, dim3(grid), dim3(RT), (size_t)op.w0.k * 4, st, pdl, op);
+}
+template <int R>
+cudaError_t rows_out_r(const RowsOut& op, int num_sms, cudaStream_t st, bool pdl) {
+    static bool done[64] = {};
+    cudaError_t err = allow_smem(rows_out_kernel<R>, 224 * 1024, done);
+    if (err != cudaSuccess) return err;
+    const uint32_t items = (op.w1.n + R - 1) / R;
+    const uint32_t grid = std::min<uint32_t>((items + RW - 1) / RW, (uint32_t)num_sms * 2);
+    return launch_pdl(rows_out_kernel<R>, dim3(grid), dim3(RT), (size_t)(op.w1.k + (op.w2.n ? op.w2.k : 0)) * 4, st, pdl, op);
+}
+
+}  // namespace
+
+cudaError_t launch_rows_in(const RowsIn& op, int num_sms, cudaStream_t st, bool pdl) {
+    if (!op.w0.n || op.w0.k % DENSE_PAD || (op.gu.n && (op.gu.k != op.w0.k || op.gu.n % 128)) || (size_t)op.w0.k * 4 > 220 * 1024) return cudaErrorInvalidValue;
+    // enough items to give every SM two dozen warps: fewer rows per warp for the small matrices
+    if (op.w0.n + op.gu.n >= (uint32_t)num_sms * 24 * 4) return rows_in_r<4>(op, num_sms, st, pdl);
+    return rows_in_r<2>(op, num_sms, st, pdl);
+}
+
+cudaError_t launch_rows_out(const RowsOut& op, int num_sms, cudaStream_t st, bool pdl) {
+    if (!op.w1.n || op.w1.k % DENSE_PAD || (op.w2.n && (op.w2.n != op.w1.n || op.w2.k % DENSE_PAD))) return cudaErrorInvalidValue;
+    if ((size_t)(op.w1.k + (op.w2.n ? op.w2.k : 0)) * 4 > 220 * 1024) return cudaErrorInvalidValue;
+    if (op.w1.n >= (uint32_t)num_sms * 16 * 2) return rows_out_r<2>(op, num_sms, st, pdl);
+    return rows_out_r<1>(op, num_sms, st, pdl);
+}
+
+}  // namespace alice

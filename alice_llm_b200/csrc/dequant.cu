@@ -79,6 +79,7 @@ __device__ float deq_elem(WeightFormat fmt, const uint8_t* row, uint32_t c, uint
             const uint32_t code = (row[c >> 2] >> ((c & 3) * 2)) & 3;
             return __fmul_rn(scales[r], code == 1 ? 1.0f : (code == 3 ? -1.0f : 0.0f));
         }
+        case WF_BF16: return __uint_as_float(((uint32_t)row[2 * c] | ((uint32_t)row[2 * c + 1] << 8)) << 16);
         default: return 0.0f;
     }
 }

@@ -14,27 +14,6 @@ namespace alice {
 
 bool format_uses_q8k(WeightFormat f) { return f == WF_Q4_K || f == WF_Q5_K || f == WF_Q6_K; }
 
-uint32_t ggml_block_bytes(WeightFormat f) {
-    switch (f) {
-        case WF_Q8_0: return 34; case WF_Q4_K: return 144; case WF_Q5_K: return 176;
-        case WF_Q6_K: return 210; case WF_Q1_0: return 18; case WF_Q2_0: return 34;
-        default: return 0;
-    }
-}
-uint32_t ggml_block_elems(WeightFormat f) {
-    switch (f) {
-        case WF_Q8_0: return 32;
-        case WF_Q4_K: case WF_Q5_K: case WF_Q6_K: return 256;
-        case WF_Q1_0: case WF_Q2_0: return 128;
-        default: return 0;
-    }
-}
-uint32_t ggml_row_bytes(WeightFormat f, uint32_t cols) {
-    const uint32_t e = ggml_block_elems(f);
-    if (e == 0 || cols == 0 || cols % e != 0) return 0;
-    return cols / e * ggml_block_bytes(f);
-}
-
 namespace {
 
 // Shared memory per CTA: two CTAs share an SM when a lane holds at most two activation positions

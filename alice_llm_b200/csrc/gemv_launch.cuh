@@ -11,6 +11,7 @@ namespace alice {
 // Storage formats of a device-resident weight matrix.
 enum WeightFormat : uint32_t {
     WF_Q8_0 = 8, WF_Q4_K = 12, WF_Q5_K = 13, WF_Q6_K = 14, WF_Q1_0 = 41, WF_Q2_0 = 42,  // GGML ids (src/gguf.rs:101-122)
+    WF_BF16 = 30,              // dense bfloat16 rows (csrc/dense.cuh)
     WF_TERNARY = 1000,         // interleaved bit planes, see FmtTernary
     WF_SPARSE_TERNARY = 1001,  // packed 2-bit codes, see FmtSparseTernary
 };

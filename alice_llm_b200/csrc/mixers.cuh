@@ -1,0 +1,98 @@
+// Token mixers of layer-stack models (csrc/delta.cu, csrc/latent.cu) and the small per-token kernels around them
+// (csrc/stack_ops.cu). Sizes are run-time values; positions come from device memory so that a captured step can be replayed.
+#pragma once
+#include "dense.cuh"
+
+namespace alice {
+
+// ---- stack_ops.cu -------------------------------------------------------------------------------
+// x[t] <- (set ? 0 : x[t]) + (emb ? emb[tokens[t]] * scale : 0) + (step ? step : 0), columns [0, n); [n, ld) untouched.
+struct EnterArgs {
+    const bf16* emb = nullptr;
+    const int* tokens = nullptr;
+    uint32_t vocab = 0, emb_ld = 0, n = 0, ld = 0;
+    float scale = 1.f;
+    const float* step = nullptr;
+    bool set = false;
+    float* x = nullptr;
+};
+cudaError_t launch_enter(const EnterArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
+
+constexpr uint32_t MAX_NORM_ROWS = 64;
+struct NormArgs {
+    const float* x = nullptr;
+    uint32_t ldx = 0, n = 0, k = 0;   // true and padded length; out rows are k apart, zero beyond n
+    const float* w = nullptr;
+    float eps = 0.f;
+    void* out = nullptr;
+    bool out_bf16 = false;
+    bool gather = false;              // read rows idx[i] instead of i (at most MAX_NORM_ROWS)
+    uint32_t idx[MAX_NORM_ROWS] = {};
+};
+cudaError_t launch_layer_norm(const NormArgs& a, uint32_t rows, cudaStream_t st, bool pdl);
+
+// ---- delta.cu: delta rule with one decay per key channel ----------------------------------------
+struct DeltaShape {
+    uint32_t heads, kv_heads, dim, vdim, taps;
+    uint32_t dp, vp;                  // dim and vdim padded (dp: 32, 64, 128 or 256; vp: multiple of 32)
+    uint32_t off_q, off_k, off_v, off_b, conv_cols;   // columns of the projection output; the convolution covers [0, conv_cols)
+};
+constexpr uint32_t DELTA_MAX_DIM = 256;
+inline uint32_t delta_pad_dim(uint32_t d) { return d <= 32 ? 32 : d <= 64 ? 64 : d <= 128 ? 128 : 256; }
+
+struct DeltaArgs {
+    DeltaShape s;
+    const float* y = nullptr;         // projections [t][ldy]: q | k | v | b | ...
+    uint32_t ldy = 0;
+    const float* conv_w = nullptr;    // [conv_cols][taps]
+    float* conv_state = nullptr;      // [taps - 1][conv_cols], oldest first
+    float* state = nullptr;           // [heads][vp][dp]
+    float *qn = nullptr, *kn = nullptr, *kq = nullptr, *v = nullptr, *beta = nullptr;   // prepared inputs of the recurrence
+    const float* g = nullptr;         // decays [t][heads][dp]
+    float* o = nullptr;               // [t][heads][vdim]
+    const float* gate = nullptr;      // sigmoid already applied, [t][heads * vdim]
+    const float* norm_w = nullptr;
+    float eps = 0.f;
+    void* out = nullptr;              // [t][ldo]
+    uint32_t ldo = 0;
+    bool out_bf16 = false;
+};
+// short convolution + silu + unit vectors + step sizes; then the convolution's tail moves into its state
+cudaError_t launch_delta_prepare(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
+cudaError_t launch_delta_scan(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
+cudaError_t launch_delta_out(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
+
+// ---- latent.cu: attention over a cached latent ---------------------------------------------------
+struct LatentShape {
+    uint32_t heads, dim, rot, rot_dims, vdim, q_rank, kv_rank;
+    uint32_t qp, cp, rp;              // padded q_rank, kv_rank (64s) and rot (16s): a cache row is cp + rp wide
+    uint32_t off_q, off_kv, off_g;    // columns of the projection output
+    float scale;
+};
+constexpr uint32_t LATENT_MAX_RANK = 512;
+
+struct LatentArgs {
+    LatentShape s;
+    const float* y = nullptr;         // projections [t][ldy]: query latent | key latent, rotated key | gate
+    uint32_t ldy = 0;
+    const float *q_norm = nullptr, *kv_norm = nullptr, *sink = nullptr, *freq = nullptr;
+    float eps = 0.f;
+    const bf16 *uk = nullptr, *uv = nullptr;   // [heads * dim][cp], [heads * vdim][cp]
+    const int* pos = nullptr;
+    void* cache = nullptr;            // [max_seq][cp + rp]
+    bool cache_bf16 = false;
+    void* cqn = nullptr;              // normalised query latent [t][qp]
+    bool act_bf16 = false;            // type of cqn and out
+    const float* q = nullptr;         // [t][heads * (dim + rot)]
+    float* ql = nullptr;              // [t][heads][cp + rp]: queries taken into the latent space, rotated part
+    float* part = nullptr;            // [t][splits][heads][cp + 2]
+    uint32_t splits = 1;
+    void* out = nullptr;              // [t][ldo]
+    uint32_t ldo = 0;
+};
+cudaError_t launch_latent_norm(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
+cudaError_t launch_latent_absorb(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
+cudaError_t launch_latent_attn(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
+cudaError_t launch_latent_out(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
+
+}  // namespace alice

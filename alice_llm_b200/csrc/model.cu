@@ -11,12 +11,14 @@
 #include "abi_internal.cuh"
 #include "attn_body.cuh"
 #include "glue.cuh"
+#include "model_base.cuh"
 #include "tp.cuh"
 
 using namespace alice;
 
-struct alice_model {
-    alice_engine* e = nullptr;
+namespace {
+
+struct LlamaModel final : alice_model {
     alice_model_config cfg{};
     struct Layer {
         WeightDesc q, k, v, o, gate, up, down;
@@ -27,7 +29,7 @@ struct alice_model {
     WeightDesc emb{}, out{};
     float* out_norm = nullptr;
     // activations, each for up to MAX_BATCH tokens: [k][dim]
-    float *hidden = nullptr, *qkv = nullptr, *attn_out = nullptr, *ffn_h = nullptr, *logits = nullptr;
+    float *hidden = nullptr, *qkv = nullptr, *attn_out = nullptr, *ffn_h = nullptr;   // and the base's logits
     float *kcache = nullptr, *vcache = nullptr;  // [layer][max_seq][kv_dim]
     float* attn_part = nullptr;
     float* rope_freq = nullptr;  // 1 / theta^(2j / head_dim), j < 64, computed on the host (libm powf, as the CPU path)
@@ -54,40 +56,23 @@ struct alice_model {
     uint32_t npeers = 0;
     uint32_t peer_rank[7] = {};
     uint8_t* peer_base[7] = {};
-    // device-side state: position, current tokens, tokens chosen per position
-    int *d_pos = nullptr, *d_token = nullptr, *d_trace = nullptr;
-    uint32_t pos = 0;  // host mirror of *d_pos
-    cudaGraphExec_t graph_greedy = nullptr;
-    bool graph_tried = false;
-    std::vector<void*> owned;
+    ~LlamaModel() override {
+        for (uint32_t p = 0; p < npeers; p++) cudaIpcCloseMemHandle(peer_base[p]);
+    }
+    uint32_t max_tokens() const override { return MAX_BATCH; }
+    int enqueue_step(uint32_t batch, bool greedy_feed) override;
+    int enqueue_rows(uint32_t n, const uint32_t* rows, uint32_t nrows, float* host_logits) override;
+    int clear_state() override;
 };
 
-namespace {
-
-#define MCU(call)                                                       \
-    do {                                                                \
-        cudaError_t err__ = (call);                                     \
-        if (err__ != cudaSuccess) return alice_cuda_fail(err__, #call); \
-    } while (0)
-
-template <class T>
-int dev_alloc(alice_model* m, T** p, size_t n) {
-    void* q = nullptr;
-    cudaError_t err = cudaMalloc(&q, std::max<size_t>(n, 1) * sizeof(T));
-    if (err != cudaSuccess) return alice_cuda_fail(err, "alice_model_create: cudaMalloc");
-    m->owned.push_back(q);
-    *p = static_cast<T*>(q);
-    return ALICE_OK;
-}
-
-int upload_norm(alice_model* m, float** dst, const float* host, size_t n) {
+int upload_norm(LlamaModel* m, float** dst, const float* host, size_t n) {
     int rc = dev_alloc(m, dst, n);
     if (rc) return rc;
     MCU(cudaMemcpy(*dst, host, n * sizeof(float), cudaMemcpyHostToDevice));
     return ALICE_OK;
 }
 
-int gemv(alice_model* m, GemvOp& op, const char* what) {
+int gemv(LlamaModel* m, GemvOp& op, const char* what) {
     op.wait_limit = m->e->wait_limit;
     op.prep = m->prep; op.prep_bytes = m->prep_bytes;
     const int rc = launch_stream_gemv_op(op, alice_cfg_of(m->e));
@@ -138,7 +123,8 @@ void fill_dst(PublishDst& d, const Need& nd, uint8_t* q8_base, float* xn, uint32
 // rows into every peer's copy, with one flag per vector that a one-CTA kernel behind it raises on the peers and waits for
 // here before it prepares the vector for the next op. Attention runs on the rank's own KV heads (its q, k, v rows), so
 // only its output needs exchanging (it is the input of the output projection).
-int enqueue_step(alice_model* m, uint32_t batch, bool greedy_feed) {
+int LlamaModel::enqueue_step(uint32_t batch, bool greedy_feed) {
+    LlamaModel* const m = this;
     const alice_model_config& c = m->cfg;
     cudaStream_t st = m->e->stream;
     const bool pdl = m->e->pdl;
@@ -219,7 +205,7 @@ int enqueue_step(alice_model* m, uint32_t batch, bool greedy_feed) {
     // embedding + rotation table + hidden prepared for layer 0
     Need nd0;
     {
-        const alice_model::Layer& L = m->layers[0];
+        const LlamaModel::Layer& L = m->layers[0];
         need_of(nd0, L.q, true); need_of(nd0, L.k, true); need_of(nd0, L.v, true);
     }
     EmbedArgs ea{};
@@ -234,7 +220,7 @@ int enqueue_step(alice_model* m, uint32_t batch, bool greedy_feed) {
     MCU(launch_embed_q8_0(ea, st, pdl));
 
     for (uint32_t l = 0; l < L_n; l++) {
-        const alice_model::Layer& L = m->layers[l];
+        const LlamaModel::Layer& L = m->layers[l];
         float* kc = m->kcache + (size_t)l * c.max_seq_len * lkv;
         float* vc = m->vcache + (size_t)l * c.max_seq_len * lkv;
         const uint32_t qkv_stride = lq + 2 * lkv;
@@ -319,7 +305,7 @@ int enqueue_step(alice_model* m, uint32_t batch, bool greedy_feed) {
             Need nd;
             const float* norm_w;
             if (l + 1 < L_n) {
-                const alice_model::Layer& N = m->layers[l + 1];
+                const LlamaModel::Layer& N = m->layers[l + 1];
                 need_of(nd, N.q, true); need_of(nd, N.k, true); need_of(nd, N.v, true);
                 norm_w = N.attn_norm;
             } else {
@@ -358,10 +344,20 @@ int enqueue_step(alice_model* m, uint32_t batch, bool greedy_feed) {
     return ALICE_OK;
 }
 
-int check_room(const alice_model* m, uint32_t steps, const char* who) {
-    if ((uint64_t)m->pos + steps > m->cfg.max_seq_len)
-        return alice_fail(ALICE_E_SHAPE, "%s: position %u + %u steps exceeds max_seq_len %u", who, m->pos, steps,
-                          m->cfg.max_seq_len);
+// Every row of the batch has its logits (the head runs over the whole batch): the wanted ones are copied out.
+int LlamaModel::enqueue_rows(uint32_t n, const uint32_t* rows, uint32_t nrows, float* host_logits) {
+    const int rc = enqueue_step(n, false);
+    if (rc) return rc;
+    for (uint32_t i = 0; i < nrows; i++)
+        MCU(cudaMemcpyAsync(host_logits + (size_t)i * cfg.vocab_size, logits + (size_t)rows[i] * cfg.vocab_size, (size_t)cfg.vocab_size * 4,
+                            cudaMemcpyDeviceToHost, e->stream));
+    return ALICE_OK;
+}
+
+int LlamaModel::clear_state() {
+    const size_t kv_bytes = (size_t)cfg.num_layers * cfg.max_seq_len * lkv * 4;
+    MCU(cudaMemsetAsync(kcache, 0, kv_bytes, e->stream));
+    MCU(cudaMemsetAsync(vcache, 0, kv_bytes, e->stream));
     return ALICE_OK;
 }
 
@@ -396,8 +392,8 @@ int32_t alice_model_create(alice_engine* e, const alice_model_config* cfg, const
         return alice_fail(ALICE_E_SHAPE, "%s: embedding must be Q8_0 [vocab x hidden]", who);
     if (!same_shape(output->d, lV, c.hidden_dim)) return alice_fail(ALICE_E_SHAPE, "%s: output head shape", who);
     MCU(cudaSetDevice(e->device));
-    auto* m = new alice_model();
-    m->e = e; m->cfg = c; m->emb = embedding->d; m->out = output->d;
+    auto* m = new LlamaModel();
+    m->e = e; m->cfg = c; m->vocab = c.vocab_size; m->max_seq = c.max_seq_len; m->emb = embedding->d; m->out = output->d;
     alice_engine_retain(e);
     m->tp_n = n; m->tp_r = e->tp_rank; m->lq = lq; m->lkv = lkv; m->lH = lH; m->lF = lF; m->lV = lV;
     int rc = ALICE_OK;
@@ -414,7 +410,7 @@ int32_t alice_model_create(alice_engine* e, const alice_model_config* cfg, const
             rc = alice_fail(ALICE_E_SHAPE, "%s: layer %u weight shapes do not match the config (rows are this rank's 1/%u share)", who, l, n);
             break;
         }
-        alice_model::Layer L;
+        LlamaModel::Layer L;
         L.q = s.q->d; L.k = s.k->d; L.v = s.v->d; L.o = s.o->d; L.gate = s.gate->d; L.up = s.up->d; L.down = s.down->d;
         rc = upload_norm(m, &L.attn_norm, s.attn_norm, c.hidden_dim);
         if (!rc) rc = upload_norm(m, &L.ffn_norm, s.ffn_norm, c.hidden_dim);
@@ -482,118 +478,10 @@ int32_t alice_model_create(alice_engine* e, const alice_model_config* cfg, const
     return ALICE_OK;
 }
 
-int32_t alice_model_destroy(alice_model* m) {
-    if (!m) return ALICE_OK;
-    cudaSetDevice(m->e->device);
-    if (!m->e->dead) cudaStreamSynchronize(m->e->stream);
-    if (m->graph_greedy) cudaGraphExecDestroy(m->graph_greedy);
-    for (uint32_t p = 0; p < m->npeers; p++) cudaIpcCloseMemHandle(m->peer_base[p]);
-    for (void* p : m->owned) cudaFree(p);
-    alice_engine_release(m->e);
-    delete m;
-    return ALICE_OK;
-}
-
-static int set_tokens(alice_model* m, const uint32_t* tokens, uint32_t n) {
-    int t[MAX_BATCH];
-    for (uint32_t k = 0; k < n; k++) {
-        if (tokens[k] >= m->cfg.vocab_size) return alice_fail(ALICE_E_INVALID, "alice_model: token %u >= vocab %u", tokens[k], m->cfg.vocab_size);
-        t[k] = (int)tokens[k];
-    }
-    MCU(cudaMemcpyAsync(m->d_token, t, 4 * n, cudaMemcpyHostToDevice, m->e->stream));
-    MCU(cudaStreamSynchronize(m->e->stream));  // `t` lives on this stack frame
-    return ALICE_OK;
-}
-static int set_token(alice_model* m, uint32_t token) { return set_tokens(m, &token, 1); }
-
-int32_t alice_model_forward(alice_model* m, uint32_t token) {
-    if (!m) return alice_fail(ALICE_E_INVALID, "alice_model_forward: null model");
-    MCU(cudaSetDevice(m->e->device));
-    int rc = check_room(m, 1, "alice_model_forward");
-    if (!rc) rc = set_token(m, token);
-    if (!rc) rc = enqueue_step(m, 1, false);
-    if (!rc) m->pos += 1;
-    return rc;
-}
-
-int32_t alice_model_forward_batch(alice_model* m, const uint32_t* tokens, uint32_t n) {
-    const char* who = "alice_model_forward_batch";
-    if (!m || !tokens) return alice_fail(ALICE_E_INVALID, "%s: null argument", who);
-    if (n == 0 || n > (uint32_t)MAX_BATCH) return alice_fail(ALICE_E_SHAPE, "%s: %u tokens outside 1..%d", who, n, MAX_BATCH);
-    MCU(cudaSetDevice(m->e->device));
-    int rc = check_room(m, n, who);
-    if (!rc) rc = set_tokens(m, tokens, n);
-    if (!rc) rc = enqueue_step(m, n, false);
-    if (!rc) m->pos += n;
-    return rc;
-}
-
-int32_t alice_model_forward_batch_read(alice_model* m, const uint32_t* tokens, uint32_t n, float* logits) {
-    if (!logits) return alice_fail(ALICE_E_INVALID, "alice_model_forward_batch_read: null argument");
-    int rc = alice_model_forward_batch(m, tokens, n);
-    if (rc) return rc;
-    MCU(cudaMemcpyAsync(logits, m->logits, (size_t)n * m->cfg.vocab_size * 4, cudaMemcpyDeviceToHost, m->e->stream));
-    MCU(cudaStreamSynchronize(m->e->stream));
-    return alice_sync(m->e);
-}
-
-int32_t alice_model_read_logits(alice_model* m, float* logits) {
-    if (!m || !logits) return alice_fail(ALICE_E_INVALID, "alice_model_read_logits: null argument");
-    MCU(cudaMemcpyAsync(logits, m->logits, (size_t)m->cfg.vocab_size * 4, cudaMemcpyDeviceToHost, m->e->stream));
-    MCU(cudaStreamSynchronize(m->e->stream));
-    return alice_sync(m->e);
-}
-
-int32_t alice_model_forward_read(alice_model* m, uint32_t token, float* logits) {
-    int rc = alice_model_forward(m, token);
-    if (rc) return rc;
-    return alice_model_read_logits(m, logits);
-}
-
-int32_t alice_model_decode_greedy(alice_model* m, uint32_t first_token, uint32_t n, uint32_t* out_tokens) {
-    const char* who = "alice_model_decode_greedy";
-    if (!m || (!out_tokens && n)) return alice_fail(ALICE_E_INVALID, "%s: null argument", who);
-    if (n == 0) return ALICE_OK;
-    MCU(cudaSetDevice(m->e->device));
-    int rc = check_room(m, n, who);
-    if (!rc) rc = set_token(m, first_token);
-    if (rc) return rc;
-    cudaStream_t st = m->e->stream;
-    const uint32_t pos0 = m->pos;
-    if (!m->graph_tried) {
-        // Capture one step (every kernel reads position and token from device memory) and replay it.
-        m->graph_tried = true;
-        rc = enqueue_step(m, 1, true);   // eager first step: also sets per-kernel attributes outside capture
-        if (rc) return rc;
-        m->pos += 1;
-        cudaGraph_t g = nullptr;
-        if (cudaStreamBeginCapture(st, cudaStreamCaptureModeThreadLocal) == cudaSuccess) {
-            const int crc = enqueue_step(m, 1, true);
-            cudaError_t err = cudaStreamEndCapture(st, &g);
-            if (crc == ALICE_OK && err == cudaSuccess && g) {
-                if (cudaGraphInstantiate(&m->graph_greedy, g, 0) != cudaSuccess) m->graph_greedy = nullptr;
-            }
-            if (g) cudaGraphDestroy(g);
-            cudaGetLastError();  // a failed capture only means the steps are launched one by one
-        }
-    }
-    while (m->pos < pos0 + n) {
-        if (m->graph_greedy) {
-            MCU(cudaGraphLaunch(m->graph_greedy, st));
-        } else {
-            rc = enqueue_step(m, 1, true);
-            if (rc) return rc;
-        }
-        m->pos += 1;
-    }
-    static_assert(sizeof(uint32_t) == sizeof(int), "token trace is copied as 32-bit words");
-    MCU(cudaMemcpyAsync(out_tokens, m->d_trace + pos0, (size_t)n * 4, cudaMemcpyDeviceToHost, st));
-    MCU(cudaStreamSynchronize(st));
-    return alice_sync(m->e);
-}
-
-int32_t alice_model_tp_export(alice_model* m, void* out, size_t nbytes) {
-    if (!m || !out) return alice_fail(ALICE_E_INVALID, "alice_model_tp_export: null argument");
+int32_t alice_model_tp_export(alice_model* base, void* out, size_t nbytes) {
+    if (!base || !out) return alice_fail(ALICE_E_INVALID, "alice_model_tp_export: null argument");
+    auto* m = dynamic_cast<LlamaModel*>(base);
+    if (!m) return alice_fail(ALICE_E_UNSUPPORTED, "alice_model_tp_export: this model runs on one GPU");
     if (nbytes < sizeof(cudaIpcMemHandle_t)) return alice_fail(ALICE_E_INVALID, "alice_model_tp_export: need %zu bytes", sizeof(cudaIpcMemHandle_t));
     MCU(cudaSetDevice(m->e->device));
     cudaIpcMemHandle_t h;
@@ -603,8 +491,10 @@ int32_t alice_model_tp_export(alice_model* m, void* out, size_t nbytes) {
     return ALICE_OK;
 }
 
-int32_t alice_model_tp_connect(alice_model* m, const void* handles, size_t bytes_per_handle) {
-    if (!m || !handles) return alice_fail(ALICE_E_INVALID, "alice_model_tp_connect: null argument");
+int32_t alice_model_tp_connect(alice_model* base, const void* handles, size_t bytes_per_handle) {
+    if (!base || !handles) return alice_fail(ALICE_E_INVALID, "alice_model_tp_connect: null argument");
+    auto* m = dynamic_cast<LlamaModel*>(base);
+    if (!m) return alice_fail(ALICE_E_UNSUPPORTED, "alice_model_tp_connect: this model runs on one GPU");
     if (bytes_per_handle < sizeof(cudaIpcMemHandle_t)) return alice_fail(ALICE_E_INVALID, "alice_model_tp_connect: handles of %zu bytes, need %zu", bytes_per_handle, sizeof(cudaIpcMemHandle_t));
     if (m->peer_mode) return alice_fail(ALICE_E_INVALID, "alice_model_tp_connect: already connected");
     if (m->tp_n <= 1) return ALICE_OK;
@@ -632,46 +522,10 @@ int32_t alice_model_tp_connect(alice_model* m, const void* handles, size_t bytes
     return ALICE_OK;
 }
 
-int32_t alice_model_position(const alice_model* m, uint32_t* pos) {
-    if (!m || !pos) return alice_fail(ALICE_E_INVALID, "alice_model_position: null argument");
-    *pos = m->pos;
-    return ALICE_OK;
-}
-
-int32_t alice_model_vocab_size(const alice_model* m, uint32_t* vocab) {
-    if (!m || !vocab) return alice_fail(ALICE_E_INVALID, "alice_model_vocab_size: null argument");
-    *vocab = m->cfg.vocab_size;
-    return ALICE_OK;
-}
-
-int32_t alice_model_set_position(alice_model* m, uint32_t pos) {
-    if (!m) return alice_fail(ALICE_E_INVALID, "alice_model_set_position: null model");
-    if (pos > m->cfg.max_seq_len) return alice_fail(ALICE_E_SHAPE, "alice_model_set_position: %u > max_seq_len %u", pos, m->cfg.max_seq_len);
-    const int p = (int)pos;
-    MCU(cudaSetDevice(m->e->device));
-    MCU(cudaMemcpyAsync(m->d_pos, &p, 4, cudaMemcpyHostToDevice, m->e->stream));
-    MCU(cudaStreamSynchronize(m->e->stream));
-    m->pos = pos;
-    return ALICE_OK;
-}
-
-int32_t alice_model_rollback_to(alice_model* m, uint32_t pos) {
-    if (!m) return alice_fail(ALICE_E_INVALID, "alice_model_rollback_to: null model");
-    if (pos > m->pos) return ALICE_OK;  // only ever lowers the counter (src/gpu.rs:5645-5652)
-    return alice_model_set_position(m, pos);
-}
-
-int32_t alice_model_reset(alice_model* m) {
-    if (!m) return alice_fail(ALICE_E_INVALID, "alice_model_reset: null model");
-    const size_t kv_bytes = (size_t)m->cfg.num_layers * m->cfg.max_seq_len * m->lkv * 4;
-    MCU(cudaSetDevice(m->e->device));
-    MCU(cudaMemsetAsync(m->kcache, 0, kv_bytes, m->e->stream));
-    MCU(cudaMemsetAsync(m->vcache, 0, kv_bytes, m->e->stream));
-    return alice_model_set_position(m, 0);
-}
-
-static int kv_copy(alice_model* m, uint32_t layer, uint32_t pos0, uint32_t npos, float* k, float* v, bool to_device) {
-    if (!m || !k || !v) return alice_fail(ALICE_E_INVALID, "alice_model_kv: null argument");
+static int kv_copy(alice_model* base, uint32_t layer, uint32_t pos0, uint32_t npos, float* k, float* v, bool to_device) {
+    if (!base || !k || !v) return alice_fail(ALICE_E_INVALID, "alice_model_kv: null argument");
+    auto* m = dynamic_cast<LlamaModel*>(base);
+    if (!m) return alice_fail(ALICE_E_UNSUPPORTED, "alice_model_kv: this model keeps no key / value rows");
     const alice_model_config& c = m->cfg;
     if (layer >= c.num_layers || (uint64_t)pos0 + npos > c.max_seq_len) return alice_fail(ALICE_E_SHAPE, "alice_model_kv: layer / position out of range");
     const size_t kv_dim = m->lkv;   // this rank's KV heads

@@ -25,6 +25,7 @@ class GpuQuantType(Enum):
     Q8_0 = 8
     Q1_0 = 41
     Q2_0 = 42
+    BF16 = 30
     Ternary = 1000
     SparseTernary = 1001
 
@@ -557,7 +558,18 @@ class GpuModel:
         gm._keep.append(gf)
         return gm
 
-    def config(self) -> GpuModelConfig:
+    @classmethod
+    def load_stack(cls, engine: GpuEngine, source, dtype: str = "bfloat16", max_seq_len: int = 4096) -> "GpuModel":
+        """A layer-stack model (alice_llm_b200.stack) from a checkpoint folder, or from (config dict, {name: array}).
+        dtype "float32" keeps every activation, product and cache in 32 bits."""
+        from . import stack
+        if isinstance(source, tuple):
+            h, cfg, keep = stack.load_tensors(engine, source[0], source[1], dtype, max_seq_len)
+        else:
+            h, cfg, keep = stack.load_dir(engine, source, dtype, max_seq_len)
+        return cls(engine, h, cfg, keep)
+
+    def config(self):
         return self._config
 
     def free(self):
@@ -612,6 +624,36 @@ class GpuModel:
         check(self.engine._lib.alice_model_forward_batch_read(self._h, _ptr(t), t.size, _ptr(out)))
         return out
 
+    def forward_rows(self, token_ids, rows) -> np.ndarray:
+        """Any number of consecutive tokens; -> logits [len(rows), vocab] at the ascending places `rows` among them."""
+        t, r = _np(token_ids, np.uint32).reshape(-1), _np(rows, np.uint32).reshape(-1)
+        out = np.empty((r.size, self._config.vocab_size), np.float32)
+        check(self.engine._lib.alice_model_forward_rows(self._h, _ptr(t), t.size, _ptr(r), r.size, _ptr(out)))
+        return out
+
+    def generate(self, prompt, n: int) -> np.ndarray:
+        """n greedy tokens after `prompt` from the present position (Llama3Model::generate, src/llama3.rs:16084): the prompt
+        but its last token as one forward pass, then the decode loop on the device."""
+        prompt = _np(prompt, np.uint32).reshape(-1)
+        if prompt.size == 0:
+            raise AliceError(_lib.E_SHAPE, "generate: empty prompt")
+        if prompt.size > 1:
+            self.forward_rows(prompt[:-1], [])
+        return self.decode_greedy(int(prompt[-1]), n)
+
+    # -- layer-stack models: the residual stream after every layer run --
+    def trace(self, on: bool):
+        check(self.engine._lib.alice_stack_trace(self._h, int(on)))
+
+    def read_trace(self) -> np.ndarray:
+        """[layer runs, tokens, width] of the most recent forward call."""
+        runs, tokens = C.c_uint32(), C.c_uint32()
+        fn = self.engine._lib.alice_stack_read_trace
+        check(fn(self._h, None, 0, C.byref(runs), C.byref(tokens)))
+        out = np.empty((runs.value, tokens.value, self._config.width), np.float32)
+        check(fn(self._h, _ptr(out), out.size, C.byref(runs), C.byref(tokens)))
+        return out
+
     def decode_greedy(self, first_token: int, n: int) -> np.ndarray:
         out = np.empty(n, np.uint32)
         check(self.engine._lib.alice_model_decode_greedy(self._h, first_token, n, _ptr(out)))
@@ -635,6 +677,8 @@ class GpuModel:
     # -- pre-filled context (no reference counterpart: the benchmark starts from a filled KV cache) --
     def _local_kv_dim(self) -> int:
         """Floats per cached position on this rank: the KV heads are sharded over a tensor-parallel group."""
+        if not hasattr(self._config, "num_kv_heads"):
+            raise AliceError(_lib.E_UNSUPPORTED, "this model keeps no key / value rows")
         return self._config.num_kv_heads * self._config.head_dim // self.engine.tp_info()[1]
 
     def kv_write(self, layer: int, pos0: int, k, v):

@@ -43,6 +43,7 @@ extern "C" {
 #define ALICE_TYPE_Q6_K 14u
 #define ALICE_TYPE_Q1_0 41u
 #define ALICE_TYPE_Q2_0 42u
+#define ALICE_TYPE_BF16 30u /* dense bfloat16 rows; alice_matvec wants cols % 64 == 0 */
 
 typedef struct alice_engine alice_engine;   /* GpuEngine, src/gpu.rs:320 */
 typedef struct alice_weights alice_weights; /* GpuWeightBuffer, src/gpu.rs:302 */
@@ -236,6 +237,10 @@ int32_t alice_model_forward_batch_read(alice_model* m, const uint32_t* tokens, u
  * step i. No host round trip between steps. */
 int32_t alice_model_decode_greedy(alice_model* m, uint32_t first_token, uint32_t n, uint32_t* out_tokens);
 int32_t alice_model_read_logits(alice_model* m, float* logits);
+/* Any number of consecutive tokens (cut into pieces the model takes at once), with the logits of rows[0 .. nrows)
+ * (ascending places among these tokens, possibly none) written to logits[i * vocab + v]. Blocks. The prompt phase of
+ * Llama3Model::generate (src/llama3.rs:16084), which looks at the last token's logits only. */
+int32_t alice_model_forward_rows(alice_model* m, const uint32_t* tokens, uint32_t n, const uint32_t* rows, uint32_t nrows, float* logits);
 /* Tensor parallel without collective calls: after every rank has created its model, each exports a handle to its
  * exchange region (ALICE_TP_HANDLE_BYTES; CUDA IPC, same node), the host gathers the handles of all ranks in rank
  * order and every rank connects. From then on the kernel that produces a sharded vector stores its rows straight
@@ -259,6 +264,61 @@ int32_t alice_model_reset(alice_model* m);
 int32_t alice_model_kv_write(alice_model* m, uint32_t layer, uint32_t pos0, uint32_t npos, const float* k, const float* v);
 int32_t alice_model_kv_read(alice_model* m, uint32_t layer, uint32_t pos0, uint32_t npos, float* k, float* v);
 int32_t alice_model_set_position(alice_model* m, uint32_t pos);
+
+/* ---- layer-stack models ------------------------------------------------------------------------ */
+/* A decoder whose layers are listed one by one, each with its own token mixer, as another kind of alice_model: the same
+ * step, greedy-decode, logits and reset calls drive it. No counterpart in the reference. Each layer adds
+ *   ls1 * mixer(h) + ls2 * mlp(h),   h = layer_norm(x) (weight, no bias),
+ * to a 32-bit residual stream; the head is the embedding table behind a last layer norm. Layers loop_start .. loop_stop - 1
+ * run loop_times times in a row with the same weights and a state or cache per pass; ahead of pass t the embedding output
+ * (t > 0) and loop_step[t] join the stream. loop_times == 0: no loop.
+ *
+ * Mixers:
+ *   ALICE_MIX_LATENT  attention over a cached latent row per token (query through a latent of q_rank, one rotated key part of
+ *                     rot_dim for all heads, half-split rotation of its first rot_dims), softmax with a sink per head,
+ *                     sigmoid output gate.
+ *   ALICE_MIX_DELTA   gated delta rule with one decay per key channel, short causal convolutions on q, k, v, root-mean-square
+ *                     norm and sigmoid gate on the output; recurrent state in 32 bits.
+ *
+ * Matrices are ALICE_TYPE_BF16 handles whose columns are zero-padded to a multiple of 64 (P() below), and whose row segments
+ * start at multiples of 64 rows (zero rows between):
+ *   in    latent: [P(q_rank) query latent | P(kv_rank + rot_dim) key latent, key part | P(heads * vdim) gate]
+ *         delta:  [P(kv_heads * dim) q | same k | P(heads * vdim) v | P(heads) step | P(decay_rank) | P(gate_rank)]
+ *   uq    [heads * (dim + rot_dim)][P(q_rank)]       uk [heads * dim][P(kv_rank)]      uv [heads * vdim][P(kv_rank)]
+ *   a2    [heads * D][P(decay_rank)] with dim padded to D = 32, 64, 128 or 256 per head; dt_bias likewise [heads * D]
+ *   g2    [heads * vdim][P(gate_rank)]               o  [width][P(heads * vdim)]
+ *   gu    64 gate rows, 64 up rows, 64 gate rows, ... of P(ff) each [2 P(ff)][P(width)]; down [width][P(ff)]
+ *   embed [vocab][P(width)]
+ * and gate_bias / up_bias hold P(ff) floats. conv [columns of q | k | v in `in`][conv_taps]. Float arrays are copied. */
+#define ALICE_MIX_LATENT 1u
+#define ALICE_MIX_DELTA 2u
+typedef struct {
+    uint32_t mixer;
+    uint32_t heads, kv_heads, dim, vdim;
+    uint32_t q_rank, kv_rank, rot_dim, rot_dims;     /* latent */
+    uint32_t conv_taps, decay_rank, gate_rank;       /* delta */
+    uint32_t ff;                                     /* 0: no feed-forward */
+    float scale;                                     /* latent: factor on the scores */
+    double rot_base;
+    const alice_weights *in, *uq, *uk, *uv, *a2, *g2, *o, *gu, *down;
+    const float *norm, *ls1, *ls2, *gate_bias, *up_bias, *down_bias;
+    const float *q_norm, *kv_norm, *sink;            /* latent */
+    const float *conv, *a_log, *dt_bias, *head_norm; /* delta */
+} alice_stack_layer;
+typedef struct {
+    uint32_t num_layers, width, vocab_size, max_seq_len;
+    uint32_t loop_start, loop_stop, loop_times;
+    uint32_t exact;                                  /* 1: every activation, product and cache in 32 bits */
+    float eps, embed_scale;
+    const float* loop_step;                          /* [loop_times][width] */
+} alice_stack_config;
+int32_t alice_stack_create(alice_engine* e, const alice_stack_config* cfg, const alice_stack_layer* layers, const alice_weights* embed,
+                           const float* final_norm, alice_model** out);
+/* The residual stream (width floats per token) of the tokens of the most recent forward call, after each layer run that
+ * follows: 1 switches the recording on (forward calls then take at most 256 tokens), 0 off. alice_stack_read_trace copies
+ * it out as [layer runs][tokens][width]; *runs and *tokens tell the extents (out may be null to ask). */
+int32_t alice_stack_trace(alice_model* m, int32_t on);
+int32_t alice_stack_read_trace(alice_model* m, float* out, size_t out_floats, uint32_t* runs, uint32_t* tokens);
 
 /* ---- no-allocation variant ---------------------------------------------------------------- */
 /* Has no counterpart in the reference. alice_matvec_preq for Q1_0 / Q2_0 weights needs an f32 copy
