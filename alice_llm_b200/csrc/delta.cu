@@ -10,18 +10,31 @@
 namespace alice {
 namespace {
 
-// Convolution input of channel c, `back` tokens before token t (the state holds the tokens before the first one).
-__device__ __forceinline__ float conv_in(const DeltaArgs& a, int t, int back, uint32_t c) {
-    const int s = t - back;
-    if (s >= 0) return a.y[(size_t)s * a.ldy + c];
-    return a.conv_state[(size_t)((int)a.s.taps - 1 + s) * a.s.conv_cols + c];
+// Inputs of the convolution before the tokens at hand, and where those of the next call go.
+__device__ __forceinline__ const float* conv_before(const DeltaArgs& a) {
+    return a.conv_state + (size_t)(*a.pos & 1) * (a.s.taps - 1) * a.s.conv_cols;
 }
-__device__ __forceinline__ float conv_silu(const DeltaArgs& a, int t, uint32_t c) {
+__device__ __forceinline__ float* conv_after(const DeltaArgs& a, uint32_t tokens) {
+    return a.conv_state + (size_t)((*a.pos + (int)tokens) & 1) * (a.s.taps - 1) * a.s.conv_cols;
+}
+// Convolution and silu of channel c at token t.
+__device__ __forceinline__ float conv_silu(const DeltaArgs& a, const float* before, int t, uint32_t c) {
     const int taps = (int)a.s.taps;
     const float* w = a.conv_w + (size_t)c * taps;
     float v = 0.0f;
-    for (int j = 0; j < taps; j++) v = fmaf(w[j], conv_in(a, t, taps - 1 - j, c), v);
+    for (int j = 0; j < taps; j++) {
+        const int s = t - (taps - 1 - j);
+        v = fmaf(w[j], s >= 0 ? a.y[(size_t)s * a.ldy + c] : before[(size_t)(taps - 1 + s) * a.s.conv_cols + c], v);
+    }
     return silu_ref(v);
+}
+// Inputs of channel c that the next call needs: the last taps - 1 of [before; the tokens at hand].
+__device__ __forceinline__ void conv_keep(const DeltaArgs& a, const float* before, float* after, uint32_t tokens, uint32_t c) {
+    const uint32_t keep = a.s.taps - 1;
+    for (uint32_t j = 0; j < keep; j++) {
+        const uint32_t i = tokens + j;
+        after[(size_t)j * a.s.conv_cols + c] = i < keep ? before[(size_t)i * a.s.conv_cols + c] : a.y[(size_t)(i - keep) * a.ldy + c];
+    }
 }
 
 // One warp per (token, key head) or (token, value head).
@@ -32,6 +45,7 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const __grid_constan
     const uint32_t lane = threadIdx.x & 31, per = s.kv_heads + s.heads;
     const size_t task = (size_t)blockIdx.x * 8 + (threadIdx.x >> 5);
     if (task >= (size_t)tokens * per) return;
+    const float* before = conv_before(a);
     const uint32_t t = (uint32_t)(task / per), i = (uint32_t)(task % per);
     if (i < s.kv_heads) {
         constexpr int N = DELTA_MAX_DIM / 32;
@@ -41,8 +55,8 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const __grid_constan
             const uint32_t d = lane + 32 * j;
             q[j] = k[j] = 0.0f;
             if (d < s.dim) {
-                q[j] = conv_silu(a, (int)t, s.off_q + i * s.dim + d);
-                k[j] = conv_silu(a, (int)t, s.off_k + i * s.dim + d);
+                q[j] = conv_silu(a, before, (int)t, s.off_q + i * s.dim + d);
+                k[j] = conv_silu(a, before, (int)t, s.off_k + i * s.dim + d);
             }
             sq = fmaf(q[j], q[j], sq); sk = fmaf(k[j], k[j], sk);
         }
@@ -62,22 +76,18 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const __grid_constan
     } else {
         const uint32_t h = i - s.kv_heads;
         const size_t o = ((size_t)t * s.heads + h) * s.vp;
-        for (uint32_t d = lane; d < s.vp; d += 32) a.v[o + d] = d < s.vdim ? conv_silu(a, (int)t, s.off_v + h * s.vdim + d) : 0.0f;
+        for (uint32_t d = lane; d < s.vp; d += 32) a.v[o + d] = d < s.vdim ? conv_silu(a, before, (int)t, s.off_v + h * s.vdim + d) : 0.0f;
         if (lane == 0) a.beta[(size_t)t * s.heads + h] = sigmoid_f(a.y[(size_t)t * a.ldy + s.off_b + h]);
     }
 }
 
-// The last taps - 1 inputs of every channel (ascending, so an entry is read before it is overwritten).
+// The two halves of the convolution state differ unless an even number of tokens passed: then this call reads and writes the
+// same half. A thread owns its channel, reads ahead of what it overwrites, and runs after all other readers.
 __global__ void __launch_bounds__(256) conv_tail_kernel(const __grid_constant__ DeltaArgs a, uint32_t tokens) {
     pdl_launch_dependents();
     pdl_wait();
-    const uint32_t c = blockIdx.x * 256 + threadIdx.x, keep = a.s.taps - 1;
-    if (c >= a.s.conv_cols) return;
-    for (uint32_t j = 0; j < keep; j++) {
-        const uint32_t i = tokens + j;      // index into [state; new tokens]
-        a.conv_state[(size_t)j * a.s.conv_cols + c] =
-            i < keep ? a.conv_state[(size_t)i * a.s.conv_cols + c] : a.y[(size_t)(i - keep) * a.ldy + c];
-    }
+    const uint32_t c = blockIdx.x * 256 + threadIdx.x;
+    if (c < a.s.conv_cols) conv_keep(a, conv_before(a), conv_after(a, tokens), tokens, c);
 }
 
 constexpr int SCAN_COLS = 32, SCAN_CHUNK = 8;   // columns per CTA, tokens per staged chunk
@@ -198,6 +208,134 @@ __global__ void __launch_bounds__(256) delta_out_kernel(const __grid_constant__ 
         for (uint32_t d = s.vdim + lane; d < a.ldo - h * s.vdim; d += 32) put(out + d, 0.0f);
 }
 
+// One token. A cluster of vp / 32 CTAs per head, each with 32 columns of the state (eight lanes a column); the head's
+// convolutions, decays and step size are worked out by every CTA for itself, the norm over vdim joins them.
+template <int E>
+__global__ void __launch_bounds__(256, 2) delta_step_kernel(const __grid_constant__ DeltaStepArgs a) {
+    constexpr uint32_t DP = 8 * E;
+    __shared__ __align__(16) float q[DP], k[DP], g[DP], v[SCAN_COLS], gate[SCAN_COLS], os[SCAN_COLS], red[8];
+    extern __shared__ __align__(16) float low[];   // low-rank inputs of the decay and of the gate
+    __shared__ float part[8];                      // one partial sum of squares per CTA of the cluster
+    const DeltaArgs& d = a.d;
+    const DeltaShape& s = d.s;
+    const uint32_t ncta = s.vp / SCAN_COLS, h = blockIdx.x / ncta, rank = blockIdx.x % ncta, c0 = rank * SCAN_COLS, kh = h / (s.heads / s.kv_heads);
+    const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, l = lane & 7, col = warp * 4 + (lane >> 3);
+    float* sp = d.state + ((size_t)h * s.vp + c0 + col) * DP + l * 4;
+    const bf16* wa = a.a2.w + (size_t)h * DP * a.a2.k;
+    const bf16* wg = a.g2.w + ((size_t)h * s.vdim + c0) * a.g2.k;
+    const uint32_t vrows = min((uint32_t)SCAN_COLS, s.vdim - c0);
+    pdl_launch_dependents();
+    asm volatile("barrier.cluster.arrive.relaxed;" ::: "memory");   // every CTA of the cluster runs before one writes to another
+#pragma unroll
+    for (int e = 0; e < E; e += 4) if (l == 0) prefetch_l2(sp + e * 8);
+    for (uint32_t i = tid; i < DP * (a.a2.k / 64); i += 256) prefetch_l2(wa + (size_t)i * 64);
+    for (uint32_t i = tid; i < vrows * (a.g2.k / 64); i += 256) prefetch_l2(wg + (size_t)i * 64);
+    pdl_wait();
+    const float* before = conv_before(d);
+    float S[E];
+#pragma unroll
+    for (int e = 0; e < E; e += 4) {
+        const float4 f = *reinterpret_cast<const float4*>(sp + e * 8);
+        S[e] = f.x; S[e + 1] = f.y; S[e + 2] = f.z; S[e + 3] = f.w;
+    }
+    for (uint32_t i = tid; i < a.a2.k; i += 256) low[i] = d.y[a.off_a + i];
+    for (uint32_t i = tid; i < a.g2.k; i += 256) low[a.a2.k + i] = d.y[a.off_g + i];
+    const float qv = tid < s.dim ? conv_silu(d, before, 0, s.off_q + kh * s.dim + tid) : 0.0f;
+    const float kv = tid < s.dim ? conv_silu(d, before, 0, s.off_k + kh * s.dim + tid) : 0.0f;
+    const float sq = block_sum<8>(qv * qv, red), sk = block_sum<8>(kv * kv, red);   // also publishes `low`
+    if (tid < DP) {
+        q[tid] = qv * __frcp_rn(__fsqrt_rn(sq + 1e-6f)) * __frcp_rn(__fsqrt_rn((float)s.dim));
+        k[tid] = kv * __frcp_rn(__fsqrt_rn(sk + 1e-6f));
+    }
+    if (tid < SCAN_COLS) v[tid] = c0 + tid < s.vdim ? conv_silu(d, before, 0, s.off_v + h * s.vdim + c0 + tid) : 0.0f;
+    const float beta = sigmoid_f(d.y[s.off_b + h]), rate = expf(a.a_log[h]);
+    // low-rank projections: sixteen lanes a row
+    const uint32_t hw = tid >> 4, hl = tid & 15;
+    for (uint32_t r = hw; r < DP + SCAN_COLS; r += 16) {
+        const bool decay = r < DP;
+        const uint32_t kk = decay ? a.a2.k : a.g2.k, row = decay ? r : r - DP;
+        const bf16* w = decay ? wa + (size_t)row * kk : wg + (size_t)min(row, vrows - 1) * kk;
+        const float* x = decay ? low : low + a.a2.k;
+        float acc = 0.0f;
+        for (uint32_t c = hl * 8; c < kk; c += 128) {
+            const uint4 u = __ldg(reinterpret_cast<const uint4*>(w + c));
+            const float2 e0 = bf2(u.x), e1 = bf2(u.y), e2 = bf2(u.z), e3 = bf2(u.w);
+            acc = fmaf(e0.x, x[c], acc); acc = fmaf(e0.y, x[c + 1], acc); acc = fmaf(e1.x, x[c + 2], acc); acc = fmaf(e1.y, x[c + 3], acc);
+            acc = fmaf(e2.x, x[c + 4], acc); acc = fmaf(e2.y, x[c + 5], acc); acc = fmaf(e3.x, x[c + 6], acc); acc = fmaf(e3.y, x[c + 7], acc);
+        }
+#pragma unroll
+        for (int o = 8; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+        if (hl == 0) {
+            if (decay) g[row] = expf(-rate * softplus_f(acc + a.dt_bias[(size_t)h * DP + row]));
+            else gate[row] = sigmoid_f(acc);
+        }
+    }
+    __syncthreads();
+    float dk = 0.0f, dq = 0.0f, kq = 0.0f;
+#pragma unroll
+    for (int e = 0; e < E; e++) {
+        const uint32_t i = (e / 4) * 32 + l * 4 + e % 4;
+        S[e] *= g[i];
+        dk = fmaf(S[e], k[i], dk);
+        dq = fmaf(S[e], q[i], dq);
+        kq = fmaf(k[i], q[i], kq);
+    }
+#pragma unroll
+    for (int o = 4; o > 0; o >>= 1) {
+        dk += __shfl_xor_sync(0xffffffffu, dk, o);
+        dq += __shfl_xor_sync(0xffffffffu, dq, o);
+        kq += __shfl_xor_sync(0xffffffffu, kq, o);
+    }
+    const float u = beta * (v[col] - dk);
+#pragma unroll
+    for (int e = 0; e < E; e += 4) {
+        const uint32_t i = e * 8 + l * 4;
+        *reinterpret_cast<float4*>(sp + e * 8) = make_float4(fmaf(k[i], u, S[e]), fmaf(k[i + 1], u, S[e + 1]), fmaf(k[i + 2], u, S[e + 2]), fmaf(k[i + 3], u, S[e + 3]));
+    }
+    if (l == 0) os[col] = fmaf(kq, u, dq);
+    __syncthreads();
+    asm volatile("barrier.cluster.wait;" ::: "memory");
+    float ss = 0.0f;
+    if (warp == 0) {
+        ss = warp_sum(lane < vrows ? os[lane] * os[lane] : 0.0f);
+        if (lane < ncta) {   // the slice's sum of squares into every CTA of the cluster
+            uint32_t dst;
+            asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(dst) : "r"(smem_u32(&part[rank])), "r"(lane));
+            asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(dst), "f"(ss) : "memory");
+        }
+    }
+    asm volatile("barrier.cluster.arrive.release;\n\tbarrier.cluster.wait.acquire;" ::: "memory");
+    if (tid < vrows) {
+        float tot = 0.0f;
+        for (uint32_t i = 0; i < ncta; i++) tot += part[i];
+        const float inv = __frcp_rn(__fsqrt_rn(tot / (float)s.vdim + d.eps));
+        static_cast<float*>(d.out)[(size_t)h * s.vdim + c0 + tid] = os[tid] * inv * d.norm_w[c0 + tid] * gate[tid];
+    }
+    // what the next token's convolution needs: a head's own value columns, and the key head's channels once per key head
+    float* after = conv_after(d, 1);
+    if (tid < vrows) conv_keep(d, before, after, 1, s.off_v + h * s.vdim + c0 + tid);
+    if (rank == 0 && h % (s.heads / s.kv_heads) == 0 && tid < s.dim) {
+        conv_keep(d, before, after, 1, s.off_q + kh * s.dim + tid);
+        conv_keep(d, before, after, 1, s.off_k + kh * s.dim + tid);
+    }
+    if (h + 1 == s.heads && rank + 1 == ncta)   // padding up to the stride
+        for (uint32_t i = s.heads * s.vdim + tid; i < d.ldo; i += 256) static_cast<float*>(d.out)[i] = 0.0f;
+}
+
+template <int E>
+cudaError_t step_e(const DeltaStepArgs& a, cudaStream_t st, bool pdl) {
+    const uint32_t ncta = a.d.s.vp / SCAN_COLS;
+    cudaLaunchConfig_t lc = {};
+    lc.gridDim = dim3(a.d.s.heads * ncta); lc.blockDim = dim3(256); lc.dynamicSmemBytes = (size_t)(a.a2.k + a.g2.k) * 4; lc.stream = st;
+    cudaLaunchAttribute at[2];
+    at[0].id = cudaLaunchAttributeClusterDimension;
+    at[0].val.clusterDim.x = ncta; at[0].val.clusterDim.y = 1; at[0].val.clusterDim.z = 1;
+    at[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[1].val.programmaticStreamSerializationAllowed = 1;
+    lc.attrs = at; lc.numAttrs = pdl ? 2 : 1;
+    return cudaLaunchKernelEx(&lc, delta_step_kernel<E>, a);
+}
+
 template <int E>
 cudaError_t scan_e(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
     static bool done[64] = {};
@@ -222,6 +360,17 @@ cudaError_t launch_delta_scan(const DeltaArgs& a, uint32_t tokens, cudaStream_t 
         case 64: return scan_e<8>(a, tokens, st, pdl);
         case 128: return scan_e<16>(a, tokens, st, pdl);
         case 256: return scan_e<32>(a, tokens, st, pdl);
+        default: return cudaErrorInvalidValue;
+    }
+}
+
+cudaError_t launch_delta_step(const DeltaStepArgs& a, cudaStream_t st, bool pdl) {
+    if (!delta_step_fits(a.d.s) || (size_t)(a.a2.k + a.g2.k) * 4 > 32 * 1024) return cudaErrorInvalidValue;
+    switch (a.d.s.dp) {
+        case 32: return step_e<4>(a, st, pdl);
+        case 64: return step_e<8>(a, st, pdl);
+        case 128: return step_e<16>(a, st, pdl);
+        case 256: return step_e<32>(a, st, pdl);
         default: return cudaErrorInvalidValue;
     }
 }

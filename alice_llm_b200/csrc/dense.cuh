@@ -69,6 +69,6 @@ struct GemmOp {
     uint32_t dim = 1;
 };
 // bf16 inputs run on the tensor cores, f32 inputs in f32 arithmetic throughout.
-cudaError_t launch_dense_gemm(const GemmOp& op, int* status, cudaStream_t st, bool pdl);
+cudaError_t launch_dense_gemm(const GemmOp& op, int num_sms, int* status, cudaStream_t st, bool pdl);
 
 }  // namespace alice

@@ -1,5 +1,6 @@
 // Many tokens against dense bfloat16 rows. f32 inputs: register-tiled f32 arithmetic (every product and sum in 32 bits).
-#include "dense_epi.cuh"
+// bf16 inputs: tensor cores (dense_tc.cuh).
+#include "dense_tc.cuh"
 
 namespace alice {
 namespace {
@@ -10,14 +11,9 @@ __device__ __forceinline__ void load_a4(float (&r)[4], const float* p) {
     const float4 v = *reinterpret_cast<const float4*>(p);
     r[0] = v.x; r[1] = v.y; r[2] = v.z; r[3] = v.w;
 }
-__device__ __forceinline__ void load_a4(float (&r)[4], const bf16* p) {
-    const uint2 v = *reinterpret_cast<const uint2*>(p);
-    const float2 a = bf2(v.x), b = bf2(v.y);
-    r[0] = a.x; r[1] = a.y; r[2] = b.x; r[3] = b.y;
-}
 
 // 256 threads; a thread owns 4 tokens x (4 columns of the tile's first half + the same 4 of its second half).
-template <class AT, int EPI>
+template <int EPI>
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ GemmOp op) {
     __shared__ __align__(16) float As[BK][BM + 4], Bs[BK][BN + 4];
     const uint32_t tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
@@ -25,7 +21,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ G
     const uint32_t ar = tid >> 2, ak = (tid & 3) * 4, br = tid >> 1, bk = (tid & 1) * 8;
     pdl_launch_dependents();
     pdl_wait();
-    const AT* ap = static_cast<const AT*>(op.a) + (size_t)(t0 + ar) * op.lda + ak;
+    const float* ap = static_cast<const float*>(op.a) + (size_t)(t0 + ar) * op.lda + ak;
     const bf16* bp = op.w.w + (size_t)(n0 + br) * op.w.k + bk;
     const bool a_ok = t0 + ar < op.tokens, b_ok = n0 + br < op.w.n;
     float acc[4][8] = {};
@@ -72,25 +68,78 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ G
     }
 }
 
-template <class AT>
 cudaError_t launch_f32(const GemmOp& op, cudaStream_t st, bool pdl) {
     const dim3 grid((op.w.n + BN - 1) / BN, (op.tokens + BM - 1) / BM);
     switch (op.epi) {
-        case EPI_STORE: return launch_pdl(gemm_f32_kernel<AT, EPI_STORE>, grid, dim3(256), 0, st, pdl, op);
-        case EPI_SWIGLU: return launch_pdl(gemm_f32_kernel<AT, EPI_SWIGLU>, grid, dim3(256), 0, st, pdl, op);
-        case EPI_RESID: return launch_pdl(gemm_f32_kernel<AT, EPI_RESID>, grid, dim3(256), 0, st, pdl, op);
-        case EPI_DECAY: return launch_pdl(gemm_f32_kernel<AT, EPI_DECAY>, grid, dim3(256), 0, st, pdl, op);
-        case EPI_SIGMOID: return launch_pdl(gemm_f32_kernel<AT, EPI_SIGMOID>, grid, dim3(256), 0, st, pdl, op);
+        case EPI_STORE: return launch_pdl(gemm_f32_kernel<EPI_STORE>, grid, dim3(256), 0, st, pdl, op);
+        case EPI_SWIGLU: return launch_pdl(gemm_f32_kernel<EPI_SWIGLU>, grid, dim3(256), 0, st, pdl, op);
+        case EPI_RESID: return launch_pdl(gemm_f32_kernel<EPI_RESID>, grid, dim3(256), 0, st, pdl, op);
+        case EPI_DECAY: return launch_pdl(gemm_f32_kernel<EPI_DECAY>, grid, dim3(256), 0, st, pdl, op);
+        case EPI_SIGMOID: return launch_pdl(gemm_f32_kernel<EPI_SIGMOID>, grid, dim3(256), 0, st, pdl, op);
         default: return cudaErrorInvalidValue;
     }
 }
 
+using EncodeFn = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
+                              const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+EncodeFn encode_fn() {
+    static EncodeFn fn = [] {
+        void* p = nullptr;
+        cudaDriverEntryPointQueryResult q;
+        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q) != cudaSuccess || q != cudaDriverEntryPointSuccess) p = nullptr;
+        return reinterpret_cast<EncodeFn>(p);
+    }();
+    return fn;
+}
+
+// rows x cols bf16, ld elements between rows, copied as tiles of box_rows x 64 (rows past the end read as zero)
+bool tile_map(CUtensorMap* map, const void* base, uint32_t rows, uint32_t cols, uint32_t ld, uint32_t box_rows) {
+    const cuuint64_t dims[2] = {cols, rows}, strides[1] = {(cuuint64_t)ld * 2};
+    const cuuint32_t box[2] = {TC_BK, box_rows}, step[2] = {1, 1};
+    return encode_fn()(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, step, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                       CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+
+template <int BN, int EPI>
+cudaError_t tc_inst(const TcArgs& a, uint32_t grid, cudaStream_t st, bool pdl) {
+    static bool done[64] = {};
+    const cudaError_t err = allow_smem(gemm_tc_kernel<BN, EPI>, TcGeom<BN>::SMEM, done);
+    if (err != cudaSuccess) return err;
+    return launch_pdl(gemm_tc_kernel<BN, EPI>, dim3(grid), dim3(TC_THREADS), TcGeom<BN>::SMEM, st, pdl, a);
+}
+template <int BN>
+cudaError_t tc_epi(const TcArgs& a, uint32_t grid, cudaStream_t st, bool pdl) {
+    switch (a.op.epi) {
+        case EPI_STORE: return tc_inst<BN, EPI_STORE>(a, grid, st, pdl);
+        case EPI_SWIGLU: return tc_inst<BN, EPI_SWIGLU>(a, grid, st, pdl);
+        case EPI_RESID: return tc_inst<BN, EPI_RESID>(a, grid, st, pdl);
+        case EPI_DECAY: return tc_inst<BN, EPI_DECAY>(a, grid, st, pdl);
+        case EPI_SIGMOID: return tc_inst<BN, EPI_SIGMOID>(a, grid, st, pdl);
+        default: return cudaErrorInvalidValue;
+    }
+}
+
+cudaError_t launch_tc(const GemmOp& op, int num_sms, int* status, cudaStream_t st, bool pdl) {
+    if (!encode_fn()) return cudaErrorNotSupported;
+    TcArgs a;
+    a.op = op; a.status = status;
+    const uint32_t tt = (op.tokens + TC_BM - 1) / TC_BM;
+    // wide tiles when they still give every SM one
+    const bool wide = tt * ((op.w.n + 255) / 256) >= (uint32_t)num_sms;
+    const uint32_t bn = wide ? 256 : 128, tiles = tt * ((op.w.n + bn - 1) / bn);
+    if (!tile_map(&a.ta, op.a, op.tokens, op.w.k, op.lda, TC_BM) || !tile_map(&a.tw, op.w.w, op.w.n, op.w.k, op.w.k, bn)) return cudaErrorInvalidValue;
+    const uint32_t grid = std::min(tiles, (uint32_t)num_sms);
+    return wide ? tc_epi<256>(a, grid, st, pdl) : tc_epi<128>(a, grid, st, pdl);
+}
+
 }  // namespace
 
-cudaError_t launch_dense_gemm(const GemmOp& op, int* status, cudaStream_t st, bool pdl) {
-    (void)status;
-    if (!op.tokens || !op.w.n || op.w.k % DENSE_PAD || op.lda % 8 || ((uintptr_t)op.a & 15) || (op.epi == EPI_SWIGLU && op.w.n % 128)) return cudaErrorInvalidValue;
-    return op.a_bf16 ? launch_f32<bf16>(op, st, pdl) : launch_f32<float>(op, st, pdl);
+cudaError_t launch_dense_gemm(const GemmOp& op, int num_sms, int* status, cudaStream_t st, bool pdl) {
+    if (!op.tokens || !op.w.n || op.w.k % DENSE_PAD || op.lda % 8 || ((uintptr_t)op.a & 15) || ((uintptr_t)op.out & 15) || (op.epi == EPI_SWIGLU && op.w.n % 128))
+        return cudaErrorInvalidValue;
+    if (!op.a_bf16) return launch_f32(op, st, pdl);
+    if (op.epi == EPI_SWIGLU && (!op.out_bf16 || op.ldo % 8)) return cudaErrorInvalidValue;
+    return launch_tc(op, num_sms, status, st, pdl);
 }
 
 }  // namespace alice

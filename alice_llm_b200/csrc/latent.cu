@@ -14,39 +14,50 @@ __device__ __forceinline__ void rotate_pair(float u, float v, float angle, float
     b = v * c + u * s;
 }
 
-// One CTA per token: norm of the query latent; norm of the key latent and the rotated key part into the cache.
+// Norm of the key latent and the rotated key part into the cache (a block of NT threads).
+template <class CT, int NT>
+__device__ __forceinline__ void cache_append(const LatentArgs& a, uint32_t t, float* red) {
+    const LatentShape& s = a.s;
+    const uint32_t p = (uint32_t)*a.pos + t;
+    const float* y = a.y + (size_t)t * a.ldy + s.off_kv;
+    float q = 0.0f;
+    for (uint32_t i = threadIdx.x; i < s.kv_rank; i += NT) q = fmaf(y[i], y[i], q);
+    q = block_sum<NT / 32>(q, red);
+    const float inv = __frcp_rn(__fsqrt_rn(q / (float)s.kv_rank + a.eps));
+    CT* row = static_cast<CT*>(a.cache) + (size_t)p * (s.cp + s.rp);
+    for (uint32_t i = threadIdx.x; i < s.kv_rank; i += NT) put(row + i, y[i] * inv * a.kv_norm[i]);
+    const float* kr = y + s.kv_rank;
+    const uint32_t half = s.rot_dims / 2;
+    for (uint32_t i = threadIdx.x; i < half; i += NT) {
+        float u, v;
+        rotate_pair(kr[i], kr[half + i], (float)p * a.freq[i], u, v);
+        put(row + s.cp + i, u);
+        put(row + s.cp + half + i, v);
+    }
+    for (uint32_t i = s.rot_dims + threadIdx.x; i < s.rot; i += NT) put(row + s.cp + i, kr[i]);
+}
+
+// One CTA per token: norm of the query latent, and the token's cache row.
 template <class OT, class CT>
 __global__ void __launch_bounds__(128) latent_norm_kernel(const __grid_constant__ LatentArgs a) {
     __shared__ float red[4];
     pdl_launch_dependents();
     pdl_wait();
     const LatentShape& s = a.s;
-    const uint32_t t = blockIdx.x, p = (uint32_t)*a.pos + t;
-    const float* y = a.y + (size_t)t * a.ldy;
+    const uint32_t t = blockIdx.x;
+    const float* y = a.y + (size_t)t * a.ldy + s.off_q;
     float q = 0.0f;
-    for (uint32_t i = threadIdx.x; i < s.q_rank; i += 128) q = fmaf(y[s.off_q + i], y[s.off_q + i], q);
+    for (uint32_t i = threadIdx.x; i < s.q_rank; i += 128) q = fmaf(y[i], y[i], q);
     q = block_sum<4>(q, red);
-    float inv = __frcp_rn(__fsqrt_rn(q / (float)s.q_rank + a.eps));
+    const float inv = __frcp_rn(__fsqrt_rn(q / (float)s.q_rank + a.eps));
     OT* cq = static_cast<OT*>(a.cqn) + (size_t)t * s.qp;
-    for (uint32_t i = threadIdx.x; i < s.qp; i += 128) put(cq + i, i < s.q_rank ? y[s.off_q + i] * inv * a.q_norm[i] : 0.0f);
-    q = 0.0f;
-    for (uint32_t i = threadIdx.x; i < s.kv_rank; i += 128) q = fmaf(y[s.off_kv + i], y[s.off_kv + i], q);
-    q = block_sum<4>(q, red);
-    inv = __frcp_rn(__fsqrt_rn(q / (float)s.kv_rank + a.eps));
-    CT* row = static_cast<CT*>(a.cache) + (size_t)p * (s.cp + s.rp);
-    for (uint32_t i = threadIdx.x; i < s.kv_rank; i += 128) put(row + i, y[s.off_kv + i] * inv * a.kv_norm[i]);
-    const float* kr = y + s.off_kv + s.kv_rank;
-    const uint32_t half = s.rot_dims / 2;
-    for (uint32_t i = threadIdx.x; i < half; i += 128) {
-        float u, v;
-        rotate_pair(kr[i], kr[half + i], (float)p * a.freq[i], u, v);
-        put(row + s.cp + i, u);
-        put(row + s.cp + half + i, v);
-    }
-    for (uint32_t i = s.rot_dims + threadIdx.x; i < s.rot; i += 128) put(row + s.cp + i, kr[i]);
+    for (uint32_t i = threadIdx.x; i < s.qp; i += 128) put(cq + i, i < s.q_rank ? y[i] * inv * a.q_norm[i] : 0.0f);
+    cache_append<CT, 128>(a, t, red);
 }
 
-// grid (heads, cp / 64, tokens): 64 latent columns of one head's query; the first slice also rotates the rotated part.
+// grid (heads, cp / 64, tokens): 64 latent columns of one head's query; the first slice also rotates the rotated part. With
+// a.append one more row of CTAs (blockIdx.x == heads, first slice) makes the token's cache row.
+template <class CT>
 __global__ void __launch_bounds__(256) latent_absorb_kernel(const __grid_constant__ LatentArgs a) {
     extern __shared__ __align__(16) float sm[];   // query [dim], then 4 x 64 partial sums
     const LatentShape& s = a.s;
@@ -54,6 +65,11 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const __grid_constan
     float* qs = sm;
     float* part = sm + ((s.dim + 3) & ~3u);
     pdl_launch_dependents();
+    if (h == s.heads) {
+        pdl_wait();
+        if (blockIdx.y == 0) cache_append<CT, 256>(a, t, part);
+        return;
+    }
     const bf16* w = a.uk + (size_t)h * s.dim * s.cp + c0;
     // a thread sums 8 columns over every 32nd row; rows of the first round travel ahead of the wait
     const uint32_t cg = threadIdx.x & 7, dr = threadIdx.x >> 3;
@@ -281,7 +297,10 @@ cudaError_t launch_latent_norm(const LatentArgs& a, uint32_t tokens, cudaStream_
                         : launch_pdl(latent_norm_kernel<float, float>, dim3(tokens), dim3(128), 0, st, pdl, a);
 }
 cudaError_t launch_latent_absorb(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
-    return launch_pdl(latent_absorb_kernel, dim3(a.s.heads, a.s.cp / 64, tokens), dim3(256), (size_t)(((a.s.dim + 3) & ~3u) + 512) * 4, st, pdl, a);
+    const dim3 grid(a.s.heads + (a.append ? 1 : 0), a.s.cp / 64, tokens);
+    const size_t smem = (size_t)(((a.s.dim + 3) & ~3u) + 512) * 4;
+    return a.cache_bf16 ? launch_pdl(latent_absorb_kernel<bf16>, grid, dim3(256), smem, st, pdl, a)
+                        : launch_pdl(latent_absorb_kernel<float>, grid, dim3(256), smem, st, pdl, a);
 }
 cudaError_t launch_latent_attn(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
     return a.cache_bf16 ? attn_type<bf16>(a, tokens, st, pdl) : attn_type<float>(a, tokens, st, pdl);

@@ -1,0 +1,233 @@
+// Causal attention of many tokens over keys and values made from the cached latent rows, on the tensor cores: bf16 queries,
+// keys and values, f32 scores, softmax and sums. The softmax weights enter the weighted sum as a bf16 pair (value and
+// remainder), so they are not cut to eight bits. The sink of a head is the state the online softmax starts from: a key that
+// scores `sink` and has no value.
+#include "dense_dev.cuh"
+#include "mixers.cuh"
+
+namespace alice {
+namespace {
+
+constexpr int PF_KEYS = 64, PF_ROWS = 128;   // keys per tile; queries per CTA, 16 per warp
+
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
+    const __nv_bfloat162 b = __floats2bfloat162_rn(lo, hi);
+    return *reinterpret_cast<const uint32_t*>(&b);
+}
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool ok) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(ok ? 16u : 0u) : "memory");
+}
+
+// DQ, DV: query / key and value dimensions the tiles have room for (multiples of 16, zero beyond the true sizes).
+template <int DQ, int DV>
+struct PfGeom {
+    static constexpr int LQ = DQ + 8, LV = DV + 8;   // row strides: eight rows land in different banks
+    static constexpr size_t Q = (size_t)PF_ROWS * LQ * 2, K = (size_t)PF_KEYS * LQ * 2, V = (size_t)PF_KEYS * LV * 2, SMEM = Q + 2 * (K + V);
+};
+
+template <int DQ, int DV>
+__global__ void __launch_bounds__(256, 1) latent_prefill_kernel(const __grid_constant__ LatentArgs a, uint32_t tokens) {
+    using G = PfGeom<DQ, DV>;
+    extern __shared__ __align__(128) uint8_t sm[];
+    const LatentShape& s = a.s;
+    const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x;
+    const uint32_t t0 = (gridDim.y - 1 - blockIdx.y) * PF_ROWS;   // the longest rows first
+    auto* qs = reinterpret_cast<bf16*>(sm);
+    const uint32_t q_sm = smem_u32(sm), k_sm = q_sm + (uint32_t)G::Q, v_sm = k_sm + 2 * (uint32_t)G::K;
+    pdl_launch_dependents();
+    pdl_wait();
+    const uint32_t p0 = (uint32_t)*a.pos, qd = s.dim + s.rot;
+    const uint32_t rows = min((uint32_t)PF_ROWS, tokens - t0), keys = p0 + t0 + rows, ntiles = (keys + PF_KEYS - 1) / PF_KEYS;
+    const bf16* cache = static_cast<const bf16*>(a.cache);
+    const uint32_t cw = s.cp + s.rp, kw = s.heads * s.dim, vw = s.heads * s.vdim;
+
+    // zero what lies beyond the true sizes once (the copies below never touch it)
+    for (uint32_t i = tid; i < 2 * PF_KEYS * (DQ - qd); i += 256) {
+        const uint32_t r = i / (DQ - qd), c = qd + i % (DQ - qd);
+        reinterpret_cast<bf16*>(sm + G::Q + (r / PF_KEYS) * G::K)[(r % PF_KEYS) * G::LQ + c] = __float2bfloat16_rn(0.0f);
+    }
+    for (uint32_t i = tid; i < 2 * PF_KEYS * (DV - s.vdim); i += 256) {
+        const uint32_t r = i / (DV - s.vdim), c = s.vdim + i % (DV - s.vdim);
+        reinterpret_cast<bf16*>(sm + G::Q + 2 * G::K + (r / PF_KEYS) * G::V)[(r % PF_KEYS) * G::LV + c] = __float2bfloat16_rn(0.0f);
+    }
+    auto fetch = [&](uint32_t tile, uint32_t b) {
+        const uint32_t j0 = tile * PF_KEYS, nd = s.dim / 8, nr = s.rot / 8, nv = s.vdim / 8;
+        const uint32_t kd = k_sm + b * (uint32_t)G::K, vd = v_sm + b * (uint32_t)G::V;
+        for (uint32_t i = tid; i < PF_KEYS * nd; i += 256) {
+            const uint32_t r = i / nd, c = i % nd * 8, j = min(j0 + r, keys - 1);
+            cp16(kd + (r * G::LQ + c) * 2, a.k_all + (size_t)j * kw + (size_t)h * s.dim + c, j0 + r < keys);
+        }
+        for (uint32_t i = tid; i < PF_KEYS * nr; i += 256) {
+            const uint32_t r = i / nr, c = i % nr * 8, j = min(j0 + r, keys - 1);
+            cp16(kd + (r * G::LQ + s.dim + c) * 2, cache + (size_t)j * cw + s.cp + c, j0 + r < keys);
+        }
+        for (uint32_t i = tid; i < PF_KEYS * nv; i += 256) {
+            const uint32_t r = i / nv, c = i % nv * 8, j = min(j0 + r, keys - 1);
+            cp16(vd + (r * G::LV + c) * 2, a.v_all + (size_t)j * vw + (size_t)h * s.vdim + c, j0 + r < keys);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    fetch(0, 0);
+    // queries, the rotated part turned to its position on the way
+    const uint32_t half = s.rot_dims / 2;
+    for (uint32_t i = tid; i < PF_ROWS * DQ; i += 256) {
+        const uint32_t r = i / DQ, c = i % DQ;
+        float v = 0.0f;
+        if (r < rows && c < qd) {
+            const float* q = a.q + ((size_t)(t0 + r) * s.heads + h) * qd;
+            if (c >= s.dim && c < s.dim + s.rot_dims) {
+                const uint32_t d = c - s.dim, j = d < half ? d : d - half;
+                float sn, cs;
+                sincosf((float)(p0 + t0 + r) * a.freq[j], &sn, &cs);
+                const float x = q[s.dim + j], y = q[s.dim + half + j];
+                v = d < half ? x * cs - y * sn : y * cs + x * sn;
+            } else {
+                v = q[c];
+            }
+        }
+        qs[r * G::LQ + c] = __float2bfloat16_rn(v);
+    }
+
+    // a thread's two rows are lane / 4 and lane / 4 + 8 of its warp's sixteen
+    constexpr float LOG2E = 1.4426950408889634f;
+    const float scale = s.scale * LOG2E;
+    float m[2], l[2], o[DV / 8][4];
+    m[0] = m[1] = a.sink[h] * LOG2E;
+    l[0] = l[1] = (lane & 3) == 0 ? 1.0f : 0.0f;
+#pragma unroll
+    for (int i = 0; i < DV / 8; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
+    const uint32_t row0 = warp * 16 + lane / 4, see0 = p0 + t0 + row0, see1 = see0 + 8;   // last key a row sees
+    const uint32_t q_addr = q_sm + ((warp * 16 + lane % 16) * G::LQ + lane / 16 * 8) * 2;
+
+    for (uint32_t tile = 0; tile < ntiles; tile++) {
+        const uint32_t b = tile & 1;
+        if (tile + 1 < ntiles) {
+            fetch(tile + 1, b ^ 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        const uint32_t kt = k_sm + b * (uint32_t)G::K, vt = v_sm + b * (uint32_t)G::V;
+        float sc[PF_KEYS / 8][4];
+#pragma unroll
+        for (int i = 0; i < PF_KEYS / 8; i++) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.0f;
+        const uint32_t k_addr = kt + ((lane % 8 + lane / 16 * 8) * G::LQ + (lane / 8 % 2) * 8) * 2;
+#pragma unroll
+        for (int kk = 0; kk < DQ / 16; kk++) {
+            uint32_t qa[4];
+            ldsm4(qa, q_addr + kk * 32);
+#pragma unroll
+            for (int n = 0; n < PF_KEYS / 16; n++) {
+                uint32_t kb[4];
+                ldsm4(kb, k_addr + (n * 16 * G::LQ + kk * 16) * 2);
+                mma16816(sc[2 * n], qa, kb[0], kb[1]);
+                mma16816(sc[2 * n + 1], qa, kb[2], kb[3]);
+            }
+        }
+        const uint32_t j0 = tile * PF_KEYS + (lane & 3) * 2;
+        float top0 = m[0], top1 = m[1];
+        const bool edge = tile * PF_KEYS + PF_KEYS > p0 + t0 + warp * 16;   // some key of the tile is hidden from some row of the warp
+#pragma unroll
+        for (int i = 0; i < PF_KEYS / 8; i++) {
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                float v = sc[i][e] * scale;
+                if (edge && j0 + i * 8 + (e & 1) > (e < 2 ? see0 : see1)) v = -INFINITY;
+                sc[i][e] = v;
+            }
+            top0 = fmaxf(top0, fmaxf(sc[i][0], sc[i][1]));
+            top1 = fmaxf(top1, fmaxf(sc[i][2], sc[i][3]));
+        }
+#pragma unroll
+        for (int x = 1; x <= 2; x *= 2) {
+            top0 = fmaxf(top0, __shfl_xor_sync(0xffffffffu, top0, x));
+            top1 = fmaxf(top1, __shfl_xor_sync(0xffffffffu, top1, x));
+        }
+        const float f0 = exp2f(m[0] - top0), f1 = exp2f(m[1] - top1);
+        m[0] = top0; m[1] = top1;
+        l[0] *= f0; l[1] *= f1;
+#pragma unroll
+        for (int i = 0; i < DV / 8; i++) { o[i][0] *= f0; o[i][1] *= f0; o[i][2] *= f1; o[i][3] *= f1; }
+#pragma unroll
+        for (int i = 0; i < PF_KEYS / 8; i++) {
+            sc[i][0] = exp2f(sc[i][0] - top0); sc[i][1] = exp2f(sc[i][1] - top0);
+            sc[i][2] = exp2f(sc[i][2] - top1); sc[i][3] = exp2f(sc[i][3] - top1);
+            l[0] += sc[i][0] + sc[i][1]; l[1] += sc[i][2] + sc[i][3];
+        }
+        const uint32_t v_addr = vt + ((lane % 16) * G::LV + lane / 16 * 8) * 2;
+#pragma unroll
+        for (int kk = 0; kk < PF_KEYS / 16; kk++) {
+            uint32_t hi[4], lo[4];
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const float x = sc[2 * kk + e / 2][(e & 1) * 2], y = sc[2 * kk + e / 2][(e & 1) * 2 + 1];
+                hi[e] = pack_bf16(x, y);
+                const float2 r = bf2(hi[e]);
+                lo[e] = pack_bf16(x - r.x, y - r.y);
+            }
+#pragma unroll
+            for (int n = 0; n < DV / 16; n++) {
+                uint32_t vb[4];
+                ldsm4t(vb, v_addr + (kk * 16 * G::LV + n * 16) * 2);
+                mma16816(o[2 * n], hi, vb[0], vb[1]);
+                mma16816(o[2 * n + 1], hi, vb[2], vb[3]);
+                mma16816(o[2 * n], lo, vb[0], vb[1]);
+                mma16816(o[2 * n + 1], lo, vb[2], vb[3]);
+            }
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int r = 0; r < 2; r++) {
+        float den = l[r];
+        den += __shfl_xor_sync(0xffffffffu, den, 1);
+        den += __shfl_xor_sync(0xffffffffu, den, 2);
+        const float inv = __frcp_rn(den);
+        const uint32_t row = row0 + 8 * r;
+        if (row >= rows) continue;
+        const float* gate = a.y + (size_t)(t0 + row) * a.ldy + s.off_g + (size_t)h * s.vdim;
+        bf16* out = static_cast<bf16*>(a.out) + (size_t)(t0 + row) * a.ldo;
+#pragma unroll
+        for (int i = 0; i < DV / 8; i++) {
+            const uint32_t c = i * 8 + (lane & 3) * 2;
+            if (c < s.vdim)
+                *reinterpret_cast<uint32_t*>(out + (size_t)h * s.vdim + c) =
+                    pack_bf16(o[i][2 * r] * inv * sigmoid_f(gate[c]), o[i][2 * r + 1] * inv * sigmoid_f(gate[c + 1]));
+        }
+        if (h + 1 == s.heads)   // padding up to the stride
+            for (uint32_t c = s.heads * s.vdim + (lane & 3); c < a.ldo; c += 4) out[c] = __float2bfloat16_rn(0.0f);
+    }
+}
+
+template <int DQ, int DV>
+cudaError_t prefill_inst(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
+    static bool done[64] = {};
+    const cudaError_t err = allow_smem(latent_prefill_kernel<DQ, DV>, PfGeom<DQ, DV>::SMEM, done);
+    if (err != cudaSuccess) return err;
+    return launch_pdl(latent_prefill_kernel<DQ, DV>, dim3(a.s.heads, (tokens + PF_ROWS - 1) / PF_ROWS), dim3(256), PfGeom<DQ, DV>::SMEM, st, pdl, a, tokens);
+}
+
+}  // namespace
+
+cudaError_t launch_latent_prefill(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
+    if (!latent_prefill_fits(a.s) || !a.cache_bf16 || !a.act_bf16) return cudaErrorInvalidValue;
+    const uint32_t q = a.s.dim + a.s.rot, v = a.s.vdim;
+    if (q <= 64 && v <= 64) return prefill_inst<64, 64>(a, tokens, st, pdl);
+    if (q <= 128 && v <= 128) return prefill_inst<128, 128>(a, tokens, st, pdl);
+    if (q <= 192 && v <= 128) return prefill_inst<192, 128>(a, tokens, st, pdl);
+    return prefill_inst<256, 256>(a, tokens, st, pdl);
+}
+
+}  // namespace alice

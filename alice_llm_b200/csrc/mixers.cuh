@@ -45,7 +45,8 @@ struct DeltaArgs {
     const float* y = nullptr;         // projections [t][ldy]: q | k | v | b | ...
     uint32_t ldy = 0;
     const float* conv_w = nullptr;    // [conv_cols][taps]
-    float* conv_state = nullptr;      // [taps - 1][conv_cols], oldest first
+    float* conv_state = nullptr;      // two of [taps - 1][conv_cols], oldest first: the one of a position's parity holds the inputs before it
+    const int* pos = nullptr;
     float* state = nullptr;           // [heads][vp][dp]
     float *qn = nullptr, *kn = nullptr, *kq = nullptr, *v = nullptr, *beta = nullptr;   // prepared inputs of the recurrence
     const float* g = nullptr;         // decays [t][heads][dp]
@@ -61,6 +62,15 @@ struct DeltaArgs {
 cudaError_t launch_delta_prepare(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 cudaError_t launch_delta_scan(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 cudaError_t launch_delta_out(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
+// All of it for one token in one launch, the decay and gate projections included; f32 result.
+struct DeltaStepArgs {
+    DeltaArgs d;
+    DenseMat a2, g2;
+    uint32_t off_a = 0, off_g = 0;    // columns of their low-rank inputs in y
+    const float *a_log = nullptr, *dt_bias = nullptr;
+};
+inline bool delta_step_fits(const DeltaShape& s) { return s.vp <= 256; }
+cudaError_t launch_delta_step(const DeltaStepArgs& a, cudaStream_t st, bool pdl);
 
 // ---- latent.cu: attention over a cached latent ---------------------------------------------------
 struct LatentShape {
@@ -83,13 +93,21 @@ struct LatentArgs {
     bool cache_bf16 = false;
     void* cqn = nullptr;              // normalised query latent [t][qp]
     bool act_bf16 = false;            // type of cqn and out
+    bool append = false;              // launch_latent_absorb also puts the token's row into the cache
     const float* q = nullptr;         // [t][heads * (dim + rot)]
     float* ql = nullptr;              // [t][heads][cp + rp]: queries taken into the latent space, rotated part
     float* part = nullptr;            // [t][splits][heads][cp + 2]
     uint32_t splits = 1;
     void* out = nullptr;              // [t][ldo]
     uint32_t ldo = 0;
+    // tiled prefill: keys and values of every cached token, made from the latent rows
+    const bf16 *k_all = nullptr, *v_all = nullptr;   // [ctx][heads * dim], [ctx][heads * vdim]
 };
+// Whether the tensor-core prefill covers these sizes (others take the latent-space path).
+inline bool latent_prefill_fits(const LatentShape& s) {
+    return s.dim % 8 == 0 && s.rot % 8 == 0 && s.vdim % 8 == 0 && s.dim + s.rot <= 256 && s.vdim <= 256;
+}
+cudaError_t launch_latent_prefill(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 cudaError_t launch_latent_norm(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 cudaError_t launch_latent_absorb(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 cudaError_t launch_latent_attn(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);

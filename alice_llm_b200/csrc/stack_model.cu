@@ -14,7 +14,9 @@ using namespace alice;
 
 namespace {
 
-constexpr uint32_t CHUNK_EXACT = 256, CHUNK = 2048, TRACE_TOKENS = 256, DECODE_SPLITS = 64;
+constexpr uint32_t CHUNK_SMALL = 256, CHUNK = 2048, TRACE_TOKENS = 256;
+constexpr uint32_t DECODE_SPLITS = 64;   // shares of the context one decoded token's attention is cut into
+constexpr uint32_t FEW_TOKENS = 4;       // up to here attention runs in the latent space also where the tiled form exists
 
 struct StackModel;
 
@@ -32,6 +34,7 @@ struct Scratch {
     // latent
     float *q = nullptr, *ql = nullptr, *part = nullptr;
     void* cqn = nullptr;
+    bf16 *k_all = nullptr, *v_all = nullptr;         // keys and values of the whole context (tiled prefill)
     // delta
     float *qn = nullptr, *kn = nullptr, *kq = nullptr, *v = nullptr, *beta = nullptr, *g = nullptr, *gate = nullptr, *o = nullptr;
     bf16* low = nullptr;                             // bf16 copy of the low-rank columns
@@ -71,7 +74,7 @@ struct StackModel final : alice_model {
     // bf16 activations: several tokens at once, unless everything is to be in 32 bits
     bool tiled_bf16(uint32_t tokens) const { return tokens > 1 && !exact(); }
     uint32_t runs() const { return cfg.num_layers + (cfg.loop_times ? (cfg.loop_times - 1) * (cfg.loop_stop - cfg.loop_start) : 0); }
-    uint32_t max_tokens() const override { return tracing ? TRACE_TOKENS : chunk; }
+    uint32_t max_tokens() const override { return tracing ? std::min(chunk, TRACE_TOKENS) : chunk; }
     int enqueue_step(uint32_t n, bool greedy_feed) override;
     int enqueue_rows(uint32_t n, const uint32_t* rows, uint32_t nrows, float* host_logits) override;
     int clear_state() override;
@@ -85,7 +88,7 @@ struct StackModel final : alice_model {
     int layer(uint32_t i, uint32_t n, uint32_t pass);
     int head(uint32_t n, const uint32_t* rows, uint32_t nrows, bool argmax);
     int product(GemmOp& op) {
-        MCU(launch_dense_gemm(op, e->status, e->stream, e->pdl));
+        MCU(launch_dense_gemm(op, e->num_sms, e->status, e->stream, e->pdl));
         return ALICE_OK;
     }
     // out[t] = W a[t] for every token: the row kernel for one token, a tiled product for more (EPI_STORE, f32 result)
@@ -108,6 +111,7 @@ struct LatentMixer final : Mixer {
     size_t cache_bytes = 0;
 
     bool recurrent() const override { return false; }
+    bool tiled(const StackModel* m) const { return !m->exact() && latent_prefill_fits(sh); }
     int clear(cudaStream_t st) override {
         for (void* c : cache) MCU(cudaMemsetAsync(c, 0, cache_bytes, st));
         return ALICE_OK;
@@ -120,10 +124,30 @@ struct LatentMixer final : Mixer {
         a.s = sh; a.y = s.y; a.ldy = s.ldy; a.q_norm = q_norm; a.kv_norm = kv_norm; a.sink = sink; a.freq = freq; a.eps = m->cfg.eps;
         a.uk = uk.w; a.uv = uv.w; a.pos = m->d_pos; a.cache = cache[pass]; a.cache_bf16 = !m->exact();
         a.cqn = s.cqn; a.act_bf16 = m->tiled_bf16(n); a.q = s.q; a.ql = s.ql; a.part = s.part; a.out = s.a; a.ldo = o.k;
-        a.splits = n == 1 ? DECODE_SPLITS : 1;
-        MCU(launch_latent_norm(a, n, st, pdl));
-        const int rc = m->project(n, s.cqn, sh.qp, uq, s.q, uq.n);
-        if (rc) return rc;
+        a.splits = n <= FEW_TOKENS ? DECODE_SPLITS / n : 1;
+        if (n == 1) {
+            RowsIn in;
+            in.x = s.y + sh.off_q; in.n_x = sh.q_rank; in.norm = NORM_RMS; in.norm_w = q_norm; in.eps = m->cfg.eps; in.w0 = uq; in.y0 = s.q;
+            MCU(launch_rows_in(in, m->e->num_sms, st, pdl));
+            a.append = true;
+        } else {
+            MCU(launch_latent_norm(a, n, st, pdl));
+            const int rc = m->project(n, s.cqn, sh.qp, uq, s.q, uq.n);
+            if (rc) return rc;
+        }
+        if (n > FEW_TOKENS && tiled(m)) {
+            const uint32_t ctx = m->pos + n;   // a tiled step is never replayed, so the host's position is the device's
+            GemmOp op;
+            op.tokens = ctx; op.a = cache[pass]; op.lda = sh.cp + sh.rp; op.a_bf16 = true; op.out_bf16 = true;
+            op.w = uk; op.out = s.k_all; op.ldo = uk.n;
+            int erc = m->product(op);
+            op.w = uv; op.out = s.v_all; op.ldo = uv.n;
+            if (!erc) erc = m->product(op);
+            if (erc) return erc;
+            a.k_all = s.k_all; a.v_all = s.v_all;
+            MCU(launch_latent_prefill(a, n, st, pdl));
+            return ALICE_OK;
+        }
         MCU(launch_latent_absorb(a, n, st, pdl));
         MCU(launch_latent_attn(a, n, st, pdl));
         MCU(launch_latent_out(a, n, st, pdl));
@@ -156,7 +180,13 @@ struct DeltaMixer final : Mixer {
         DeltaArgs a;
         a.s = sh; a.y = s.y; a.ldy = s.ldy; a.conv_w = conv; a.conv_state = states[pass].conv; a.state = states[pass].s;
         a.qn = s.qn; a.kn = s.kn; a.kq = s.kq; a.v = s.v; a.beta = s.beta; a.g = s.g; a.o = s.o; a.gate = s.gate; a.norm_w = norm; a.eps = m->cfg.eps;
-        a.out = s.a; a.ldo = o.k; a.out_bf16 = low;
+        a.out = s.a; a.ldo = o.k; a.out_bf16 = low; a.pos = m->d_pos;
+        if (n == 1 && delta_step_fits(sh)) {
+            DeltaStepArgs sa;
+            sa.d = a; sa.a2 = a2; sa.g2 = g2; sa.off_a = off_a; sa.off_g = off_g; sa.a_log = a_log; sa.dt_bias = dt_bias;
+            MCU(launch_delta_step(sa, st, pdl));
+            return ALICE_OK;
+        }
         const uint32_t ldl = in.n - off_a;
         const void* va = low ? (const void*)s.low : (const void*)(s.y + off_a);
         const void* vg = low ? (const void*)(s.low + (off_g - off_a)) : (const void*)(s.y + off_g);
@@ -382,7 +412,7 @@ void build_delta(Builder& b, const alice_stack_layer& L, uint32_t wp, uint32_t p
     mx.a_log = b.floats(L.a_log, L.heads, "a_log");
     mx.dt_bias = b.floats(L.dt_bias, (size_t)L.heads * s.dp, "dt_bias");
     mx.norm = b.floats(L.head_norm, L.vdim, "head_norm");
-    mx.conv_bytes = (size_t)std::max<uint32_t>(1, L.conv_taps - 1) * s.conv_cols * 4;
+    mx.conv_bytes = (size_t)2 * std::max<uint32_t>(1, L.conv_taps - 1) * s.conv_cols * 4;
     mx.state_bytes = (size_t)L.heads * s.vp * s.dp * 4;
     for (uint32_t p = 0; p < passes; p++) {
         DeltaMixer::State st{b.zeros<float>(mx.conv_bytes / 4), b.zeros<float>(mx.state_bytes / 4)};
@@ -394,7 +424,13 @@ void build_delta(Builder& b, const alice_stack_layer& L, uint32_t wp, uint32_t p
 void build_scratch(Builder& b) {
     StackModel* m = b.m;
     Scratch& s = m->s;
-    const uint32_t M = m->chunk;
+    // where attention of many tokens runs in the latent space, fewer of them go at once
+    bool small = m->exact();
+    for (const auto& L : m->layers)
+        if (const auto* x = dynamic_cast<const LatentMixer*>(L.mixer.get())) small |= !x->tiled(m);
+    m->chunk = std::min<uint32_t>(small ? CHUNK_SMALL : CHUNK, pad_to(m->max_seq, 64));
+    const uint32_t M = m->chunk, ML = small ? M : std::min(M, FEW_TOKENS);
+    uint32_t k_all = 0, v_all = 0;
     uint32_t ldy = 0, ldf = 0, lda = 0, q = 0, ql = 0, part = 0, qp = 0, kd = 0, kh = 0, v = 0, h = 0, g = 0, o = 0, low = 0;
     for (const auto& L : m->layers) {
         ldy = std::max(ldy, L.mixer->in.n);
@@ -402,6 +438,7 @@ void build_scratch(Builder& b) {
         ldf = std::max(ldf, L.down.k);
         if (const auto* x = dynamic_cast<const LatentMixer*>(L.mixer.get())) {
             const LatentShape& z = x->sh;
+            if (x->tiled(m)) { k_all = std::max(k_all, x->uk.n); v_all = std::max(v_all, x->uv.n); }
             q = std::max(q, x->uq.n); qp = std::max(qp, z.qp);
             ql = std::max(ql, z.heads * (z.cp + z.rp)); part = std::max(part, z.heads * (z.cp + 2));
         } else if (const auto* x = dynamic_cast<const DeltaMixer*>(L.mixer.get())) {
@@ -418,8 +455,10 @@ void build_scratch(Builder& b) {
     s.a = b.zeros<float>((size_t)M * lda);     // heads * vdim columns and the padding of each mixer's own stride
     s.q = b.zeros<float>((size_t)M * q);
     s.cqn = b.zeros<float>((size_t)M * qp);
-    s.ql = b.zeros<float>((size_t)M * ql);
-    s.part = b.zeros<float>((size_t)std::max(M, DECODE_SPLITS) * part);
+    s.ql = b.zeros<float>((size_t)ML * ql);
+    s.part = b.zeros<float>((size_t)std::max(ML, DECODE_SPLITS) * part);
+    s.k_all = b.zeros<bf16>((size_t)m->max_seq * k_all);
+    s.v_all = b.zeros<bf16>((size_t)m->max_seq * v_all);
     s.qn = b.zeros<float>((size_t)M * kd); s.kn = b.zeros<float>((size_t)M * kd); s.kq = b.zeros<float>((size_t)M * kh);
     s.v = b.zeros<float>((size_t)M * v); s.beta = b.zeros<float>((size_t)M * h); s.g = b.zeros<float>((size_t)M * g);
     s.gate = b.zeros<float>((size_t)M * o); s.o = b.zeros<float>((size_t)M * o);
@@ -448,7 +487,6 @@ int32_t alice_stack_create(alice_engine* e, const alice_stack_config* cfg, const
     MCU(cudaSetDevice(e->device));
     auto* m = new StackModel();
     m->e = e; m->cfg = c; m->vocab = c.vocab_size; m->max_seq = c.max_seq_len;
-    m->chunk = std::min<uint32_t>(c.exact ? CHUNK_EXACT : CHUNK, pad_to(c.max_seq_len, 64));
     alice_engine_retain(e);
     Builder b{m};
     const uint32_t wp = P(c.width);

@@ -819,6 +819,154 @@ def run_ours(args, rank, world, local_rank):
             pass
 
 
+# ---- layer-stack models (--stack) -------------------------------------------------------------------------
+# width, feed-forward, heads and layer count of each size; half of the layers are latent attention, half delta rule. The
+# compared Llama has the same width, feed-forward, heads, layer count and vocabulary, in the Q4_K_M mix.
+STACK_SIZES = {
+    "w2048": dict(width=2048, ff=8192, heads=16, q_rank=768, kv_rank=512, rank=128, layers=8, vocab=32000),
+    "w4096": dict(width=4096, ff=14336, heads=32, q_rank=1536, kv_rank=512, rank=128, layers=8, vocab=32000),
+}
+
+
+def stack_config(z):
+    latent = {"type": "latent_attention", "mlp": {"kind": "dense", "ff": z["ff"]},
+              "mixer": dict(heads=z["heads"], dim=128, rot_dim=64, vdim=128, q_rank=z["q_rank"], kv_rank=z["kv_rank"], scale=192 ** -0.5,
+                            rot=dict(base=10000.0, dims=64))}
+    delta = {"type": "channel_delta", "mlp": {"kind": "dense", "ff": z["ff"]},
+             "mixer": dict(heads=z["heads"], kv_heads=z["heads"], dim=128, vdim=128, conv=4)}
+    return {"architecture": "Zamitar", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "layers": [delta if i % 2 == 0 else latent for i in range(z["layers"])], "loop": None}
+
+
+def build_stack(eng, z, max_seq_len, seed=0):
+    """-> (GpuModel, weight bytes one token reads, matrix FLOPs per token). Weights drawn on the device."""
+    import torch
+    from alice_llm_b200 import stack
+    from alice_llm_b200.gpu import GpuModel, GpuQuantType
+    dev = torch.device("cuda", eng.device)
+    gen = torch.Generator(device=dev)
+    gen.manual_seed(seed)
+    rng = np.random.default_rng(seed)
+    cfg = stack.StackConfig(stack_config(z), max_seq_len)
+    keep, nbytes = [], 0
+
+    def mat(rows, cols):
+        nonlocal nbytes
+        t = (torch.randn(rows, cols, device=dev, generator=gen) * cols ** -0.5).to(torch.bfloat16)
+        keep.append(t)
+        nbytes += rows * cols * 2
+        return eng.weights_from_device(t.data_ptr(), rows * cols * 2, rows, cols, GpuQuantType.BF16)
+
+    one = lambda n: (1.0 + 0.02 * rng.standard_normal(n)).astype(np.float32)
+    small = lambda *n: (0.1 * rng.standard_normal(n)).astype(np.float32)
+    packed = []
+    for L in cfg.layers:
+        L.decay_rank = L.gate_rank = z["rank"] if L.kind == stack.MIX_DELTA else 0
+        mats = {n: mat(*shape) for n, shape in L.packed_shapes(cfg.width).items()}
+        w, ff = cfg.width, stack.pad(L.ff)
+        vecs = dict(norm=one(w), ls1=small(w), ls2=small(w), gate_bias=small(ff), up_bias=small(ff), down_bias=small(w))
+        if L.kind == stack.MIX_LATENT:
+            vecs.update(q_norm=one(L.q_rank), kv_norm=one(L.kv_rank), sink=small(L.heads))
+        else:
+            vecs.update(conv=small(sum(stack.pad(r) for _, r in L.input_segments()[:3]), L.conv_taps), a_log=small(L.heads),
+                        dt_bias=small(L.heads * stack.delta_dim(L.dim)) - 2.0, head_norm=one(L.vdim))
+        packed.append((mats, vecs))
+    embed = mat(cfg.vocab_size, stack.pad(cfg.width))
+    h, more = stack.create(eng, cfg, packed, embed, one(cfg.width), None, False)
+    return GpuModel(eng, h, cfg, [keep, more]), nbytes, nbytes      # two FLOPs per weight = its two bytes
+
+
+def llama_like(z, context):
+    from alice_llm_b200 import synth
+    mix = dict(q=synth.Q4_K, k=synth.Q4_K, v=synth.Q6_K, o=synth.Q4_K, gate=synth.Q4_K, up=synth.Q4_K, down=synth.Q6_K, output=synth.Q6_K)
+    return dict(num_layers=z["layers"], hidden_dim=z["width"], intermediate_dim=z["ff"], num_heads=z["heads"], num_kv_heads=z["heads"] // 4, head_dim=128,
+                vocab_size=z["vocab"], rope_theta=500000.0, eps=1e-5, context=context, mix=mix)
+
+
+def run_stack(args):
+    """Prefill and greedy decode of layer-stack models beside a quantized Llama of the same size, on one GPU."""
+    import torch
+    from alice_llm_b200.gpu import GpuEngine
+    torch.cuda.set_device(0)
+    peak, source = measured_peak()
+    tflops = 1590.0
+    try:
+        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+            tflops = float(json.load(f)["bf16_tflops"])
+    except Exception:
+        pass
+    eng = GpuEngine(0)
+    stream = torch.cuda.Stream()
+    torch.cuda.set_stream(stream)
+    eng.set_stream(stream.cuda_stream)
+    ctx, tokens = args.stack_context, 64
+
+    def timed(fn, n=1):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record(stream)
+        for _ in range(n):
+            fn()
+        e1.record(stream)
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / n
+
+    clocks = ClockSampler(0)
+    clocks.start()
+    out = {}
+    for name in args.stack.split(","):
+        z = STACK_SIZES[name]
+        rng = np.random.default_rng(1)
+        prompt = rng.integers(0, z["vocab"], ctx).astype(np.uint32)
+        gm, nbytes, flops = build_stack(eng, z, ctx + 256)
+
+        def prefill():
+            gm.reset()
+            gm.forward_rows(prompt, [ctx - 1])
+        for _ in range(3):
+            prefill()
+        pf = timed(prefill, 5)
+        gm.decode_greedy(1, 8)
+        dec = timed(lambda: gm.decode_greedy(1, tokens)) / tokens
+        half = z["layers"] // 2
+        extra = half * (2 * z["heads"] * 128 * 128 * 4) + half * ctx * (z["kv_rank"] + 64) * 2   # states read and written, latent rows read
+        # attention: scores and sums over half of the context on average, keys and values made from the latent once
+        aflops = half * (2 * z["heads"] * (192 + 128) * ctx / 2)
+        out[name] = {"prefill_tokens_per_s": round(ctx / pf * 1e3), "prefill_ms": round(pf, 3),
+                     "prefill_tflops": round((flops + aflops) * ctx / pf / 1e9, 1), "prefill_of_bf16_peak": round((flops + aflops) * ctx / pf / 1e9 / tflops, 3),
+                     "decode_ms_per_token": round(dec, 4), "decode_gbs": round((nbytes + extra) / dec / 1e6), "decode_of_hbm_peak": round((nbytes + extra) / dec / 1e6 / peak, 3)}
+        gm.free()
+        if not args.stack_only:
+            DECODE_CONFIGS["llama_" + name] = llama_like(z, ctx)
+            lm, info = build_model(eng, "llama_" + name)
+
+            def verify():
+                lm.set_position(ctx)
+                lm.forward_batch(prompt[:8])
+            for _ in range(3):
+                verify()
+            b8 = timed(verify, 20)
+            lm.set_position(ctx)
+            ld, _ = timed_decode(lm, ctx, tokens, stream, 1, None, None)
+            ld /= tokens
+            lb = info["weight_bytes_per_token"] + info["kv_bytes_per_token"]
+            out[name]["llama_q4km_equal_size"] = {
+                "prefill_tokens_per_s": round(8 / b8 * 1e3), "prefill_tflops": round(info_flops(z) * 8 / b8 / 1e9, 2),
+                "prefill_of_bf16_peak": round(info_flops(z) * 8 / b8 / 1e9 / tflops, 5), "decode_ms_per_token": round(ld, 4),
+                "decode_gbs": round(lb / ld / 1e6), "decode_of_hbm_peak": round(lb / ld / 1e6 / peak, 3)}
+            lm.free()
+        torch.cuda.empty_cache()
+    print(json.dumps({"metric": "layer_stack_prefill_and_decode", "context": ctx, "sizes": out, "hbm_gbs_peak": peak, "bf16_tflops_peak": tflops, "peak_source": source,
+                      "dtype": "bf16", "data": "synthetic (random weights)", "clocks": clocks.stop()}))
+
+
+def info_flops(z):
+    """Matrix FLOPs of one token of the compared Llama."""
+    kv = z["heads"] // 4 * 128
+    per = z["width"] * (2 * z["heads"] * 128 + 2 * kv) + 3 * z["width"] * z["ff"]
+    return 2 * (z["layers"] * per + z["vocab"] * z["width"])
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -833,7 +981,14 @@ def main():
     ap.add_argument("--decode", default="auto", help="auto | none | comma list of c3_8b_q4km,c4_27b_q1_0,c5_70b_ternary")
     ap.add_argument("--decode-tokens", type=int, default=128)
     ap.add_argument("--decode-seconds", type=float, default=300.0, help="time limit of the whole-model section")
+    ap.add_argument("--stack", nargs="?", const=",".join(STACK_SIZES), default="",
+                    help="instead of the default workload: prefill and decode of layer-stack models beside a Llama of equal size (comma list of " +
+                         ", ".join(STACK_SIZES) + ")")
+    ap.add_argument("--stack-context", type=int, default=2048, help="prompt length of --stack")
+    ap.add_argument("--stack-only", action="store_true", help="--stack without the compared Llama")
     args = ap.parse_args()
+    if args.stack:
+        return run_stack(args)
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))
