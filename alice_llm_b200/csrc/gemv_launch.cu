@@ -4,6 +4,7 @@
 #include <cstdlib>
 
 #include "../../include/alice_cuda.h"
+#include "dense.cuh"
 #include "formats.cuh"
 #include "gemv_mma.cuh"
 #include "gemv_kq_mma.cuh"
@@ -542,8 +543,25 @@ int launch_single(const GemvOp& op, const LaunchCfg& cfg) {
 
 }  // namespace
 
+// Dense bfloat16 rows (csrc/dense_rows.cu), plain products only: one launch per input vector.
+static int launch_dense_rows(const GemvOp& op, const LaunchCfg& cfg) {
+    const WeightDesc& w = *op.w[0];
+    if (op.nw != 1 || op.up || op.resid || op.npeers || op.norm_w || !op.x || !op.y) return ALICE_E_UNSUPPORTED;
+    if (w.cols % DENSE_PAD || w.cols > 55 * 1024 || ((uintptr_t)w.data & 15)) return ALICE_E_SHAPE;
+    for (uint32_t k = 0; k < op.batch; k++) {
+        RowsIn in;
+        in.x = op.x + (size_t)k * w.cols; in.n_x = w.cols;
+        in.w0.w = reinterpret_cast<const bf16*>(w.data); in.w0.n = w.rows; in.w0.k = w.cols;
+        in.y0 = op.y + op.y_off[0] + (size_t)k * (op.y_stride ? op.y_stride : w.rows);
+        in.argmax_key = op.argmax_key;
+        if (launch_rows_in(in, cfg.num_sms, cfg.stream, cfg.pdl) != cudaSuccess) return ALICE_E_CUDA;
+    }
+    return ALICE_OK;
+}
+
 int launch_stream_gemv_op(const GemvOp& op, const LaunchCfg& cfg) {
     if (op.batch == 0 || op.batch > (uint32_t)MAX_BATCH) return ALICE_E_SHAPE;
+    if (op.w[0] && op.w[0]->fmt == WF_BF16) return launch_dense_rows(op, cfg);
     if (op.batch == 1) return launch_single(op, cfg);
     if (op.argmax_key) return ALICE_E_INVALID;
     {   // K-quants with prepared Q8_K input: the int8 tensor-core kernel serves the whole batch in one pass over the weights
