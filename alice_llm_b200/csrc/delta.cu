@@ -249,25 +249,31 @@ __global__ void __launch_bounds__(256, 2) delta_step_kernel(const __grid_constan
     }
     if (tid < SCAN_COLS) v[tid] = c0 + tid < s.vdim ? conv_silu(d, before, 0, s.off_v + h * s.vdim + c0 + tid) : 0.0f;
     const float beta = sigmoid_f(d.y[s.off_b + h]), rate = expf(a.a_log[h]);
-    // low-rank projections: sixteen lanes a row
+    // low-rank projections: sixteen lanes a row, all rows of a lane group in flight at once
     const uint32_t hw = tid >> 4, hl = tid & 15;
-    for (uint32_t r = hw; r < DP + SCAN_COLS; r += 16) {
-        const bool decay = r < DP;
-        const uint32_t kk = decay ? a.a2.k : a.g2.k, row = decay ? r : r - DP;
-        const bf16* w = decay ? wa + (size_t)row * kk : wg + (size_t)min(row, vrows - 1) * kk;
-        const float* x = decay ? low : low + a.a2.k;
-        float acc = 0.0f;
-        for (uint32_t c = hl * 8; c < kk; c += 128) {
-            const uint4 u = __ldg(reinterpret_cast<const uint4*>(w + c));
-            const float2 e0 = bf2(u.x), e1 = bf2(u.y), e2 = bf2(u.z), e3 = bf2(u.w);
-            acc = fmaf(e0.x, x[c], acc); acc = fmaf(e0.y, x[c + 1], acc); acc = fmaf(e1.x, x[c + 2], acc); acc = fmaf(e1.y, x[c + 3], acc);
-            acc = fmaf(e2.x, x[c + 4], acc); acc = fmaf(e2.y, x[c + 5], acc); acc = fmaf(e3.x, x[c + 6], acc); acc = fmaf(e3.y, x[c + 7], acc);
-        }
+    constexpr int ND = DP / 16;
+    float acc[ND + 2];
 #pragma unroll
-        for (int o = 8; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+    for (int i = 0; i < ND + 2; i++) acc[i] = 0.0f;
+    for (uint32_t c = hl * 8; c < a.a2.k; c += 128) {
+        const float4 x0 = *reinterpret_cast<const float4*>(low + c), x1 = *reinterpret_cast<const float4*>(low + c + 4);
+#pragma unroll
+        for (int i = 0; i < ND; i++) acc[i] = dot8(__ldg(reinterpret_cast<const uint4*>(wa + (size_t)(hw + 16 * i) * a.a2.k + c)), x0, x1, acc[i]);
+    }
+    for (uint32_t c = hl * 8; c < a.g2.k; c += 128) {
+        const float4 x0 = *reinterpret_cast<const float4*>(low + a.a2.k + c), x1 = *reinterpret_cast<const float4*>(low + a.a2.k + c + 4);
+#pragma unroll
+        for (int i = 0; i < 2; i++)
+            acc[ND + i] = dot8(__ldg(reinterpret_cast<const uint4*>(wg + (size_t)min(hw + 16 * i, vrows - 1) * a.g2.k + c)), x0, x1, acc[ND + i]);
+    }
+#pragma unroll
+    for (int i = 0; i < ND + 2; i++) {
+#pragma unroll
+        for (int o = 8; o > 0; o >>= 1) acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], o);
+        const uint32_t row = hw + 16 * (i < ND ? i : i - ND);
         if (hl == 0) {
-            if (decay) g[row] = expf(-rate * softplus_f(acc + a.dt_bias[(size_t)h * DP + row]));
-            else gate[row] = sigmoid_f(acc);
+            if (i < ND) g[row] = expf(-rate * softplus_f(acc[i] + a.dt_bias[(size_t)h * DP + row]));
+            else gate[row] = sigmoid_f(acc[i]);
         }
     }
     __syncthreads();

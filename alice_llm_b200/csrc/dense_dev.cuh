@@ -8,6 +8,12 @@ namespace alice {
 __device__ __forceinline__ float sigmoid_f(float z) { return __fdiv_rn(1.0f, 1.0f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float2 bf2(uint32_t u) { return make_float2(__uint_as_float(u << 16), __uint_as_float(u & 0xffff0000u)); }
+__device__ __forceinline__ float dot8(uint4 v, float4 x0, float4 x1, float acc) {
+    const float2 a = bf2(v.x), b = bf2(v.y), d = bf2(v.z), e = bf2(v.w);
+    acc = fmaf(a.x, x0.x, acc); acc = fmaf(a.y, x0.y, acc); acc = fmaf(b.x, x0.z, acc); acc = fmaf(b.y, x0.w, acc);
+    acc = fmaf(d.x, x1.x, acc); acc = fmaf(d.y, x1.y, acc); acc = fmaf(e.x, x1.z, acc); acc = fmaf(e.y, x1.w, acc);
+    return acc;
+}
 __device__ __forceinline__ float warp_max(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));

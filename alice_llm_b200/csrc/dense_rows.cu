@@ -20,13 +20,7 @@ __device__ __forceinline__ void dot_rows(const bf16* const (&w)[R], const float*
         for (int r = 0; r < R; r++) v[r] = __ldg(reinterpret_cast<const uint4*>(w[r] + c));
         const float4 x0 = *reinterpret_cast<const float4*>(xs + c), x1 = *reinterpret_cast<const float4*>(xs + c + 4);
 #pragma unroll
-        for (int r = 0; r < R; r++) {
-            const float2 a = bf2(v[r].x), b = bf2(v[r].y), d = bf2(v[r].z), e = bf2(v[r].w);
-            acc[r] = fmaf(a.x, x0.x, acc[r]); acc[r] = fmaf(a.y, x0.y, acc[r]);
-            acc[r] = fmaf(b.x, x0.z, acc[r]); acc[r] = fmaf(b.y, x0.w, acc[r]);
-            acc[r] = fmaf(d.x, x1.x, acc[r]); acc[r] = fmaf(d.y, x1.y, acc[r]);
-            acc[r] = fmaf(e.x, x1.z, acc[r]); acc[r] = fmaf(e.y, x1.w, acc[r]);
-        }
+        for (int r = 0; r < R; r++) acc[r] = dot8(v[r], x0, x1, acc[r]);
     }
 #pragma unroll
     for (int r = 0; r < R; r++) acc[r] = warp_sum(acc[r]);
@@ -102,49 +96,75 @@ __global__ void __launch_bounds__(RT, 3) rows_in_kernel(const __grid_constant__ 
     if (op.argmax_key && lane == 0 && best) atomicMax(op.argmax_key, best);
 }
 
+// acc += W[.][lo, hi) x[lo, hi) of one matrix, lanes 8 columns apart
 template <int R>
-__global__ void __launch_bounds__(RT, 2) rows_out_kernel(const __grid_constant__ RowsOut op) {
+__device__ __forceinline__ void dot_range(const bf16* const (&w)[R], const float* xs, uint32_t lo, uint32_t hi, uint32_t lane, float (&acc)[R]) {
+#pragma unroll 4
+    for (uint32_t c = lo + lane * 8; c < hi; c += 256) {
+        uint4 v[R];
+#pragma unroll
+        for (int r = 0; r < R; r++) v[r] = __ldg(reinterpret_cast<const uint4*>(w[r] + c));
+        const float4 x0 = *reinterpret_cast<const float4*>(xs + c), x1 = *reinterpret_cast<const float4*>(xs + c + 4);
+#pragma unroll
+        for (int r = 0; r < R; r++) acc[r] = dot8(v[r], x0, x1, acc[r]);
+    }
+}
+
+// The CTA's warps share R rows: each takes an eighth of the columns of [W1 | W2] (so it reads only that part of the inputs),
+// scales its two partial sums and the parts meet in shared memory.
+template <int R>
+__global__ void __launch_bounds__(RT, 3) rows_out_kernel(const __grid_constant__ RowsOut op) {
     extern __shared__ __align__(16) float xs[];
-    const uint32_t lane = threadIdx.x & 31, warps = gridDim.x * RW;
-    const uint32_t n = op.w1.n, k1 = op.w1.k, k2 = op.w2.n ? op.w2.k : 0;
-    const uint32_t items = (n + R - 1) / R, w_id = blockIdx.x + (threadIdx.x >> 5) * gridDim.x;
+    __shared__ float part[2][RW][R];
+    const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const uint32_t n = op.w1.n, k1 = op.w1.k, k2 = op.w2.n ? op.w2.k : 0, k = k1 + k2;
+    const uint32_t items = (n + R - 1) / R;
+    const uint32_t lo = k / 64 * warp / RW * 64, hi = k / 64 * (warp + 1) / RW * 64;   // this warp's columns
+    const uint32_t lo1 = min(lo, k1), hi1 = min(hi, k1), lo2 = max(lo, k1) - k1, hi2 = max(hi, k1) - k1;
     const bf16 *u[R], *d[R];
     auto rows_of = [&](uint32_t item) {
 #pragma unroll
         for (int r = 0; r < R; r++) {
             const uint32_t row = min(item * R + r, n - 1);
             u[r] = op.w1.w + (size_t)row * k1;
-            d[r] = k2 ? op.w2.w + (size_t)row * k2 : nullptr;
+            d[r] = k2 ? op.w2.w + (size_t)row * k2 : u[r];
         }
     };
     pdl_launch_dependents();
-    if (w_id < items) {
-        rows_of(w_id);
+    for (uint32_t item = blockIdx.x; item < min(items, blockIdx.x + 2 * gridDim.x); item += gridDim.x) {
+        rows_of(item);
 #pragma unroll
         for (int r = 0; r < R; r++) {
-            prefetch_row(u[r], k1, lane);
-            if (k2) prefetch_row(d[r], k2, lane);
+            for (uint32_t c = lo1 + lane * 64; c < hi1; c += 2048) prefetch_l2(u[r] + c);
+            for (uint32_t c = lo2 + lane * 64; c < hi2; c += 2048) prefetch_l2(d[r] + c);
         }
     }
     pdl_wait();
-    for (uint32_t i = threadIdx.x * 4; i < k1; i += RT * 4) *reinterpret_cast<float4*>(xs + i) = __ldcg(reinterpret_cast<const float4*>(op.a + i));
-    for (uint32_t i = threadIdx.x * 4; i < k2; i += RT * 4) *reinterpret_cast<float4*>(xs + k1 + i) = __ldcg(reinterpret_cast<const float4*>(op.f + i));
-    __syncthreads();
-    for (uint32_t item = w_id; item < items; item += warps) {
+    for (uint32_t i = lo1 + lane * 4; i < hi1; i += 128) *reinterpret_cast<float4*>(xs + i) = __ldcg(reinterpret_cast<const float4*>(op.a + i));
+    for (uint32_t i = lo2 + lane * 4; i < hi2; i += 128) *reinterpret_cast<float4*>(xs + k1 + i) = __ldcg(reinterpret_cast<const float4*>(op.f + i));
+    __syncwarp();
+    uint32_t buf = 0;
+    for (uint32_t item = blockIdx.x; item < items; item += gridDim.x, buf ^= 1) {
         rows_of(item);
         float acc1[R], acc2[R];
-        dot_rows<R>(u, xs, k1, lane, acc1);
 #pragma unroll
-        for (int r = 0; r < R; r++) acc2[r] = 0.0f;
-        if (k2) dot_rows<R>(d, xs + k1, k2, lane, acc2);
+        for (int r = 0; r < R; r++) acc1[r] = acc2[r] = 0.0f;
+        dot_range<R>(u, xs, lo1, hi1, lane, acc1);
+        dot_range<R>(d, xs + k1, lo2, hi2, lane, acc2);
 #pragma unroll
         for (int r = 0; r < R; r++) {
-            const uint32_t row = item * R + r;
-            if (lane == (uint32_t)r && row < n) {
-                float v = op.s1[row] * acc1[r];
-                if (k2) v += op.s2[row] * (acc2[r] + op.b2[row]);
-                op.x[row] += v;
-            }
+            const uint32_t row = min(item * R + r, n - 1);
+            const float v = warp_sum(k2 ? op.s1[row] * acc1[r] + op.s2[row] * acc2[r] : op.s1[row] * acc1[r]);
+            if (lane == 0) part[buf][warp][r] = v;
+        }
+        __syncthreads();   // the other buffer's readers are done before anyone writes it again
+        const uint32_t row = item * R + threadIdx.x;
+        if (threadIdx.x < R && row < n) {
+            float v = 0.0f;
+#pragma unroll
+            for (int w = 0; w < RW; w++) v += part[buf][w][threadIdx.x];
+            if (k2) v += op.s2[row] * op.b2[row];
+            op.x[row] += v;
         }
     }
 }
@@ -164,7 +184,7 @@ cudaError_t rows_out_r(const RowsOut& op, int num_sms, cudaStream_t st, bool pdl
     cudaError_t err = allow_smem(rows_out_kernel<R>, 224 * 1024, done);
     if (err != cudaSuccess) return err;
     const uint32_t items = (op.w1.n + R - 1) / R;
-    const uint32_t grid = std::min<uint32_t>((items + RW - 1) / RW, (uint32_t)num_sms * 2);
+    const uint32_t grid = std::min<uint32_t>(items, (uint32_t)num_sms * 3);
     return launch_pdl(rows_out_kernel<R>, dim3(grid), dim3(RT), (size_t)(op.w1.k + (op.w2.n ? op.w2.k : 0)) * 4, st, pdl, op);
 }
 
@@ -180,8 +200,7 @@ cudaError_t launch_rows_in(const RowsIn& op, int num_sms, cudaStream_t st, bool 
 cudaError_t launch_rows_out(const RowsOut& op, int num_sms, cudaStream_t st, bool pdl) {
     if (!op.w1.n || op.w1.k % DENSE_PAD || (op.w2.n && (op.w2.n != op.w1.n || op.w2.k % DENSE_PAD))) return cudaErrorInvalidValue;
     if ((size_t)(op.w1.k + (op.w2.n ? op.w2.k : 0)) * 4 > 220 * 1024) return cudaErrorInvalidValue;
-    if (op.w1.n >= (uint32_t)num_sms * 16 * 2) return rows_out_r<2>(op, num_sms, st, pdl);
-    return rows_out_r<1>(op, num_sms, st, pdl);
+    return rows_out_r<2>(op, num_sms, st, pdl);
 }
 
 }  // namespace alice

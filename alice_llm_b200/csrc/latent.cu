@@ -219,27 +219,22 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const __grid_constant_
     }
 }
 
-// grid (heads, tokens): joins the splits and the sink, then value rows, output gate.
-template <class OT>
-__global__ void __launch_bounds__(256) latent_out_kernel(const __grid_constant__ LatentArgs a) {
-    extern __shared__ __align__(16) float sm[];   // latent [cp], then one weight per split
+// Joins the shares of the context and the sink: weighted latent of every head. grid (heads, cp / 64, tokens), 64 threads.
+__global__ void __launch_bounds__(64) latent_join_kernel(const __grid_constant__ LatentArgs a) {
+    extern __shared__ float wt[];   // one weight per share
     const LatentShape& s = a.s;
-    const uint32_t h = blockIdx.x, t = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    float* c = sm;
-    float* wt = sm + s.cp;
+    const uint32_t h = blockIdx.x, t = blockIdx.z, lane = threadIdx.x & 31, c = blockIdx.y * 64 + threadIdx.x;
     pdl_launch_dependents();
-    const bf16* uv = a.uv + (size_t)h * s.vdim * s.cp;
-    for (uint32_t i = threadIdx.x; i < s.vdim * (s.cp / 64); i += 256) prefetch_l2(uv + (size_t)i * 64);
     pdl_wait();
     const float* part = a.part + ((size_t)t * a.splits * s.heads + h) * (s.cp + 2);
     const size_t step = (size_t)s.heads * (s.cp + 2);
-    if (warp == 0) {
+    if (threadIdx.x < 32) {
         float top = a.sink[h];
         for (uint32_t i = lane; i < a.splits; i += 32) top = fmaxf(top, part[i * step + s.cp]);
         top = warp_max(top);
         float den = 0.0f;
         for (uint32_t i = lane; i < a.splits; i += 32) {
-            const float f = expf(part[i * step + s.cp] - top);   // an empty split left -inf
+            const float f = expf(part[i * step + s.cp] - top);   // an empty share left -inf
             wt[i] = f;
             den = fmaf(f, part[i * step + s.cp + 1], den);
         }
@@ -248,15 +243,30 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const __grid_constant__
         for (uint32_t i = lane; i < a.splits; i += 32) wt[i] *= inv;
     }
     __syncthreads();
-    for (uint32_t i = threadIdx.x; i < s.cp; i += 256) {
-        float v = 0.0f;
-        for (uint32_t k = 0; k < a.splits; k++) v = fmaf(wt[k], part[k * step + i], v);
-        c[i] = v;
-    }
+    float v = 0.0f;
+#pragma unroll 8
+    for (uint32_t k = 0; k < a.splits; k++)
+        if (wt[k] != 0.0f) v = fmaf(wt[k], part[k * step + c], v);   // an empty share holds no sums
+    a.mix[((size_t)t * s.heads + h) * s.cp + c] = v;
+}
+
+// Value rows of the weighted latent and the output gate. grid (heads, groups of 16 rows, tokens), 8 warps of two rows.
+template <class OT>
+__global__ void __launch_bounds__(256) latent_value_kernel(const __grid_constant__ LatentArgs a) {
+    extern __shared__ __align__(16) float c[];   // latent [cp]
+    const LatentShape& s = a.s;
+    const uint32_t h = blockIdx.x, t = blockIdx.z, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, r0 = blockIdx.y * 16 + warp;
+    const bf16* uv = a.uv + (size_t)h * s.vdim * s.cp;
+    pdl_launch_dependents();
+    for (uint32_t r = r0; r < min(s.vdim, r0 + 16); r += 8)
+        for (uint32_t i = lane * 64; i < s.cp; i += 32 * 64) prefetch_l2(uv + (size_t)r * s.cp + i);
+    pdl_wait();
+    const float* mix = a.mix + ((size_t)t * s.heads + h) * s.cp;
+    for (uint32_t i = threadIdx.x; i < s.cp; i += 256) c[i] = mix[i];
     __syncthreads();
     const float* gate = a.y + (size_t)t * a.ldy + s.off_g + (size_t)h * s.vdim;
     OT* out = static_cast<OT*>(a.out) + (size_t)t * a.ldo + (size_t)h * s.vdim;
-    for (uint32_t r = warp; r < s.vdim; r += 8) {
+    for (uint32_t r = r0; r < min(s.vdim, r0 + 16); r += 8) {
         float v = 0.0f;
         for (uint32_t i = lane * 8; i < s.cp; i += 256) {
             const uint4 w = __ldg(reinterpret_cast<const uint4*>(uv + (size_t)r * s.cp + i));
@@ -267,7 +277,7 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const __grid_constant__
         v = warp_sum(v);
         if (lane == 0) put(out + r, v * sigmoid_f(gate[r]));
     }
-    if (h + 1 == s.heads)   // padding up to the stride
+    if (h + 1 == s.heads && blockIdx.y == 0)   // padding up to the stride
         for (uint32_t i = s.vdim + threadIdx.x; i < a.ldo - h * s.vdim; i += 256) put(out + i, 0.0f);
 }
 
@@ -303,12 +313,15 @@ cudaError_t launch_latent_absorb(const LatentArgs& a, uint32_t tokens, cudaStrea
                         : launch_pdl(latent_absorb_kernel<float>, grid, dim3(256), smem, st, pdl, a);
 }
 cudaError_t launch_latent_attn(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
+    if (a.cache_bf16 && latent_decode_fits(a.s)) return launch_latent_decode(a, tokens, st, pdl);
     return a.cache_bf16 ? attn_type<bf16>(a, tokens, st, pdl) : attn_type<float>(a, tokens, st, pdl);
 }
 cudaError_t launch_latent_out(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
-    const size_t smem = (size_t)(a.s.cp + a.splits) * 4;
-    return a.act_bf16 ? launch_pdl(latent_out_kernel<bf16>, dim3(a.s.heads, tokens), dim3(256), smem, st, pdl, a)
-                      : launch_pdl(latent_out_kernel<float>, dim3(a.s.heads, tokens), dim3(256), smem, st, pdl, a);
+    const cudaError_t err = launch_pdl(latent_join_kernel, dim3(a.s.heads, a.s.cp / 64, tokens), dim3(64), (size_t)a.splits * 4, st, pdl, a);
+    if (err != cudaSuccess) return err;
+    const dim3 grid(a.s.heads, (a.s.vdim + 15) / 16, tokens);
+    return a.act_bf16 ? launch_pdl(latent_value_kernel<bf16>, grid, dim3(256), (size_t)a.s.cp * 4, st, pdl, a)
+                      : launch_pdl(latent_value_kernel<float>, grid, dim3(256), (size_t)a.s.cp * 4, st, pdl, a);
 }
 
 }  // namespace alice

@@ -98,6 +98,7 @@ struct LatentArgs {
     float* ql = nullptr;              // [t][heads][cp + rp]: queries taken into the latent space, rotated part
     float* part = nullptr;            // [t][splits][heads][cp + 2]
     uint32_t splits = 1;
+    float* mix = nullptr;             // [t][heads][cp]: weighted latent
     void* out = nullptr;              // [t][ldo]
     uint32_t ldo = 0;
     // tiled prefill: keys and values of every cached token, made from the latent rows
@@ -110,6 +111,9 @@ inline bool latent_prefill_fits(const LatentShape& s) {
 cudaError_t launch_latent_prefill(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 cudaError_t launch_latent_norm(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 cudaError_t launch_latent_absorb(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
+// scores and weighted sums of queries in the latent space (launch_latent_decode: its tensor-core form, bf16 cache)
+bool latent_decode_fits(const LatentShape& s);
+cudaError_t launch_latent_decode(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 cudaError_t launch_latent_attn(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 cudaError_t launch_latent_out(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 

@@ -32,7 +32,7 @@ struct Scratch {
     float *x = nullptr, *y = nullptr;
     void *h = nullptr, *f = nullptr, *a = nullptr;   // activations: f32, or bf16 in tiled products
     // latent
-    float *q = nullptr, *ql = nullptr, *part = nullptr;
+    float *q = nullptr, *ql = nullptr, *part = nullptr, *mix = nullptr;
     void* cqn = nullptr;
     bf16 *k_all = nullptr, *v_all = nullptr;         // keys and values of the whole context (tiled prefill)
     // delta
@@ -123,7 +123,7 @@ struct LatentMixer final : Mixer {
         LatentArgs a;
         a.s = sh; a.y = s.y; a.ldy = s.ldy; a.q_norm = q_norm; a.kv_norm = kv_norm; a.sink = sink; a.freq = freq; a.eps = m->cfg.eps;
         a.uk = uk.w; a.uv = uv.w; a.pos = m->d_pos; a.cache = cache[pass]; a.cache_bf16 = !m->exact();
-        a.cqn = s.cqn; a.act_bf16 = m->tiled_bf16(n); a.q = s.q; a.ql = s.ql; a.part = s.part; a.out = s.a; a.ldo = o.k;
+        a.cqn = s.cqn; a.act_bf16 = m->tiled_bf16(n); a.q = s.q; a.ql = s.ql; a.part = s.part; a.mix = s.mix; a.out = s.a; a.ldo = o.k;
         a.splits = n <= FEW_TOKENS ? DECODE_SPLITS / n : 1;
         if (n == 1) {
             RowsIn in;
@@ -431,7 +431,7 @@ void build_scratch(Builder& b) {
     m->chunk = std::min<uint32_t>(small ? CHUNK_SMALL : CHUNK, pad_to(m->max_seq, 64));
     const uint32_t M = m->chunk, ML = small ? M : std::min(M, FEW_TOKENS);
     uint32_t k_all = 0, v_all = 0;
-    uint32_t ldy = 0, ldf = 0, lda = 0, q = 0, ql = 0, part = 0, qp = 0, kd = 0, kh = 0, v = 0, h = 0, g = 0, o = 0, low = 0;
+    uint32_t ldy = 0, ldf = 0, lda = 0, q = 0, ql = 0, part = 0, mix = 0, qp = 0, kd = 0, kh = 0, v = 0, h = 0, g = 0, o = 0, low = 0;
     for (const auto& L : m->layers) {
         ldy = std::max(ldy, L.mixer->in.n);
         lda = std::max(lda, L.mixer->o.k);
@@ -440,7 +440,7 @@ void build_scratch(Builder& b) {
             const LatentShape& z = x->sh;
             if (x->tiled(m)) { k_all = std::max(k_all, x->uk.n); v_all = std::max(v_all, x->uv.n); }
             q = std::max(q, x->uq.n); qp = std::max(qp, z.qp);
-            ql = std::max(ql, z.heads * (z.cp + z.rp)); part = std::max(part, z.heads * (z.cp + 2));
+            ql = std::max(ql, z.heads * (z.cp + z.rp)); part = std::max(part, z.heads * (z.cp + 2)); mix = std::max(mix, z.heads * z.cp);
         } else if (const auto* x = dynamic_cast<const DeltaMixer*>(L.mixer.get())) {
             const DeltaShape& z = x->sh;
             kd = std::max(kd, z.kv_heads * z.dp); kh = std::max(kh, z.kv_heads); v = std::max(v, z.heads * z.vp); h = std::max(h, z.heads);
@@ -457,6 +457,7 @@ void build_scratch(Builder& b) {
     s.cqn = b.zeros<float>((size_t)M * qp);
     s.ql = b.zeros<float>((size_t)ML * ql);
     s.part = b.zeros<float>((size_t)std::max(ML, DECODE_SPLITS) * part);
+    s.mix = b.zeros<float>((size_t)ML * mix);
     s.k_all = b.zeros<bf16>((size_t)m->max_seq * k_all);
     s.v_all = b.zeros<bf16>((size_t)m->max_seq * v_all);
     s.qn = b.zeros<float>((size_t)M * kd); s.kn = b.zeros<float>((size_t)M * kd); s.kq = b.zeros<float>((size_t)M * kh);

@@ -6,7 +6,7 @@
 namespace alice {
 namespace {
 
-__global__ void __launch_bounds__(256) enter_kernel(const __grid_constant__ EnterArgs a) {
+__global__ void __launch_bounds__(1024) enter_kernel(const __grid_constant__ EnterArgs a) {
     pdl_launch_dependents();
     pdl_wait();
     const uint32_t t = blockIdx.x;
@@ -37,7 +37,7 @@ __global__ void __launch_bounds__(256) layer_norm_kernel(const __grid_constant__
 }  // namespace
 
 cudaError_t launch_enter(const EnterArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
-    return launch_pdl(enter_kernel, dim3(tokens), dim3(256), 0, st, pdl, a);
+    return launch_pdl(enter_kernel, dim3(tokens), dim3(a.n > 512 ? 1024 : 256), 0, st, pdl, a);
 }
 
 cudaError_t launch_layer_norm(const NormArgs& a, uint32_t rows, cudaStream_t st, bool pdl) {
