@@ -1,9 +1,12 @@
 // Delta rule with one decay per key channel. Per head, with a state S [dim][vdim] kept in f32:
 //   S <- g * S (rows);  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q.
-// A column of S never meets another one, so the recurrence runs column-parallel: eight lanes hold one column in registers
-// for as long as the tokens last. Both products of a token are taken from the decayed column in one pass,
-//   o = (gS)^T q + (k.q) u,   with k.q prepared per token,
-// which leaves one eight-lane reduction on the token-to-token path.
+// Columns of S never meet, so the state is cut by columns. Many tokens go in blocks of W = 16. With G_t the product of the
+// decays up to token t of a block, and P_st that of the decays after s up to t,
+//   A_ts = sum_d k_t k_s P_st (s < t),  B_ts = sum_d q_t k_s P_st (s <= t),
+// the block's writes solve (I + diag(beta) A) u = diag(beta) (v - S^T (G k)), and
+//   o_t = S^T (G_t q_t) + sum_s B_ts u_s,   S <- G_W S + sum_s (P_sW k_s) u_s^T.
+// A, B and the inverse depend on the projections only and are made for all blocks at once; what remains on the path from
+// block to block are three small products per block, in f32. Decays enter as products, never as quotients.
 #include "dense_dev.cuh"
 #include "mixers.cuh"
 
@@ -20,11 +23,11 @@ __device__ __forceinline__ float* conv_after(const DeltaArgs& a, uint32_t tokens
 // Convolution and silu of channel c at token t.
 __device__ __forceinline__ float conv_silu(const DeltaArgs& a, const float* before, int t, uint32_t c) {
     const int taps = (int)a.s.taps;
-    const float* w = a.conv_w + (size_t)c * taps;
+    const float* w = a.conv_w + c;
     float v = 0.0f;
     for (int j = 0; j < taps; j++) {
         const int s = t - (taps - 1 - j);
-        v = fmaf(w[j], s >= 0 ? a.y[(size_t)s * a.ldy + c] : before[(size_t)(taps - 1 + s) * a.s.conv_cols + c], v);
+        v = fmaf(w[(size_t)j * a.s.conv_cols], s >= 0 ? a.y[(size_t)s * a.ldy + c] : before[(size_t)(taps - 1 + s) * a.s.conv_cols + c], v);
     }
     return silu_ref(v);
 }
@@ -37,16 +40,15 @@ __device__ __forceinline__ void conv_keep(const DeltaArgs& a, const float* befor
     }
 }
 
-// One warp per (token, key head) or (token, value head).
+// One warp per (token, key head) or (token, value head); the warps of a CTA take consecutive tokens of one head, so the
+// convolution's window comes from L1.
 __global__ void __launch_bounds__(256) delta_prepare_kernel(const __grid_constant__ DeltaArgs a, uint32_t tokens) {
     pdl_launch_dependents();
     pdl_wait();
     const DeltaShape& s = a.s;
-    const uint32_t lane = threadIdx.x & 31, per = s.kv_heads + s.heads;
-    const size_t task = (size_t)blockIdx.x * 8 + (threadIdx.x >> 5);
-    if (task >= (size_t)tokens * per) return;
+    const uint32_t lane = threadIdx.x & 31, t = blockIdx.x * 8 + (threadIdx.x >> 5), i = blockIdx.y;
+    if (t >= tokens) return;
     const float* before = conv_before(a);
-    const uint32_t t = (uint32_t)(task / per), i = (uint32_t)(task % per);
     if (i < s.kv_heads) {
         constexpr int N = DELTA_MAX_DIM / 32;
         float q[N], k[N], sq = 0.0f, sk = 0.0f;
@@ -62,17 +64,12 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const __grid_constan
         }
         sq = warp_sum(sq); sk = warp_sum(sk);
         const float iq = __frcp_rn(__fsqrt_rn(sq + 1e-6f)) * __frcp_rn(__fsqrt_rn((float)s.dim)), ik = __frcp_rn(__fsqrt_rn(sk + 1e-6f));
-        float dot = 0.0f;
         const size_t o = ((size_t)t * s.kv_heads + i) * s.dp;
 #pragma unroll
         for (int j = 0; j < N; j++) {
             const uint32_t d = lane + 32 * j;
-            q[j] *= iq; k[j] *= ik;
-            dot = fmaf(q[j], k[j], dot);
-            if (d < s.dp) { a.qn[o + d] = q[j]; a.kn[o + d] = k[j]; }
+            if (d < s.dp) { a.qn[o + d] = q[j] * iq; a.kn[o + d] = k[j] * ik; }
         }
-        dot = warp_sum(dot);
-        if (lane == 0) a.kq[(size_t)t * s.kv_heads + i] = dot;
     } else {
         const uint32_t h = i - s.kv_heads;
         const size_t o = ((size_t)t * s.heads + h) * s.vp;
@@ -90,100 +87,271 @@ __global__ void __launch_bounds__(256) conv_tail_kernel(const __grid_constant__ 
     if (c < a.s.conv_cols) conv_keep(a, conv_before(a), conv_after(a, tokens), tokens, c);
 }
 
-constexpr int SCAN_COLS = 32, SCAN_CHUNK = 8;   // columns per CTA, tokens per staged chunk
+constexpr int SCAN_COLS = 32;   // columns per CTA of a single token's step
+constexpr int W = 16;           // tokens per block
 
-__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+__device__ __forceinline__ void cp_async16(void* dst, const void* src, bool ok = true) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(ok ? 16u : 0u) : "memory");
 }
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N>
 __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// E elements of a column per lane: element e of lane l is dim (e / 4) * 32 + l * 4 + e % 4.
-template <int E>
-struct ScanStage {
-    float k[SCAN_CHUNK][8 * E], q[SCAN_CHUNK][8 * E], g[SCAN_CHUNK][8 * E], v[SCAN_CHUNK][SCAN_COLS];
-    float beta[SCAN_CHUNK], kq[SCAN_CHUNK];
-};
-
-template <int E>
-__device__ __forceinline__ void scan_fetch(ScanStage<E>& st, const DeltaArgs& a, uint32_t t0, uint32_t n, uint32_t h, uint32_t kh, uint32_t c0) {
+// grid (blocks, heads): inv = (I + diag(beta) A)^-1 diag(beta) and B of every block, [W][W] each. Sixteen lanes share a key s
+// and walk its decayed form along the later tokens.
+template <int DP>
+__global__ void __launch_bounds__(256) delta_pairs_kernel(const __grid_constant__ DeltaArgs a, uint32_t tokens) {
+    constexpr int ED = DP / 16;
+    extern __shared__ __align__(16) float sm[];
+    float *k = sm, *q = k + W * DP, *g = q + W * DP;
+    __shared__ float A[W][W + 1], B[W][W + 1], beta[W];
     const DeltaShape& s = a.s;
-    constexpr uint32_t P = 8 * E / 4;
-    for (uint32_t i = threadIdx.x; i < n * P; i += 256) {
-        const uint32_t j = i / P, d = i % P * 4;
-        const size_t ko = ((size_t)(t0 + j) * s.kv_heads + kh) * s.dp + d;
-        cp_async16(&st.k[j][d], a.kn + ko);
-        cp_async16(&st.q[j][d], a.qn + ko);
-        cp_async16(&st.g[j][d], a.g + ((size_t)(t0 + j) * s.heads + h) * s.dp + d);
+    const uint32_t tid = threadIdx.x, h = blockIdx.y, kh = h / (s.heads / s.kv_heads), t0 = blockIdx.x * W, n = min(tokens - t0, (uint32_t)W);
+    pdl_launch_dependents();
+    pdl_wait();
+    for (uint32_t i = tid; i < W * DP / 4; i += 256) {
+        const uint32_t t = i / (DP / 4), d = i % (DP / 4) * 4;
+        float4 kk = make_float4(0.f, 0.f, 0.f, 0.f), qq = kk, gg = kk;
+        if (t < n) {
+            const size_t ko = ((size_t)(t0 + t) * s.kv_heads + kh) * DP + d;
+            kk = *reinterpret_cast<const float4*>(a.kn + ko);
+            qq = *reinterpret_cast<const float4*>(a.qn + ko);
+            gg = *reinterpret_cast<const float4*>(a.g + ((size_t)(t0 + t) * s.heads + h) * DP + d);
+        }
+        *reinterpret_cast<float4*>(k + t * DP + d) = kk;
+        *reinterpret_cast<float4*>(q + t * DP + d) = qq;
+        *reinterpret_cast<float4*>(g + t * DP + d) = gg;
     }
-    for (uint32_t i = threadIdx.x; i < n * (SCAN_COLS / 4); i += 256) {
-        const uint32_t j = i / (SCAN_COLS / 4), d = i % (SCAN_COLS / 4) * 4;
-        cp_async16(&st.v[j][d], a.v + ((size_t)(t0 + j) * s.heads + h) * s.vp + c0 + d);
+    if (tid < W) beta[tid] = tid < n ? a.beta[(size_t)(t0 + tid) * s.heads + h] : 0.0f;
+    A[tid / W][tid % W] = 0.0f;
+    B[tid / W][tid % W] = 0.0f;
+    __syncthreads();
+    const uint32_t ks = tid >> 4, l = tid & 15;
+    float p[ED];
+#pragma unroll
+    for (int e = 0; e < ED; e++) p[e] = k[ks * DP + (e / 4) * 64 + l * 4 + e % 4];
+    for (uint32_t t = (tid >> 5) * 2; t < W; t++) {   // the first of the warp's two keys
+        float x = 0.0f, y = 0.0f;
+#pragma unroll
+        for (int e = 0; e < ED; e += 4) {
+            const uint32_t o = t * DP + e * 16 + l * 4;
+            const float4 kk = *reinterpret_cast<const float4*>(k + o), qq = *reinterpret_cast<const float4*>(q + o), gg = *reinterpret_cast<const float4*>(g + o);
+            if (t > ks) { p[e] *= gg.x; p[e + 1] *= gg.y; p[e + 2] *= gg.z; p[e + 3] *= gg.w; }
+            x = fmaf(p[e], kk.x, x); x = fmaf(p[e + 1], kk.y, x); x = fmaf(p[e + 2], kk.z, x); x = fmaf(p[e + 3], kk.w, x);
+            y = fmaf(p[e], qq.x, y); y = fmaf(p[e + 1], qq.y, y); y = fmaf(p[e + 2], qq.z, y); y = fmaf(p[e + 3], qq.w, y);
+        }
+#pragma unroll
+        for (int o = 8; o > 0; o >>= 1) {
+            x += __shfl_xor_sync(0xffffffffu, x, o);
+            y += __shfl_xor_sync(0xffffffffu, y, o);
+        }
+        if (l == 0 && t >= ks) {
+            if (t > ks) A[t][ks] = beta[t] * x;
+            B[t][ks] = y;
+        }
     }
-    if (threadIdx.x < n) {
-        st.beta[threadIdx.x] = a.beta[(size_t)(t0 + threadIdx.x) * s.heads + h];
-        st.kq[threadIdx.x] = a.kq[(size_t)(t0 + threadIdx.x) * s.kv_heads + kh];
+    __syncthreads();
+    const size_t o = ((size_t)blockIdx.x * s.heads + h) * W * W;
+    a.pair_b[o + tid] = B[tid / W][tid % W];
+    if (tid < W) {   // column tid of the inverse by forward substitution
+        float x[W];
+#pragma unroll
+        for (int t = 0; t < W; t++) {
+            float v = t == (int)tid ? beta[t] : 0.0f;
+#pragma unroll
+            for (int j = 0; j < t; j++) v = fmaf(-A[t][j], x[j], v);
+            x[t] = v;
+        }
+#pragma unroll
+        for (int t = 0; t < W; t++) a.pair_inv[o + t * W + tid] = x[t];
     }
 }
 
-template <int E>
-__global__ void __launch_bounds__(256) delta_scan_kernel(const __grid_constant__ DeltaArgs a, uint32_t tokens) {
-    extern __shared__ __align__(16) uint8_t smem[];
-    auto* stage = reinterpret_cast<ScanStage<E>*>(smem);   // two
-    __shared__ float os[SCAN_CHUNK][SCAN_COLS];
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+    float2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;"
+        : "=l"(*reinterpret_cast<unsigned long long*>(&d))
+        : "l"(*reinterpret_cast<const unsigned long long*>(&a)), "l"(*reinterpret_cast<const unsigned long long*>(&b)),
+          "l"(*reinterpret_cast<const unsigned long long*>(&c)));
+    return d;
+}
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) { return make_float2(a.x * b.x, a.y * b.y); }
+
+// Sums 64 values over the warp; lane l is left with those of index 2 l and 2 l + 1.
+__device__ __forceinline__ float2 reduce64(float (&v)[64], uint32_t lane) {
+#pragma unroll
+    for (int half = 32, o = 16; o > 0; half >>= 1, o >>= 1) {
+        const bool up = lane & o;
+#pragma unroll
+        for (int i = 0; i < half; i++) {
+            const float send = up ? v[i] : v[i + half], keep = up ? v[i + half] : v[i];
+            v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+        }
+    }
+    return make_float2(v[0], v[1]);
+}
+
+template <int DP, int NW>
+struct ScanStage {
+    float k[W][DP], q[W][DP], g[W][DP], v[W][4 * NW], inv[W][W], b[W][W];
+};
+template <int DP, int NW>
+struct ScanSmem {
+    ScanStage<DP, NW> st[2];
+    float end[DP];                 // decay over the whole block
+    float w[W][4 * NW];            // v - S^T (G k)
+    float y[W][4 * NW];            // S^T (G q)
+    float2 u[W][4 * NW];           // writes, twice each
+};
+
+template <int DP, int NW>
+__device__ __forceinline__ void scan_fetch(ScanStage<DP, NW>& st, const DeltaArgs& a, uint32_t t0, uint32_t n, uint32_t h, uint32_t kh, uint32_t c0) {
     const DeltaShape& s = a.s;
-    const uint32_t h = blockIdx.y, kh = h / (s.heads / s.kv_heads), c0 = blockIdx.x * SCAN_COLS;
-    const uint32_t lane = threadIdx.x & 31, l = lane & 7, col = (threadIdx.x >> 5) * 4 + (lane >> 3);
-    float* sp = a.state + ((size_t)h * s.vp + c0 + col) * s.dp + l * 4;
+    for (uint32_t i = threadIdx.x; i < W * DP / 4; i += NW * 32) {
+        const uint32_t j = i / (DP / 4), d = i % (DP / 4) * 4, t = t0 + min(j, n - 1);
+        const size_t ko = ((size_t)t * s.kv_heads + kh) * DP + d;
+        cp_async16(&st.k[j][d], a.kn + ko, j < n);
+        cp_async16(&st.q[j][d], a.qn + ko, j < n);
+        cp_async16(&st.g[j][d], a.g + ((size_t)t * s.heads + h) * DP + d, j < n);
+    }
+    for (uint32_t i = threadIdx.x; i < W * NW; i += NW * 32) {
+        const uint32_t j = i / NW, d = i % NW * 4, t = t0 + min(j, n - 1);
+        cp_async16(&st.v[j][d], a.v + ((size_t)t * s.heads + h) * s.vp + c0 + d, j < n);
+    }
+    const size_t o = ((size_t)(t0 / W) * s.heads + h) * W * W;
+    for (uint32_t i = threadIdx.x; i < W * W / 4; i += NW * 32) {
+        cp_async16(&st.inv[0][0] + i * 4, a.pair_inv + o + i * 4);
+        cp_async16(&st.b[0][0] + i * 4, a.pair_b + o + i * 4);
+    }
+}
+
+// grid (vp / (4 NW), heads), NW warps; a warp owns four columns of the state, a lane DP / 32 of their rows (register pairs).
+template <int DP, int NW>
+__global__ void __launch_bounds__(NW * 32) delta_scan_kernel(const __grid_constant__ DeltaArgs a, uint32_t tokens) {
+    constexpr int EL = DP / 32, NP = EL / 2, VEC = EL < 4 ? EL : 4, NC = EL / VEC, COLS = 4 * NW;   // rows per lane, in NC runs of VEC
+    extern __shared__ __align__(16) uint8_t raw[];
+    auto& sm = *reinterpret_cast<ScanSmem<DP, NW>*>(raw);
+    const DeltaShape& s = a.s;
+    const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, kh = h / (s.heads / s.kv_heads), c0 = blockIdx.x * COLS;
+    float* sp = a.state + ((size_t)h * s.vp + c0 + warp * 4) * DP + lane * VEC;
     pdl_launch_dependents();
     pdl_wait();
-    float S[E];
+    auto rows = [](const float* p, float2 (&r)[NP]) {   // this lane's rows of a [DP] vector
 #pragma unroll
-    for (int e = 0; e < E; e += 4) {
-        const float4 f = *reinterpret_cast<const float4*>(sp + e * 8);
-        S[e] = f.x; S[e + 1] = f.y; S[e + 2] = f.z; S[e + 3] = f.w;
-    }
-    scan_fetch<E>(stage[0], a, 0, min(tokens, (uint32_t)SCAN_CHUNK), h, kh, c0);
+        for (int i = 0; i < NC; i++) {
+            if constexpr (VEC == 4) {
+                const float4 f = *reinterpret_cast<const float4*>(p + i * 32 * VEC);
+                r[2 * i] = make_float2(f.x, f.y); r[2 * i + 1] = make_float2(f.z, f.w);
+            } else {
+                r[i] = *reinterpret_cast<const float2*>(p + i * 32 * VEC);
+            }
+        }
+    };
+    float2 S[4][NP];
+#pragma unroll
+    for (int c = 0; c < 4; c++) rows(sp + c * DP, S[c]);
+    const uint32_t nblk = (tokens + W - 1) / W;
+    scan_fetch<DP, NW>(sm.st[0], a, 0, min(tokens, (uint32_t)W), h, kh, c0);
     cp_commit();
-    for (uint32_t t0 = 0, b = 0; t0 < tokens; t0 += SCAN_CHUNK, b ^= 1) {
-        const uint32_t n = min(tokens - t0, (uint32_t)SCAN_CHUNK);
-        if (t0 + SCAN_CHUNK < tokens) scan_fetch<E>(stage[b ^ 1], a, t0 + SCAN_CHUNK, min(tokens - t0 - SCAN_CHUNK, (uint32_t)SCAN_CHUNK), h, kh, c0);
+    for (uint32_t blk = 0; blk < nblk; blk++) {
+        const uint32_t t0 = blk * W, n = min(tokens - t0, (uint32_t)W);
+        ScanStage<DP, NW>& st = sm.st[blk & 1];
+        if (blk + 1 < nblk) scan_fetch<DP, NW>(sm.st[(blk + 1) & 1], a, t0 + W, min(tokens - t0 - W, (uint32_t)W), h, kh, c0);
         cp_commit();
         cp_wait<1>();
         __syncthreads();
-        const ScanStage<E>& st = stage[b];
-        for (uint32_t j = 0; j < n; j++) {
-            float k[E], dk = 0.0f, dq = 0.0f, dk2 = 0.0f, dq2 = 0.0f;
+        // in place: k -> G k, q -> G q, g -> (decays after s) k_s; absent tokens have k = q = 0 and decay 1
+        for (uint32_t d = tid; d < DP; d += NW * 32) {
+            float k[W], g[W], p = 1.0f;
 #pragma unroll
-            for (int e = 0; e < E; e += 4) {
-                const float4 kk = *reinterpret_cast<const float4*>(&st.k[j][e * 8 + l * 4]), qq = *reinterpret_cast<const float4*>(&st.q[j][e * 8 + l * 4]),
-                             gg = *reinterpret_cast<const float4*>(&st.g[j][e * 8 + l * 4]);
-                S[e] *= gg.x; S[e + 1] *= gg.y; S[e + 2] *= gg.z; S[e + 3] *= gg.w;
-                dk = fmaf(S[e], kk.x, dk); dk2 = fmaf(S[e + 1], kk.y, dk2); dk = fmaf(S[e + 2], kk.z, dk); dk2 = fmaf(S[e + 3], kk.w, dk2);
-                dq = fmaf(S[e], qq.x, dq); dq2 = fmaf(S[e + 1], qq.y, dq2); dq = fmaf(S[e + 2], qq.z, dq); dq2 = fmaf(S[e + 3], qq.w, dq2);
-                k[e] = kk.x; k[e + 1] = kk.y; k[e + 2] = kk.z; k[e + 3] = kk.w;
+            for (int t = 0; t < W; t++) {
+                k[t] = st.k[t][d];
+                g[t] = (uint32_t)t < n ? st.g[t][d] : 1.0f;
+                p *= g[t];
+                st.k[t][d] = p * k[t];
+                st.q[t][d] *= p;
             }
-            dk += dk2; dq += dq2;
+            sm.end[d] = p;
+            p = 1.0f;
 #pragma unroll
-            for (int o = 4; o > 0; o >>= 1) {
-                dk += __shfl_xor_sync(0xffffffffu, dk, o);
-                dq += __shfl_xor_sync(0xffffffffu, dq, o);
+            for (int t = W - 1; t >= 0; t--) {
+                st.g[t][d] = p * k[t];
+                p *= g[t];
             }
-            const float u = st.beta[j] * (st.v[j][col] - dk);
-#pragma unroll
-            for (int e = 0; e < E; e++) S[e] = fmaf(k[e], u, S[e]);
-            if (l == 0) os[j][col] = fmaf(st.kq[j], u, dq);
         }
         __syncthreads();
-        for (uint32_t i = threadIdx.x; i < n * SCAN_COLS; i += 256) {
-            const uint32_t j = i / SCAN_COLS, c = i % SCAN_COLS;
-            if (c0 + c < s.vdim) a.o[((size_t)(t0 + j) * s.heads + h) * s.vdim + c0 + c] = os[j][c];
+#pragma unroll
+        for (int pass = 0; pass < 2; pass++) {   // S^T (G k), then S^T (G q)
+            float v[64];
+#pragma unroll
+            for (int t = 0; t < W; t++) {
+                float2 x[NP];
+                rows((pass ? st.q[t] : st.k[t]) + lane * VEC, x);
+#pragma unroll
+                for (int c = 0; c < 4; c++) {
+                    float2 acc = mul2(x[0], S[c][0]);
+#pragma unroll
+                    for (int i = 1; i < NP; i++) acc = fma2(x[i], S[c][i], acc);
+                    v[t * 4 + c] = acc.x + acc.y;
+                }
+            }
+            const float2 r = reduce64(v, lane);
+            const uint32_t t = lane / 2, c = warp * 4 + (lane & 1) * 2;
+            if (pass == 0) *reinterpret_cast<float2*>(&sm.w[t][c]) = make_float2(st.v[t][c] - r.x, st.v[t][c + 1] - r.y);
+            else *reinterpret_cast<float2*>(&sm.y[t][c]) = r;
+        }
+        __syncwarp();   // from here to the end of the block a warp works on its own columns only
+        {
+            const uint32_t c = warp * 4 + (lane & 3), t1 = lane >> 2, t2 = t1 + 8;   // two tokens of one column
+            float u1 = 0.0f, u2 = 0.0f;
+#pragma unroll
+            for (int j = 0; j < W; j++) {
+                const float w = sm.w[j][c];
+                u1 = fmaf(st.inv[t1][j], w, u1);
+                u2 = fmaf(st.inv[t2][j], w, u2);
+            }
+            sm.u[t1][c] = make_float2(u1, u1);
+            sm.u[t2][c] = make_float2(u2, u2);
+            __syncwarp();
+            float o1 = sm.y[t1][c], o2 = sm.y[t2][c];
+#pragma unroll
+            for (int j = 0; j < W; j++) {
+                const float u = sm.u[j][c].x;
+                o1 = fmaf(st.b[t1][j], u, o1);
+                o2 = fmaf(st.b[t2][j], u, o2);
+            }
+            if (c0 + c < s.vdim) {
+                if (t1 < n) a.o[((size_t)(t0 + t1) * s.heads + h) * s.vdim + c0 + c] = o1;
+                if (t2 < n) a.o[((size_t)(t0 + t2) * s.heads + h) * s.vdim + c0 + c] = o2;
+            }
+        }
+        float2 e[NP];
+        rows(sm.end + lane * VEC, e);
+#pragma unroll
+        for (int c = 0; c < 4; c++)
+#pragma unroll
+            for (int i = 0; i < NP; i++) S[c][i] = mul2(e[i], S[c][i]);
+#pragma unroll
+        for (int t = 0; t < W; t++) {
+            float2 x[NP];
+            rows(st.g[t] + lane * VEC, x);
+#pragma unroll
+            for (int c = 0; c < 4; c++) {
+                const float2 u = sm.u[t][warp * 4 + c];
+#pragma unroll
+                for (int i = 0; i < NP; i++) S[c][i] = fma2(x[i], u, S[c][i]);
+            }
         }
         __syncthreads();
     }
 #pragma unroll
-    for (int e = 0; e < E; e += 4) *reinterpret_cast<float4*>(sp + e * 8) = make_float4(S[e], S[e + 1], S[e + 2], S[e + 3]);
+    for (int c = 0; c < 4; c++)
+#pragma unroll
+        for (int i = 0; i < NC; i++) {
+            float* p = sp + c * DP + i * 32 * VEC;
+            if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(S[c][2 * i].x, S[c][2 * i].y, S[c][2 * i + 1].x, S[c][2 * i + 1].y);
+            else *reinterpret_cast<float2*>(p) = S[c][i];
+        }
 }
 
 // One warp per (token, head): root-mean-square norm over vdim, weight, gate.
@@ -230,6 +398,12 @@ __global__ void __launch_bounds__(256, 2) delta_step_kernel(const __grid_constan
     for (int e = 0; e < E; e += 4) if (l == 0) prefetch_l2(sp + e * 8);
     for (uint32_t i = tid; i < DP * (a.a2.k / 64); i += 256) prefetch_l2(wa + (size_t)i * 64);
     for (uint32_t i = tid; i < vrows * (a.g2.k / 64); i += 256) prefetch_l2(wg + (size_t)i * 64);
+    for (uint32_t j = 0; j < 3 * s.taps - 2; j++) {   // the taps, and both halves of the convolution state
+        const float* b = j < s.taps ? d.conv_w + (size_t)j * s.conv_cols : d.conv_state + (size_t)(j - s.taps) * s.conv_cols;
+        if (tid < s.dim && tid % 32 == 0) { prefetch_l2(b + s.off_q + kh * s.dim + tid); prefetch_l2(b + s.off_k + kh * s.dim + tid); }
+        if (tid == 0) prefetch_l2(b + s.off_v + h * s.vdim + c0);
+    }
+    if (tid < DP && tid % 32 == 0) prefetch_l2(a.dt_bias + (size_t)h * DP + tid);
     pdl_wait();
     const float* before = conv_before(d);
     float S[E];
@@ -342,30 +516,39 @@ cudaError_t step_e(const DeltaStepArgs& a, cudaStream_t st, bool pdl) {
     return cudaLaunchKernelEx(&lc, delta_step_kernel<E>, a);
 }
 
-template <int E>
-cudaError_t scan_e(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
+template <int DP, int NW>
+cudaError_t scan_inst(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
     static bool done[64] = {};
-    constexpr size_t smem = 2 * sizeof(ScanStage<E>);
-    const cudaError_t err = allow_smem(delta_scan_kernel<E>, smem, done);
+    constexpr size_t smem = sizeof(ScanSmem<DP, NW>);
+    const cudaError_t err = allow_smem(delta_scan_kernel<DP, NW>, smem, done);
     if (err != cudaSuccess) return err;
-    return launch_pdl(delta_scan_kernel<E>, dim3(a.s.vp / SCAN_COLS, a.s.heads), dim3(256), smem, st, pdl, a, tokens);
+    return launch_pdl(delta_scan_kernel<DP, NW>, dim3(a.s.vp / (4 * NW), a.s.heads), dim3(NW * 32), smem, st, pdl, a, tokens);
+}
+template <int DP>
+cudaError_t scan_dim(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
+    static bool done[64] = {};
+    constexpr size_t smem = (size_t)3 * W * DP * sizeof(float);
+    cudaError_t err = allow_smem(delta_pairs_kernel<DP>, smem, done);
+    if (err != cudaSuccess) return err;
+    err = launch_pdl(delta_pairs_kernel<DP>, dim3((tokens + W - 1) / W, a.s.heads), dim3(256), smem, st, pdl, a, tokens);
+    if (err != cudaSuccess) return err;
+    // few columns: narrower CTAs, so that more SMs have one
+    return a.s.heads * (a.s.vp / 32) < 100 ? scan_inst<DP, 4>(a, tokens, st, pdl) : scan_inst<DP, 8>(a, tokens, st, pdl);
 }
 
 }  // namespace
 
 cudaError_t launch_delta_prepare(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
-    const size_t tasks = (size_t)tokens * (a.s.kv_heads + a.s.heads);
-    cudaError_t err = launch_pdl(delta_prepare_kernel, dim3((unsigned)((tasks + 7) / 8)), dim3(256), 0, st, pdl, a, tokens);
+    cudaError_t err = launch_pdl(delta_prepare_kernel, dim3((tokens + 7) / 8, a.s.kv_heads + a.s.heads), dim3(256), 0, st, pdl, a, tokens);
     if (err != cudaSuccess || a.s.taps <= 1) return err;
     return launch_pdl(conv_tail_kernel, dim3((a.s.conv_cols + 255) / 256), dim3(256), 0, st, pdl, a, tokens);
 }
 
 cudaError_t launch_delta_scan(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
     switch (a.s.dp) {
-        case 32: return scan_e<4>(a, tokens, st, pdl);
-        case 64: return scan_e<8>(a, tokens, st, pdl);
-        case 128: return scan_e<16>(a, tokens, st, pdl);
-        case 256: return scan_e<32>(a, tokens, st, pdl);
+        case 64: return scan_dim<64>(a, tokens, st, pdl);
+        case 128: return scan_dim<128>(a, tokens, st, pdl);
+        case 256: return scan_dim<256>(a, tokens, st, pdl);
         default: return cudaErrorInvalidValue;
     }
 }
@@ -373,7 +556,6 @@ cudaError_t launch_delta_scan(const DeltaArgs& a, uint32_t tokens, cudaStream_t 
 cudaError_t launch_delta_step(const DeltaStepArgs& a, cudaStream_t st, bool pdl) {
     if (!delta_step_fits(a.d.s) || (size_t)(a.a2.k + a.g2.k) * 4 > 32 * 1024) return cudaErrorInvalidValue;
     switch (a.d.s.dp) {
-        case 32: return step_e<4>(a, st, pdl);
         case 64: return step_e<8>(a, st, pdl);
         case 128: return step_e<16>(a, st, pdl);
         case 256: return step_e<32>(a, st, pdl);

@@ -1,5 +1,6 @@
 // One token against dense bfloat16 rows. A warp owns R consecutive rows at a time; every lane streams 16-byte pieces of
-// each (R * unroll loads in flight per lane), the input sits in shared memory as f32. The rows a warp starts with are
+// each (R times the unroll factor in flight; two CTAs of eight warps per SM are enough, which leaves room for the CTAs of the
+// next kernel), the input sits in shared memory as f32. The rows a warp starts with are
 // requested into L2 before the wait for the producing kernel, so under programmatic dependent launch the weights travel
 // while the input is still being made.
 #include "dense_dev.cuh"
@@ -57,7 +58,7 @@ __device__ __forceinline__ void item_rows(const RowsIn& op, uint32_t item, uint3
 }
 
 template <int R>
-__global__ void __launch_bounds__(RT, 3) rows_in_kernel(const __grid_constant__ RowsIn op) {
+__global__ void __launch_bounds__(RT, 2) rows_in_kernel(const __grid_constant__ RowsIn op) {
     extern __shared__ __align__(16) float xs[];
     __shared__ float red[RW];
     const uint32_t lane = threadIdx.x & 31, warps = gridDim.x * RW;
@@ -99,7 +100,7 @@ __global__ void __launch_bounds__(RT, 3) rows_in_kernel(const __grid_constant__ 
 // acc += W[.][lo, hi) x[lo, hi) of one matrix, lanes 8 columns apart
 template <int R>
 __device__ __forceinline__ void dot_range(const bf16* const (&w)[R], const float* xs, uint32_t lo, uint32_t hi, uint32_t lane, float (&acc)[R]) {
-#pragma unroll 4
+#pragma unroll 8
     for (uint32_t c = lo + lane * 8; c < hi; c += 256) {
         uint4 v[R];
 #pragma unroll
@@ -113,7 +114,7 @@ __device__ __forceinline__ void dot_range(const bf16* const (&w)[R], const float
 // The CTA's warps share R rows: each takes an eighth of the columns of [W1 | W2] (so it reads only that part of the inputs),
 // scales its two partial sums and the parts meet in shared memory.
 template <int R>
-__global__ void __launch_bounds__(RT, 3) rows_out_kernel(const __grid_constant__ RowsOut op) {
+__global__ void __launch_bounds__(RT, 2) rows_out_kernel(const __grid_constant__ RowsOut op) {
     extern __shared__ __align__(16) float xs[];
     __shared__ float part[2][RW][R];
     const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -149,6 +150,16 @@ __global__ void __launch_bounds__(RT, 3) rows_out_kernel(const __grid_constant__
         float acc1[R], acc2[R];
 #pragma unroll
         for (int r = 0; r < R; r++) acc1[r] = acc2[r] = 0.0f;
+        if (item + 2 * gridDim.x < items) {   // the one after the next one sets out for L2
+            const bf16* nu = op.w1.w + (size_t)(item + 2 * gridDim.x) * R * k1;
+            const bf16* nd = op.w2.w + (size_t)(item + 2 * gridDim.x) * R * k2;
+#pragma unroll
+            for (int r = 0; r < R; r++) {
+                if ((item + 2 * gridDim.x) * R + r >= n) break;
+                for (uint32_t c = lo1 + lane * 64; c < hi1; c += 2048) prefetch_l2(nu + (size_t)r * k1 + c);
+                for (uint32_t c = lo2 + lane * 64; c < hi2; c += 2048) prefetch_l2(nd + (size_t)r * k2 + c);
+            }
+        }
         dot_range<R>(u, xs, lo1, hi1, lane, acc1);
         dot_range<R>(d, xs + k1, lo2, hi2, lane, acc2);
 #pragma unroll
@@ -175,7 +186,7 @@ cudaError_t rows_in_r(const RowsIn& op, int num_sms, cudaStream_t st, bool pdl) 
     cudaError_t err = allow_smem(rows_in_kernel<R>, 224 * 1024, done);
     if (err != cudaSuccess) return err;
     const uint32_t items = (op.w0.n + R - 1) / R + op.gu.n / R;
-    const uint32_t grid = std::min<uint32_t>((items + RW - 1) / RW, (uint32_t)num_sms * 3);
+    const uint32_t grid = std::min<uint32_t>((items + RW - 1) / RW, (uint32_t)num_sms * 2);
     return launch_pdl(rows_in_kernel<R>, dim3(grid), dim3(RT), (size_t)op.w0.k * 4, st, pdl, op);
 }
 template <int R>
@@ -184,7 +195,7 @@ cudaError_t rows_out_r(const RowsOut& op, int num_sms, cudaStream_t st, bool pdl
     cudaError_t err = allow_smem(rows_out_kernel<R>, 224 * 1024, done);
     if (err != cudaSuccess) return err;
     const uint32_t items = (op.w1.n + R - 1) / R;
-    const uint32_t grid = std::min<uint32_t>(items, (uint32_t)num_sms * 3);
+    const uint32_t grid = std::min<uint32_t>(items, (uint32_t)num_sms * 2);
     return launch_pdl(rows_out_kernel<R>, dim3(grid), dim3(RT), (size_t)(op.w1.k + (op.w2.n ? op.w2.k : 0)) * 4, st, pdl, op);
 }
 

@@ -244,9 +244,11 @@ __global__ void __launch_bounds__(64) latent_join_kernel(const __grid_constant__
     }
     __syncthreads();
     float v = 0.0f;
-#pragma unroll 8
-    for (uint32_t k = 0; k < a.splits; k++)
-        if (wt[k] != 0.0f) v = fmaf(wt[k], part[k * step + c], v);   // an empty share holds no sums
+#pragma unroll 16
+    for (uint32_t k = 0; k < a.splits; k++) {
+        const float x = part[k * step + c], w = wt[k];
+        v = w != 0.0f ? fmaf(w, x, v) : v;   // an empty share holds no sums
+    }
     a.mix[((size_t)t * s.heads + h) * s.cp + c] = v;
 }
 

@@ -34,21 +34,23 @@ cudaError_t launch_layer_norm(const NormArgs& a, uint32_t rows, cudaStream_t st,
 // ---- delta.cu: delta rule with one decay per key channel ----------------------------------------
 struct DeltaShape {
     uint32_t heads, kv_heads, dim, vdim, taps;
-    uint32_t dp, vp;                  // dim and vdim padded (dp: 32, 64, 128 or 256; vp: multiple of 32)
+    uint32_t dp, vp;                  // dim and vdim padded (dp: 64, 128 or 256; vp: multiple of 32)
     uint32_t off_q, off_k, off_v, off_b, conv_cols;   // columns of the projection output; the convolution covers [0, conv_cols)
 };
 constexpr uint32_t DELTA_MAX_DIM = 256;
-inline uint32_t delta_pad_dim(uint32_t d) { return d <= 32 ? 32 : d <= 64 ? 64 : d <= 128 ? 128 : 256; }
+inline uint32_t delta_pad_dim(uint32_t d) { return d <= 64 ? 64 : d <= 128 ? 128 : 256; }
+constexpr uint32_t DELTA_BLOCK = 16;      // tokens per block of the recurrence
 
 struct DeltaArgs {
     DeltaShape s;
     const float* y = nullptr;         // projections [t][ldy]: q | k | v | b | ...
     uint32_t ldy = 0;
-    const float* conv_w = nullptr;    // [conv_cols][taps]
+    const float* conv_w = nullptr;    // [taps][conv_cols]
     float* conv_state = nullptr;      // two of [taps - 1][conv_cols], oldest first: the one of a position's parity holds the inputs before it
     const int* pos = nullptr;
     float* state = nullptr;           // [heads][vp][dp]
-    float *qn = nullptr, *kn = nullptr, *kq = nullptr, *v = nullptr, *beta = nullptr;   // prepared inputs of the recurrence
+    float *qn = nullptr, *kn = nullptr, *v = nullptr, *beta = nullptr;   // prepared inputs of the recurrence
+    float *pair_inv = nullptr, *pair_b = nullptr;   // [blocks][heads][DELTA_BLOCK][DELTA_BLOCK]
     const float* g = nullptr;         // decays [t][heads][dp]
     float* o = nullptr;               // [t][heads][vdim]
     const float* gate = nullptr;      // sigmoid already applied, [t][heads * vdim]

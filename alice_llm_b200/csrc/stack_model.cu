@@ -36,7 +36,7 @@ struct Scratch {
     void* cqn = nullptr;
     bf16 *k_all = nullptr, *v_all = nullptr;         // keys and values of the whole context (tiled prefill)
     // delta
-    float *qn = nullptr, *kn = nullptr, *kq = nullptr, *v = nullptr, *beta = nullptr, *g = nullptr, *gate = nullptr, *o = nullptr;
+    float *qn = nullptr, *kn = nullptr, *pair_inv = nullptr, *pair_b = nullptr, *v = nullptr, *beta = nullptr, *g = nullptr, *gate = nullptr, *o = nullptr;
     bf16* low = nullptr;                             // bf16 copy of the low-rank columns
 };
 
@@ -179,7 +179,7 @@ struct DeltaMixer final : Mixer {
         const bool pdl = m->e->pdl, low = m->tiled_bf16(n);
         DeltaArgs a;
         a.s = sh; a.y = s.y; a.ldy = s.ldy; a.conv_w = conv; a.conv_state = states[pass].conv; a.state = states[pass].s;
-        a.qn = s.qn; a.kn = s.kn; a.kq = s.kq; a.v = s.v; a.beta = s.beta; a.g = s.g; a.o = s.o; a.gate = s.gate; a.norm_w = norm; a.eps = m->cfg.eps;
+        a.qn = s.qn; a.kn = s.kn; a.pair_inv = s.pair_inv; a.pair_b = s.pair_b; a.v = s.v; a.beta = s.beta; a.g = s.g; a.o = s.o; a.gate = s.gate; a.norm_w = norm; a.eps = m->cfg.eps;
         a.out = s.a; a.ldo = o.k; a.out_bf16 = low; a.pos = m->d_pos;
         if (n == 1 && delta_step_fits(sh)) {
             DeltaStepArgs sa;
@@ -431,7 +431,7 @@ void build_scratch(Builder& b) {
     m->chunk = std::min<uint32_t>(small ? CHUNK_SMALL : CHUNK, pad_to(m->max_seq, 64));
     const uint32_t M = m->chunk, ML = small ? M : std::min(M, FEW_TOKENS);
     uint32_t k_all = 0, v_all = 0;
-    uint32_t ldy = 0, ldf = 0, lda = 0, q = 0, ql = 0, part = 0, mix = 0, qp = 0, kd = 0, kh = 0, v = 0, h = 0, g = 0, o = 0, low = 0;
+    uint32_t ldy = 0, ldf = 0, lda = 0, q = 0, ql = 0, part = 0, mix = 0, qp = 0, kd = 0, v = 0, h = 0, g = 0, o = 0, low = 0;
     for (const auto& L : m->layers) {
         ldy = std::max(ldy, L.mixer->in.n);
         lda = std::max(lda, L.mixer->o.k);
@@ -443,7 +443,7 @@ void build_scratch(Builder& b) {
             ql = std::max(ql, z.heads * (z.cp + z.rp)); part = std::max(part, z.heads * (z.cp + 2)); mix = std::max(mix, z.heads * z.cp);
         } else if (const auto* x = dynamic_cast<const DeltaMixer*>(L.mixer.get())) {
             const DeltaShape& z = x->sh;
-            kd = std::max(kd, z.kv_heads * z.dp); kh = std::max(kh, z.kv_heads); v = std::max(v, z.heads * z.vp); h = std::max(h, z.heads);
+            kd = std::max(kd, z.kv_heads * z.dp); v = std::max(v, z.heads * z.vp); h = std::max(h, z.heads);
             g = std::max(g, z.heads * z.dp); o = std::max(o, z.heads * z.vdim); low = std::max(low, x->in.n - x->off_a);
         }
     }
@@ -460,7 +460,8 @@ void build_scratch(Builder& b) {
     s.mix = b.zeros<float>((size_t)ML * mix);
     s.k_all = b.zeros<bf16>((size_t)m->max_seq * k_all);
     s.v_all = b.zeros<bf16>((size_t)m->max_seq * v_all);
-    s.qn = b.zeros<float>((size_t)M * kd); s.kn = b.zeros<float>((size_t)M * kd); s.kq = b.zeros<float>((size_t)M * kh);
+    s.qn = b.zeros<float>((size_t)M * kd); s.kn = b.zeros<float>((size_t)M * kd);
+    s.pair_inv = b.zeros<float>((size_t)M * h * DELTA_BLOCK); s.pair_b = b.zeros<float>((size_t)M * h * DELTA_BLOCK);
     s.v = b.zeros<float>((size_t)M * v); s.beta = b.zeros<float>((size_t)M * h); s.g = b.zeros<float>((size_t)M * g);
     s.gate = b.zeros<float>((size_t)M * o); s.o = b.zeros<float>((size_t)M * o);
     s.low = b.zeros<bf16>((size_t)M * low);

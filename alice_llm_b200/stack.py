@@ -26,7 +26,7 @@ def pad(n: int, m: int = PAD) -> int:
 
 def delta_dim(dim: int) -> int:
     """Key channels of a head as the recurrence keeps them."""
-    for d in (32, 64, 128, 256):
+    for d in (64, 128, 256):
         if dim <= d:
             return d
     raise ConfigError(f"channel_delta: dim {dim} above 256")
@@ -206,10 +206,10 @@ def pack_layer(ck: Checkpoint, i: int, L: LayerSpec, width: int):
         dt = np.zeros((H, dp), np.float32)
         dt[:, :D] = ck.floats(m + "dt_bias", H * D).reshape(H, D)
         convs = [ck.floats(m + f"{n}.conv", r, K) for n, r in L.input_segments()[:3]]
-        conv = np.zeros((sum(pad(len(c)) for c in convs), K), np.float32)
+        conv = np.zeros((K, sum(pad(len(c)) for c in convs)), np.float32)
         at = 0
         for c in convs:
-            conv[at:at + len(c)] = c
+            conv[:, at:at + len(c)] = c.T
             at += pad(len(c))
         vecs.update(conv=conv, a_log=ck.floats(m + "A_log", H), dt_bias=dt, head_norm=ck.floats(m + "norm", V))
     if L.ff:

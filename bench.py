@@ -868,7 +868,7 @@ def build_stack(eng, z, max_seq_len, seed=0):
         if L.kind == stack.MIX_LATENT:
             vecs.update(q_norm=one(L.q_rank), kv_norm=one(L.kv_rank), sink=small(L.heads))
         else:
-            vecs.update(conv=small(sum(stack.pad(r) for _, r in L.input_segments()[:3]), L.conv_taps), a_log=small(L.heads),
+            vecs.update(conv=small(L.conv_taps, sum(stack.pad(r) for _, r in L.input_segments()[:3])), a_log=small(L.heads),
                         dt_bias=small(L.heads * stack.delta_dim(L.dim)) - 2.0, head_norm=one(L.vdim))
         packed.append((mats, vecs))
     embed = mat(cfg.vocab_size, stack.pad(cfg.width))

@@ -285,11 +285,11 @@ int32_t alice_model_set_position(alice_model* m, uint32_t pos);
  *   in    latent: [P(q_rank) query latent | P(kv_rank + rot_dim) key latent, key part | P(heads * vdim) gate]
  *         delta:  [P(kv_heads * dim) q | same k | P(heads * vdim) v | P(heads) step | P(decay_rank) | P(gate_rank)]
  *   uq    [heads * (dim + rot_dim)][P(q_rank)]       uk [heads * dim][P(kv_rank)]      uv [heads * vdim][P(kv_rank)]
- *   a2    [heads * D][P(decay_rank)] with dim padded to D = 32, 64, 128 or 256 per head; dt_bias likewise [heads * D]
+ *   a2    [heads * D][P(decay_rank)] with dim padded to D = 64, 128 or 256 per head; dt_bias likewise [heads * D]
  *   g2    [heads * vdim][P(gate_rank)]               o  [width][P(heads * vdim)]
  *   gu    64 gate rows, 64 up rows, 64 gate rows, ... of P(ff) each [2 P(ff)][P(width)]; down [width][P(ff)]
  *   embed [vocab][P(width)]
- * and gate_bias / up_bias hold P(ff) floats. conv [columns of q | k | v in `in`][conv_taps]. Float arrays are copied. */
+ * and gate_bias / up_bias hold P(ff) floats. conv [conv_taps][columns of q | k | v in `in`]. Float arrays are copied. */
 #define ALICE_MIX_LATENT 1u
 #define ALICE_MIX_DELTA 2u
 typedef struct {

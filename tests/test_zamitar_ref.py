@@ -224,7 +224,7 @@ def test_packed_layers_hold_every_weight(name):
             dp = stack.delta_dim(L.dim)
             a2 = mats["a2"].reshape(L.heads, dp, -1)
             assert np.array_equal(a2[:, :L.dim, :L.decay_rank].reshape(L.heads * L.dim, -1), w[f"l{i}.mix.a2"])
-            assert vecs["conv"].shape == (sum(stack.pad(r) for _, r in L.input_segments()[:3]), L.conv_taps)
+            assert vecs["conv"].shape == (L.conv_taps, sum(stack.pad(r) for _, r in L.input_segments()[:3]))
 
 
 def test_registry_refuses_unknown_architectures(tmp_path):
