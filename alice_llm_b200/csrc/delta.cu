@@ -40,41 +40,79 @@ __device__ __forceinline__ void conv_keep(const DeltaArgs& a, const float* befor
     }
 }
 
-// One warp per (token, key head) or (token, value head); the warps of a CTA take consecutive tokens of one head, so the
-// convolution's window comes from L1.
-__global__ void __launch_bounds__(256) delta_prepare_kernel(const __grid_constant__ DeltaArgs a, uint32_t tokens) {
+constexpr int PREP_TOKENS = 8;   // consecutive tokens of a warp
+// Convolution and silu of channel c for PREP_TOKENS tokens from t0 on. TAPS > 0: the number of taps, known when compiled.
+template <int TAPS>
+__device__ __forceinline__ void conv_run(const DeltaArgs& a, const float* before, int t0, uint32_t tokens, uint32_t c, float (&out)[PREP_TOKENS]) {
+    if constexpr (TAPS == 0) {
+#pragma unroll
+        for (int j = 0; j < PREP_TOKENS; j++) out[j] = (uint32_t)(t0 + j) < tokens ? conv_silu(a, before, t0 + j, c) : 0.0f;
+    } else {
+        float w[TAPS], x[PREP_TOKENS + TAPS - 1];
+#pragma unroll
+        for (int j = 0; j < TAPS; j++) w[j] = a.conv_w[(size_t)j * a.s.conv_cols + c];
+#pragma unroll
+        for (int j = 0; j < PREP_TOKENS + TAPS - 1; j++) {
+            const int s = t0 + j - (TAPS - 1);
+            x[j] = s < 0 ? before[(size_t)(TAPS - 1 + s) * a.s.conv_cols + c] : (uint32_t)s < tokens ? a.y[(size_t)s * a.ldy + c] : 0.0f;
+        }
+#pragma unroll
+        for (int j = 0; j < PREP_TOKENS; j++) {
+            float v = 0.0f;
+#pragma unroll
+            for (int i = 0; i < TAPS; i++) v = fmaf(w[i], x[j + i], v);
+            out[j] = silu_ref(v);
+        }
+    }
+}
+
+// One warp per head (key heads, then value heads) and PREP_TOKENS tokens: convolution, silu, unit vectors, step size.
+template <int TAPS, int N>   // N: 32-channel groups of a padded key head
+__global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constant__ DeltaArgs a, uint32_t tokens) {
     pdl_launch_dependents();
     pdl_wait();
     const DeltaShape& s = a.s;
-    const uint32_t lane = threadIdx.x & 31, t = blockIdx.x * 8 + (threadIdx.x >> 5), i = blockIdx.y;
-    if (t >= tokens) return;
+    const uint32_t lane = threadIdx.x & 31, t0 = (blockIdx.x * 4 + (threadIdx.x >> 5)) * PREP_TOKENS, i = blockIdx.y;
+    if (t0 >= tokens) return;
+    const uint32_t n = min(tokens - t0, (uint32_t)PREP_TOKENS);
     const float* before = conv_before(a);
     if (i < s.kv_heads) {
-        constexpr int N = DELTA_MAX_DIM / 32;
-        float q[N], k[N], sq = 0.0f, sk = 0.0f;
+#pragma unroll 1
+        for (int which = 0; which < 2; which++) {   // q, then k
+            const uint32_t off = (which ? s.off_k : s.off_q) + i * s.dim;
+            float v[N][PREP_TOKENS], ss[PREP_TOKENS] = {};
 #pragma unroll
-        for (int j = 0; j < N; j++) {
-            const uint32_t d = lane + 32 * j;
-            q[j] = k[j] = 0.0f;
-            if (d < s.dim) {
-                q[j] = conv_silu(a, before, (int)t, s.off_q + i * s.dim + d);
-                k[j] = conv_silu(a, before, (int)t, s.off_k + i * s.dim + d);
+            for (int g = 0; g < N; g++) {
+                const uint32_t d = lane + 32 * g;
+                if (d < s.dim) {
+                    conv_run<TAPS>(a, before, (int)t0, tokens, off + d, v[g]);
+                } else {
+#pragma unroll
+                    for (int j = 0; j < PREP_TOKENS; j++) v[g][j] = 0.0f;
+                }
+#pragma unroll
+                for (int j = 0; j < PREP_TOKENS; j++) ss[j] = fmaf(v[g][j], v[g][j], ss[j]);
             }
-            sq = fmaf(q[j], q[j], sq); sk = fmaf(k[j], k[j], sk);
-        }
-        sq = warp_sum(sq); sk = warp_sum(sk);
-        const float iq = __frcp_rn(__fsqrt_rn(sq + 1e-6f)) * __frcp_rn(__fsqrt_rn((float)s.dim)), ik = __frcp_rn(__fsqrt_rn(sk + 1e-6f));
-        const size_t o = ((size_t)t * s.kv_heads + i) * s.dp;
+            float* out = (which ? a.kn : a.qn) + ((size_t)t0 * s.kv_heads + i) * s.dp;
 #pragma unroll
-        for (int j = 0; j < N; j++) {
-            const uint32_t d = lane + 32 * j;
-            if (d < s.dp) { a.qn[o + d] = q[j] * iq; a.kn[o + d] = k[j] * ik; }
+            for (int j = 0; j < PREP_TOKENS; j++) {
+                float inv = __frcp_rn(__fsqrt_rn(warp_sum(ss[j]) + 1e-6f));
+                if (which == 0) inv *= __frcp_rn(__fsqrt_rn((float)s.dim));
+                if ((uint32_t)j < n)
+#pragma unroll
+                    for (int g = 0; g < N; g++) out[(size_t)j * s.kv_heads * s.dp + lane + 32 * g] = v[g][j] * inv;
+            }
         }
     } else {
         const uint32_t h = i - s.kv_heads;
-        const size_t o = ((size_t)t * s.heads + h) * s.vp;
-        for (uint32_t d = lane; d < s.vp; d += 32) a.v[o + d] = d < s.vdim ? conv_silu(a, before, (int)t, s.off_v + h * s.vdim + d) : 0.0f;
-        if (lane == 0) a.beta[(size_t)t * s.heads + h] = sigmoid_f(a.y[(size_t)t * a.ldy + s.off_b + h]);
+        for (uint32_t d = lane; d < s.vp; d += 32) {
+            float v[PREP_TOKENS] = {};
+            if (d < s.vdim) conv_run<TAPS>(a, before, (int)t0, tokens, s.off_v + h * s.vdim + d, v);
+#pragma unroll
+            for (int j = 0; j < PREP_TOKENS; j++)
+                if ((uint32_t)j < n) a.v[((size_t)(t0 + j) * s.heads + h) * s.vp + d] = v[j];
+        }
+        if (lane < n) a.beta[(size_t)(t0 + lane) * s.heads + h] = sigmoid_f(a.y[(size_t)(t0 + lane) * a.ldy + s.off_b + h]);
     }
 }
 
@@ -177,10 +215,10 @@ __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
 }
 __device__ __forceinline__ float2 mul2(float2 a, float2 b) { return make_float2(a.x * b.x, a.y * b.y); }
 
-// Sums 64 values over the warp; lane l is left with those of index 2 l and 2 l + 1.
-__device__ __forceinline__ float2 reduce64(float (&v)[64], uint32_t lane) {
+// Sums 64 values over each half-warp; lane l of it is left with those of index 4 l .. 4 l + 3.
+__device__ __forceinline__ float4 reduce64(float (&v)[64], uint32_t lane) {
 #pragma unroll
-    for (int half = 32, o = 16; o > 0; half >>= 1, o >>= 1) {
+    for (int half = 32, o = 8; o > 0; half >>= 1, o >>= 1) {
         const bool up = lane & o;
 #pragma unroll
         for (int i = 0; i < half; i++) {
@@ -188,20 +226,20 @@ __device__ __forceinline__ float2 reduce64(float (&v)[64], uint32_t lane) {
             v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
         }
     }
-    return make_float2(v[0], v[1]);
+    return make_float4(v[0], v[1], v[2], v[3]);
 }
 
 template <int DP, int NW>
 struct ScanStage {
-    float k[W][DP], q[W][DP], g[W][DP], v[W][4 * NW], inv[W][W], b[W][W];
+    float k[W][DP], q[W][DP], g[W][DP], v[W][8 * NW], inv[W][W], b[W][W];
 };
 template <int DP, int NW>
 struct ScanSmem {
     ScanStage<DP, NW> st[2];
     float end[DP];                 // decay over the whole block
-    float w[W][4 * NW];            // v - S^T (G k)
-    float y[W][4 * NW];            // S^T (G q)
-    float2 u[W][4 * NW];           // writes, twice each
+    float w[W][8 * NW];            // v - S^T (G k)
+    float y[W][8 * NW];            // S^T (G q)
+    float2 u[W][8 * NW];           // writes, twice each
 };
 
 template <int DP, int NW>
@@ -214,8 +252,8 @@ __device__ __forceinline__ void scan_fetch(ScanStage<DP, NW>& st, const DeltaArg
         cp_async16(&st.q[j][d], a.qn + ko, j < n);
         cp_async16(&st.g[j][d], a.g + ((size_t)t * s.heads + h) * DP + d, j < n);
     }
-    for (uint32_t i = threadIdx.x; i < W * NW; i += NW * 32) {
-        const uint32_t j = i / NW, d = i % NW * 4, t = t0 + min(j, n - 1);
+    for (uint32_t i = threadIdx.x; i < W * 2 * NW; i += NW * 32) {
+        const uint32_t j = i / (2 * NW), d = i % (2 * NW) * 4, t = t0 + min(j, n - 1);
         cp_async16(&st.v[j][d], a.v + ((size_t)t * s.heads + h) * s.vp + c0 + d, j < n);
     }
     const size_t o = ((size_t)(t0 / W) * s.heads + h) * W * W;
@@ -225,26 +263,24 @@ __device__ __forceinline__ void scan_fetch(ScanStage<DP, NW>& st, const DeltaArg
     }
 }
 
-// grid (vp / (4 NW), heads), NW warps; a warp owns four columns of the state, a lane DP / 32 of their rows (register pairs).
+// grid (vp / (8 NW), heads), NW warps; a warp owns eight columns of the state, four per half-warp, a lane DP / 16 of their rows
+// (register pairs).
 template <int DP, int NW>
 __global__ void __launch_bounds__(NW * 32) delta_scan_kernel(const __grid_constant__ DeltaArgs a, uint32_t tokens) {
-    constexpr int EL = DP / 32, NP = EL / 2, VEC = EL < 4 ? EL : 4, NC = EL / VEC, COLS = 4 * NW;   // rows per lane, in NC runs of VEC
+    constexpr int EL = DP / 16, NP = EL / 2, NC = EL / 4, COLS = 8 * NW;   // rows per lane, in NC runs of four
     extern __shared__ __align__(16) uint8_t raw[];
     auto& sm = *reinterpret_cast<ScanSmem<DP, NW>*>(raw);
     const DeltaShape& s = a.s;
-    const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, kh = h / (s.heads / s.kv_heads), c0 = blockIdx.x * COLS;
-    float* sp = a.state + ((size_t)h * s.vp + c0 + warp * 4) * DP + lane * VEC;
+    const uint32_t tid = threadIdx.x, lane = tid & 31, dg = lane & 15, warp = tid >> 5, h = blockIdx.y, kh = h / (s.heads / s.kv_heads), c0 = blockIdx.x * COLS;
+    const uint32_t cw = warp * 8, cl = cw + (lane >> 4) * 4;   // first column of the warp, of the lane
+    float* sp = a.state + ((size_t)h * s.vp + c0 + cl) * DP + dg * 4;
     pdl_launch_dependents();
     pdl_wait();
     auto rows = [](const float* p, float2 (&r)[NP]) {   // this lane's rows of a [DP] vector
 #pragma unroll
         for (int i = 0; i < NC; i++) {
-            if constexpr (VEC == 4) {
-                const float4 f = *reinterpret_cast<const float4*>(p + i * 32 * VEC);
-                r[2 * i] = make_float2(f.x, f.y); r[2 * i + 1] = make_float2(f.z, f.w);
-            } else {
-                r[i] = *reinterpret_cast<const float2*>(p + i * 32 * VEC);
-            }
+            const float4 f = *reinterpret_cast<const float4*>(p + i * 64);
+            r[2 * i] = make_float2(f.x, f.y); r[2 * i + 1] = make_float2(f.z, f.w);
         }
     };
     float2 S[4][NP];
@@ -286,7 +322,7 @@ __global__ void __launch_bounds__(NW * 32) delta_scan_kernel(const __grid_consta
 #pragma unroll
             for (int t = 0; t < W; t++) {
                 float2 x[NP];
-                rows((pass ? st.q[t] : st.k[t]) + lane * VEC, x);
+                rows((pass ? st.q[t] : st.k[t]) + dg * 4, x);
 #pragma unroll
                 for (int c = 0; c < 4; c++) {
                     float2 acc = mul2(x[0], S[c][0]);
@@ -295,38 +331,50 @@ __global__ void __launch_bounds__(NW * 32) delta_scan_kernel(const __grid_consta
                     v[t * 4 + c] = acc.x + acc.y;
                 }
             }
-            const float2 r = reduce64(v, lane);
-            const uint32_t t = lane / 2, c = warp * 4 + (lane & 1) * 2;
-            if (pass == 0) *reinterpret_cast<float2*>(&sm.w[t][c]) = make_float2(st.v[t][c] - r.x, st.v[t][c + 1] - r.y);
-            else *reinterpret_cast<float2*>(&sm.y[t][c]) = r;
+            const float4 r = reduce64(v, lane);   // token dg, the lane's four columns
+            if (pass == 0) {
+                const float4 x = *reinterpret_cast<const float4*>(&st.v[dg][cl]);
+                *reinterpret_cast<float4*>(&sm.w[dg][cl]) = make_float4(x.x - r.x, x.y - r.y, x.z - r.z, x.w - r.w);
+            } else {
+                *reinterpret_cast<float4*>(&sm.y[dg][cl]) = r;
+            }
         }
         __syncwarp();   // from here to the end of the block a warp works on its own columns only
         {
-            const uint32_t c = warp * 4 + (lane & 3), t1 = lane >> 2, t2 = t1 + 8;   // two tokens of one column
-            float u1 = 0.0f, u2 = 0.0f;
+            const uint32_t c = cw + (lane & 7), tl = lane >> 3;   // tokens tl, tl + 4, tl + 8, tl + 12 of one column
+            float u[4] = {};
 #pragma unroll
-            for (int j = 0; j < W; j++) {
-                const float w = sm.w[j][c];
-                u1 = fmaf(st.inv[t1][j], w, u1);
-                u2 = fmaf(st.inv[t2][j], w, u2);
+            for (int j = 0; j < W; j += 4) {
+                const float w0 = sm.w[j][c], w1 = sm.w[j + 1][c], w2 = sm.w[j + 2][c], w3 = sm.w[j + 3][c];
+#pragma unroll
+                for (int i = 0; i < 4; i++) {
+                    const float4 m = *reinterpret_cast<const float4*>(&st.inv[tl + 4 * i][j]);
+                    u[i] = fmaf(m.x, w0, u[i]); u[i] = fmaf(m.y, w1, u[i]); u[i] = fmaf(m.z, w2, u[i]); u[i] = fmaf(m.w, w3, u[i]);
+                }
             }
-            sm.u[t1][c] = make_float2(u1, u1);
-            sm.u[t2][c] = make_float2(u2, u2);
+            float o[4];
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                sm.u[tl + 4 * i][c] = make_float2(u[i], u[i]);
+                o[i] = sm.y[tl + 4 * i][c];
+            }
             __syncwarp();
-            float o1 = sm.y[t1][c], o2 = sm.y[t2][c];
 #pragma unroll
-            for (int j = 0; j < W; j++) {
-                const float u = sm.u[j][c].x;
-                o1 = fmaf(st.b[t1][j], u, o1);
-                o2 = fmaf(st.b[t2][j], u, o2);
+            for (int j = 0; j < W; j += 4) {
+                const float w0 = sm.u[j][c].x, w1 = sm.u[j + 1][c].x, w2 = sm.u[j + 2][c].x, w3 = sm.u[j + 3][c].x;
+#pragma unroll
+                for (int i = 0; i < 4; i++) {
+                    const float4 m = *reinterpret_cast<const float4*>(&st.b[tl + 4 * i][j]);
+                    o[i] = fmaf(m.x, w0, o[i]); o[i] = fmaf(m.y, w1, o[i]); o[i] = fmaf(m.z, w2, o[i]); o[i] = fmaf(m.w, w3, o[i]);
+                }
             }
-            if (c0 + c < s.vdim) {
-                if (t1 < n) a.o[((size_t)(t0 + t1) * s.heads + h) * s.vdim + c0 + c] = o1;
-                if (t2 < n) a.o[((size_t)(t0 + t2) * s.heads + h) * s.vdim + c0 + c] = o2;
-            }
+            if (c0 + c < s.vdim)
+#pragma unroll
+                for (int i = 0; i < 4; i++)
+                    if (tl + 4 * i < n) a.o[((size_t)(t0 + tl + 4 * i) * s.heads + h) * s.vdim + c0 + c] = o[i];
         }
         float2 e[NP];
-        rows(sm.end + lane * VEC, e);
+        rows(sm.end + dg * 4, e);
 #pragma unroll
         for (int c = 0; c < 4; c++)
 #pragma unroll
@@ -334,10 +382,10 @@ __global__ void __launch_bounds__(NW * 32) delta_scan_kernel(const __grid_consta
 #pragma unroll
         for (int t = 0; t < W; t++) {
             float2 x[NP];
-            rows(st.g[t] + lane * VEC, x);
+            rows(st.g[t] + dg * 4, x);
 #pragma unroll
             for (int c = 0; c < 4; c++) {
-                const float2 u = sm.u[t][warp * 4 + c];
+                const float2 u = sm.u[t][cl + c];
 #pragma unroll
                 for (int i = 0; i < NP; i++) S[c][i] = fma2(x[i], u, S[c][i]);
             }
@@ -348,9 +396,7 @@ __global__ void __launch_bounds__(NW * 32) delta_scan_kernel(const __grid_consta
     for (int c = 0; c < 4; c++)
 #pragma unroll
         for (int i = 0; i < NC; i++) {
-            float* p = sp + c * DP + i * 32 * VEC;
-            if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(S[c][2 * i].x, S[c][2 * i].y, S[c][2 * i + 1].x, S[c][2 * i + 1].y);
-            else *reinterpret_cast<float2*>(p) = S[c][i];
+            *reinterpret_cast<float4*>(sp + c * DP + i * 64) = make_float4(S[c][2 * i].x, S[c][2 * i].y, S[c][2 * i + 1].x, S[c][2 * i + 1].y);
         }
 }
 
@@ -522,7 +568,7 @@ cudaError_t scan_inst(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool
     constexpr size_t smem = sizeof(ScanSmem<DP, NW>);
     const cudaError_t err = allow_smem(delta_scan_kernel<DP, NW>, smem, done);
     if (err != cudaSuccess) return err;
-    return launch_pdl(delta_scan_kernel<DP, NW>, dim3(a.s.vp / (4 * NW), a.s.heads), dim3(NW * 32), smem, st, pdl, a, tokens);
+    return launch_pdl(delta_scan_kernel<DP, NW>, dim3(a.s.vp / (8 * NW), a.s.heads), dim3(NW * 32), smem, st, pdl, a, tokens);
 }
 template <int DP>
 cudaError_t scan_dim(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
@@ -533,13 +579,24 @@ cudaError_t scan_dim(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool 
     err = launch_pdl(delta_pairs_kernel<DP>, dim3((tokens + W - 1) / W, a.s.heads), dim3(256), smem, st, pdl, a, tokens);
     if (err != cudaSuccess) return err;
     // few columns: narrower CTAs, so that more SMs have one
-    return a.s.heads * (a.s.vp / 32) < 100 ? scan_inst<DP, 4>(a, tokens, st, pdl) : scan_inst<DP, 8>(a, tokens, st, pdl);
+    return a.s.heads * (a.s.vp / 32) < 100 ? scan_inst<DP, 2>(a, tokens, st, pdl) : scan_inst<DP, 4>(a, tokens, st, pdl);
 }
 
 }  // namespace
 
+template <int TAPS>
+static cudaError_t prepare_taps(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
+    const dim3 grid((tokens + 4 * PREP_TOKENS - 1) / (4 * PREP_TOKENS), a.s.kv_heads + a.s.heads);
+    switch (a.s.dp) {
+        case 64: return launch_pdl(delta_prepare_kernel<TAPS, 2>, grid, dim3(128), 0, st, pdl, a, tokens);
+        case 128: return launch_pdl(delta_prepare_kernel<TAPS, 4>, grid, dim3(128), 0, st, pdl, a, tokens);
+        case 256: return launch_pdl(delta_prepare_kernel<TAPS, 8>, grid, dim3(128), 0, st, pdl, a, tokens);
+        default: return cudaErrorInvalidValue;
+    }
+}
 cudaError_t launch_delta_prepare(const DeltaArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
-    cudaError_t err = launch_pdl(delta_prepare_kernel, dim3((tokens + 7) / 8, a.s.kv_heads + a.s.heads), dim3(256), 0, st, pdl, a, tokens);
+    const cudaError_t err = a.s.taps == 4 ? prepare_taps<4>(a, tokens, st, pdl) : a.s.taps == 3 ? prepare_taps<3>(a, tokens, st, pdl)
+                          : a.s.taps == 2 ? prepare_taps<2>(a, tokens, st, pdl) : prepare_taps<0>(a, tokens, st, pdl);
     if (err != cudaSuccess || a.s.taps <= 1) return err;
     return launch_pdl(conv_tail_kernel, dim3((a.s.conv_cols + 255) / 256), dim3(256), 0, st, pdl, a, tokens);
 }

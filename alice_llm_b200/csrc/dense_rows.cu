@@ -10,11 +10,11 @@ namespace {
 
 constexpr int RT = 256, RW = RT / 32;
 
-template <int R>
+template <int R, int U>
 __device__ __forceinline__ void dot_rows(const bf16* const (&w)[R], const float* xs, uint32_t k, uint32_t lane, float (&acc)[R]) {
 #pragma unroll
     for (int r = 0; r < R; r++) acc[r] = 0.0f;
-#pragma unroll 4
+#pragma unroll U
     for (uint32_t c = lane * 8; c < k; c += 256) {
         uint4 v[R];
 #pragma unroll
@@ -80,7 +80,7 @@ __global__ void __launch_bounds__(RT, 2) rows_in_kernel(const __grid_constant__ 
     for (uint32_t item = w_id; item < items; item += warps) {
         item_rows<R>(op, item, items0, w, first, pair);
         float acc[R];
-        dot_rows<R>(w, xs, k, lane, acc);
+        dot_rows<R, 4>(w, xs, k, lane, acc);
         if (!pair) {
 #pragma unroll
             for (int r = 0; r < R; r++) {
@@ -97,84 +97,29 @@ __global__ void __launch_bounds__(RT, 2) rows_in_kernel(const __grid_constant__ 
     if (op.argmax_key && lane == 0 && best) atomicMax(op.argmax_key, best);
 }
 
-// acc += W[.][lo, hi) x[lo, hi) of one matrix, lanes 8 columns apart
-template <int R>
-__device__ __forceinline__ void dot_range(const bf16* const (&w)[R], const float* xs, uint32_t lo, uint32_t hi, uint32_t lane, float (&acc)[R]) {
-#pragma unroll 8
-    for (uint32_t c = lo + lane * 8; c < hi; c += 256) {
-        uint4 v[R];
-#pragma unroll
-        for (int r = 0; r < R; r++) v[r] = __ldg(reinterpret_cast<const uint4*>(w[r] + c));
-        const float4 x0 = *reinterpret_cast<const float4*>(xs + c), x1 = *reinterpret_cast<const float4*>(xs + c + 4);
-#pragma unroll
-        for (int r = 0; r < R; r++) acc[r] = dot8(v[r], x0, x1, acc[r]);
-    }
-}
-
-// The CTA's warps share R rows: each takes an eighth of the columns of [W1 | W2] (so it reads only that part of the inputs),
-// scales its two partial sums and the parts meet in shared memory.
-template <int R>
-__global__ void __launch_bounds__(RT, 2) rows_out_kernel(const __grid_constant__ RowsOut op) {
+// A warp owns one row of [W1 | W2] at a time; the CTA has as many warps as spread the rows evenly over two CTAs per SM.
+constexpr int OUT_MAX_WARPS = 16;
+__global__ void __launch_bounds__(OUT_MAX_WARPS * 32, 2) rows_out_kernel(const __grid_constant__ RowsOut op) {
     extern __shared__ __align__(16) float xs[];
-    __shared__ float part[2][RW][R];
-    const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const uint32_t n = op.w1.n, k1 = op.w1.k, k2 = op.w2.n ? op.w2.k : 0, k = k1 + k2;
-    const uint32_t items = (n + R - 1) / R;
-    const uint32_t lo = k / 64 * warp / RW * 64, hi = k / 64 * (warp + 1) / RW * 64;   // this warp's columns
-    const uint32_t lo1 = min(lo, k1), hi1 = min(hi, k1), lo2 = max(lo, k1) - k1, hi2 = max(hi, k1) - k1;
-    const bf16 *u[R], *d[R];
-    auto rows_of = [&](uint32_t item) {
-#pragma unroll
-        for (int r = 0; r < R; r++) {
-            const uint32_t row = min(item * R + r, n - 1);
-            u[r] = op.w1.w + (size_t)row * k1;
-            d[r] = k2 ? op.w2.w + (size_t)row * k2 : u[r];
-        }
-    };
+    const uint32_t lane = threadIdx.x & 31, nw = blockDim.x >> 5, warps = gridDim.x * nw, w_id = blockIdx.x + (threadIdx.x >> 5) * gridDim.x;
+    const uint32_t n = op.w1.n, k1 = op.w1.k, k2 = op.w2.n ? op.w2.k : 0;
     pdl_launch_dependents();
-    for (uint32_t item = blockIdx.x; item < min(items, blockIdx.x + 2 * gridDim.x); item += gridDim.x) {
-        rows_of(item);
-#pragma unroll
-        for (int r = 0; r < R; r++) {
-            for (uint32_t c = lo1 + lane * 64; c < hi1; c += 2048) prefetch_l2(u[r] + c);
-            for (uint32_t c = lo2 + lane * 64; c < hi2; c += 2048) prefetch_l2(d[r] + c);
-        }
+    if (w_id < n) {
+        prefetch_row(op.w1.w + (size_t)w_id * k1, k1, lane);
+        if (k2) prefetch_row(op.w2.w + (size_t)w_id * k2, k2, lane);
     }
     pdl_wait();
-    for (uint32_t i = lo1 + lane * 4; i < hi1; i += 128) *reinterpret_cast<float4*>(xs + i) = __ldcg(reinterpret_cast<const float4*>(op.a + i));
-    for (uint32_t i = lo2 + lane * 4; i < hi2; i += 128) *reinterpret_cast<float4*>(xs + k1 + i) = __ldcg(reinterpret_cast<const float4*>(op.f + i));
-    __syncwarp();
-    uint32_t buf = 0;
-    for (uint32_t item = blockIdx.x; item < items; item += gridDim.x, buf ^= 1) {
-        rows_of(item);
-        float acc1[R], acc2[R];
-#pragma unroll
-        for (int r = 0; r < R; r++) acc1[r] = acc2[r] = 0.0f;
-        if (item + 2 * gridDim.x < items) {   // the one after the next one sets out for L2
-            const bf16* nu = op.w1.w + (size_t)(item + 2 * gridDim.x) * R * k1;
-            const bf16* nd = op.w2.w + (size_t)(item + 2 * gridDim.x) * R * k2;
-#pragma unroll
-            for (int r = 0; r < R; r++) {
-                if ((item + 2 * gridDim.x) * R + r >= n) break;
-                for (uint32_t c = lo1 + lane * 64; c < hi1; c += 2048) prefetch_l2(nu + (size_t)r * k1 + c);
-                for (uint32_t c = lo2 + lane * 64; c < hi2; c += 2048) prefetch_l2(nd + (size_t)r * k2 + c);
-            }
-        }
-        dot_range<R>(u, xs, lo1, hi1, lane, acc1);
-        dot_range<R>(d, xs + k1, lo2, hi2, lane, acc2);
-#pragma unroll
-        for (int r = 0; r < R; r++) {
-            const uint32_t row = min(item * R + r, n - 1);
-            const float v = warp_sum(k2 ? op.s1[row] * acc1[r] + op.s2[row] * acc2[r] : op.s1[row] * acc1[r]);
-            if (lane == 0) part[buf][warp][r] = v;
-        }
-        __syncthreads();   // the other buffer's readers are done before anyone writes it again
-        const uint32_t row = item * R + threadIdx.x;
-        if (threadIdx.x < R && row < n) {
-            float v = 0.0f;
-#pragma unroll
-            for (int w = 0; w < RW; w++) v += part[buf][w][threadIdx.x];
-            if (k2) v += op.s2[row] * op.b2[row];
+    for (uint32_t i = threadIdx.x * 4; i < k1; i += blockDim.x * 4) *reinterpret_cast<float4*>(xs + i) = __ldcg(reinterpret_cast<const float4*>(op.a + i));
+    for (uint32_t i = threadIdx.x * 4; i < k2; i += blockDim.x * 4) *reinterpret_cast<float4*>(xs + k1 + i) = __ldcg(reinterpret_cast<const float4*>(op.f + i));
+    __syncthreads();
+    for (uint32_t row = w_id; row < n; row += warps) {
+        const bf16 *const u[1] = {op.w1.w + (size_t)row * k1}, *const d[1] = {op.w2.w + (size_t)row * k2};
+        float acc1[1], acc2[1] = {0.0f};
+        if (k2) dot_rows<1, 8>(d, xs + k1, k2, lane, acc2);
+        dot_rows<1, 8>(u, xs, k1, lane, acc1);
+        if (lane == 0) {
+            float v = op.s1[row] * acc1[0];
+            if (k2) v += op.s2[row] * (acc2[0] + op.b2[row]);
             op.x[row] += v;
         }
     }
@@ -189,16 +134,6 @@ cudaError_t rows_in_r(const RowsIn& op, int num_sms, cudaStream_t st, bool pdl) 
     const uint32_t grid = std::min<uint32_t>((items + RW - 1) / RW, (uint32_t)num_sms * 2);
     return launch_pdl(rows_in_kernel<R>, dim3(grid), dim3(RT), (size_t)op.w0.k * 4, st, pdl, op);
 }
-template <int R>
-cudaError_t rows_out_r(const RowsOut& op, int num_sms, cudaStream_t st, bool pdl) {
-    static bool done[64] = {};
-    cudaError_t err = allow_smem(rows_out_kernel<R>, 224 * 1024, done);
-    if (err != cudaSuccess) return err;
-    const uint32_t items = (op.w1.n + R - 1) / R;
-    const uint32_t grid = std::min<uint32_t>(items, (uint32_t)num_sms * 2);
-    return launch_pdl(rows_out_kernel<R>, dim3(grid), dim3(RT), (size_t)(op.w1.k + (op.w2.n ? op.w2.k : 0)) * 4, st, pdl, op);
-}
-
 }  // namespace
 
 cudaError_t launch_rows_in(const RowsIn& op, int num_sms, cudaStream_t st, bool pdl) {
@@ -211,7 +146,13 @@ cudaError_t launch_rows_in(const RowsIn& op, int num_sms, cudaStream_t st, bool 
 cudaError_t launch_rows_out(const RowsOut& op, int num_sms, cudaStream_t st, bool pdl) {
     if (!op.w1.n || op.w1.k % DENSE_PAD || (op.w2.n && (op.w2.n != op.w1.n || op.w2.k % DENSE_PAD))) return cudaErrorInvalidValue;
     if ((size_t)(op.w1.k + (op.w2.n ? op.w2.k : 0)) * 4 > 220 * 1024) return cudaErrorInvalidValue;
-    return rows_out_r<2>(op, num_sms, st, pdl);
+    static bool done[64] = {};
+    const cudaError_t err = allow_smem(rows_out_kernel, 224 * 1024, done);
+    if (err != cudaSuccess) return err;
+    const uint32_t slots = (uint32_t)num_sms * 2, rounds = (op.w1.n + slots * OUT_MAX_WARPS - 1) / (slots * OUT_MAX_WARPS);
+    const uint32_t nw = std::min<uint32_t>(OUT_MAX_WARPS, std::max<uint32_t>(4, (op.w1.n + slots * rounds - 1) / (slots * rounds)));
+    const uint32_t grid = std::min(slots, (op.w1.n + nw - 1) / nw);
+    return launch_pdl(rows_out_kernel, dim3(grid), dim3(nw * 32), (size_t)(op.w1.k + (op.w2.n ? op.w2.k : 0)) * 4, st, pdl, op);
 }
 
 }  // namespace alice

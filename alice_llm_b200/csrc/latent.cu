@@ -228,24 +228,26 @@ __global__ void __launch_bounds__(64) latent_join_kernel(const __grid_constant__
     pdl_wait();
     const float* part = a.part + ((size_t)t * a.splits * s.heads + h) * (s.cp + 2);
     const size_t step = (size_t)s.heads * (s.cp + 2);
+    // shares that can hold keys (both attention kernels hand out the context in whole tiles of at least 32)
+    const uint32_t ctx = (uint32_t)*a.pos + t + 1, shares = min(a.splits, (ctx + 31) / 32);
     if (threadIdx.x < 32) {
         float top = a.sink[h];
-        for (uint32_t i = lane; i < a.splits; i += 32) top = fmaxf(top, part[i * step + s.cp]);
+        for (uint32_t i = lane; i < shares; i += 32) top = fmaxf(top, part[i * step + s.cp]);
         top = warp_max(top);
         float den = 0.0f;
-        for (uint32_t i = lane; i < a.splits; i += 32) {
+        for (uint32_t i = lane; i < shares; i += 32) {
             const float f = expf(part[i * step + s.cp] - top);   // an empty share left -inf
             wt[i] = f;
             den = fmaf(f, part[i * step + s.cp + 1], den);
         }
         den = warp_sum(den) + expf(a.sink[h] - top);
         const float inv = __frcp_rn(den);
-        for (uint32_t i = lane; i < a.splits; i += 32) wt[i] *= inv;
+        for (uint32_t i = lane; i < shares; i += 32) wt[i] *= inv;
     }
     __syncthreads();
     float v = 0.0f;
 #pragma unroll 16
-    for (uint32_t k = 0; k < a.splits; k++) {
+    for (uint32_t k = 0; k < shares; k++) {
         const float x = part[k * step + c], w = wt[k];
         v = w != 0.0f ? fmaf(w, x, v) : v;   // an empty share holds no sums
     }

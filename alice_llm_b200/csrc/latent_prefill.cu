@@ -9,9 +9,10 @@
 namespace alice {
 namespace {
 
-constexpr int PF_KEYS = 64, PF_ROWS = 128;   // keys per tile; queries per CTA, 16 per warp
+constexpr int PF_KEYS = 32, PF_ROWS = 128, PF_THREADS = 128;   // keys per tile; queries per CTA, 32 per warp: each key fragment serves two row tiles
 
-// DQ, DV: query / key and value dimensions the tiles have room for (multiples of 16, zero beyond the true sizes).
+// DQ, DV: query / key and value dimensions the tiles have room for (multiples of 16, zero beyond the true sizes). Values wider
+// than DV are cut into slices (blockIdx.z), each with its own pass over the scores.
 template <int DQ, int DV>
 struct PfGeom {
     static constexpr int LQ = DQ + 8, LV = DV + 8;   // row strides: eight rows land in different banks
@@ -19,7 +20,7 @@ struct PfGeom {
 };
 
 template <int DQ, int DV>
-__global__ void __launch_bounds__(256, 1) latent_prefill_kernel(const __grid_constant__ LatentArgs a, uint32_t tokens) {
+__global__ void __launch_bounds__(PF_THREADS, 2) latent_prefill_kernel(const __grid_constant__ LatentArgs a, uint32_t tokens) {
     using G = PfGeom<DQ, DV>;
     extern __shared__ __align__(128) uint8_t sm[];
     const LatentShape& s = a.s;
@@ -33,37 +34,38 @@ __global__ void __launch_bounds__(256, 1) latent_prefill_kernel(const __grid_con
     const uint32_t rows = min((uint32_t)PF_ROWS, tokens - t0), keys = p0 + t0 + rows, ntiles = (keys + PF_KEYS - 1) / PF_KEYS;
     const bf16* cache = static_cast<const bf16*>(a.cache);
     const uint32_t cw = s.cp + s.rp, kw = s.heads * s.dim, vw = s.heads * s.vdim;
+    const uint32_t v0 = blockIdx.z * DV, vn = min(s.vdim - v0, (uint32_t)DV);   // this slice of the values
 
     // zero what lies beyond the true sizes once (the copies below never touch it)
-    for (uint32_t i = tid; i < 2 * PF_KEYS * (DQ - qd); i += 256) {
+    for (uint32_t i = tid; i < 2 * PF_KEYS * (DQ - qd); i += PF_THREADS) {
         const uint32_t r = i / (DQ - qd), c = qd + i % (DQ - qd);
         reinterpret_cast<bf16*>(sm + G::Q + (r / PF_KEYS) * G::K)[(r % PF_KEYS) * G::LQ + c] = __float2bfloat16_rn(0.0f);
     }
-    for (uint32_t i = tid; i < 2 * PF_KEYS * (DV - s.vdim); i += 256) {
-        const uint32_t r = i / (DV - s.vdim), c = s.vdim + i % (DV - s.vdim);
+    for (uint32_t i = tid; i < 2 * PF_KEYS * (DV - vn); i += PF_THREADS) {
+        const uint32_t r = i / (DV - vn), c = vn + i % (DV - vn);
         reinterpret_cast<bf16*>(sm + G::Q + 2 * G::K + (r / PF_KEYS) * G::V)[(r % PF_KEYS) * G::LV + c] = __float2bfloat16_rn(0.0f);
     }
     auto fetch = [&](uint32_t tile, uint32_t b) {
-        const uint32_t j0 = tile * PF_KEYS, nd = s.dim / 8, nr = s.rot / 8, nv = s.vdim / 8;
+        const uint32_t j0 = tile * PF_KEYS, nd = s.dim / 8, nr = s.rot / 8, nv = vn / 8;
         const uint32_t kd = k_sm + b * (uint32_t)G::K, vd = v_sm + b * (uint32_t)G::V;
-        for (uint32_t i = tid; i < PF_KEYS * nd; i += 256) {
+        for (uint32_t i = tid; i < PF_KEYS * nd; i += PF_THREADS) {
             const uint32_t r = i / nd, c = i % nd * 8, j = min(j0 + r, keys - 1);
             cp16(kd + (r * G::LQ + c) * 2, a.k_all + (size_t)j * kw + (size_t)h * s.dim + c, j0 + r < keys);
         }
-        for (uint32_t i = tid; i < PF_KEYS * nr; i += 256) {
+        for (uint32_t i = tid; i < PF_KEYS * nr; i += PF_THREADS) {
             const uint32_t r = i / nr, c = i % nr * 8, j = min(j0 + r, keys - 1);
             cp16(kd + (r * G::LQ + s.dim + c) * 2, cache + (size_t)j * cw + s.cp + c, j0 + r < keys);
         }
-        for (uint32_t i = tid; i < PF_KEYS * nv; i += 256) {
+        for (uint32_t i = tid; i < PF_KEYS * nv; i += PF_THREADS) {
             const uint32_t r = i / nv, c = i % nv * 8, j = min(j0 + r, keys - 1);
-            cp16(vd + (r * G::LV + c) * 2, a.v_all + (size_t)j * vw + (size_t)h * s.vdim + c, j0 + r < keys);
+            cp16(vd + (r * G::LV + c) * 2, a.v_all + (size_t)j * vw + (size_t)h * s.vdim + v0 + c, j0 + r < keys);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     fetch(0, 0);
     // queries, the rotated part turned to its position on the way
     const uint32_t half = s.rot_dims / 2;
-    for (uint32_t i = tid; i < PF_ROWS * DQ; i += 256) {
+    for (uint32_t i = tid; i < PF_ROWS * DQ; i += PF_THREADS) {
         const uint32_t r = i / DQ, c = i % DQ;
         float v = 0.0f;
         if (r < rows && c < qd) {
@@ -81,16 +83,19 @@ __global__ void __launch_bounds__(256, 1) latent_prefill_kernel(const __grid_con
         qs[r * G::LQ + c] = __float2bfloat16_rn(v);
     }
 
-    // a thread's two rows are lane / 4 and lane / 4 + 8 of its warp's sixteen
+    // a thread's rows are lane / 4 and lane / 4 + 8 of each of its warp's two 16-row tiles
     constexpr float LOG2E = 1.4426950408889634f;
     const float scale = s.scale * LOG2E;
-    float m[2], l[2], o[DV / 8][4];
-    m[0] = m[1] = a.sink[h] * LOG2E;
-    l[0] = l[1] = (lane & 3) == 0 ? 1.0f : 0.0f;
+    float m[2][2], l[2][2], o[2][DV / 8][4];
 #pragma unroll
-    for (int i = 0; i < DV / 8; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
-    const uint32_t row0 = warp * 16 + lane / 4, see0 = p0 + t0 + row0, see1 = see0 + 8;   // last key a row sees
-    const uint32_t q_addr = q_sm + ((warp * 16 + lane % 16) * G::LQ + lane / 16 * 8) * 2;
+    for (int g = 0; g < 2; g++) {
+        m[g][0] = m[g][1] = a.sink[h] * LOG2E;
+        l[g][0] = l[g][1] = (lane & 3) == 0 ? 1.0f : 0.0f;
+#pragma unroll
+        for (int i = 0; i < DV / 8; i++) o[g][i][0] = o[g][i][1] = o[g][i][2] = o[g][i][3] = 0.0f;
+    }
+    const uint32_t row0 = warp * 32 + lane / 4, see = p0 + t0 + row0;   // last key the first of them sees
+    const uint32_t q_addr = q_sm + ((warp * 32 + lane % 16) * G::LQ + lane / 16 * 8) * 2;
 
     for (uint32_t tile = 0; tile < ntiles; tile++) {
         const uint32_t b = tile & 1;
@@ -102,95 +107,112 @@ __global__ void __launch_bounds__(256, 1) latent_prefill_kernel(const __grid_con
         }
         __syncthreads();
         const uint32_t kt = k_sm + b * (uint32_t)G::K, vt = v_sm + b * (uint32_t)G::V;
-        float sc[PF_KEYS / 8][4];
+        float sc[2][PF_KEYS / 8][4];
 #pragma unroll
-        for (int i = 0; i < PF_KEYS / 8; i++) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.0f;
+        for (int g = 0; g < 2; g++)
+#pragma unroll
+            for (int i = 0; i < PF_KEYS / 8; i++) sc[g][i][0] = sc[g][i][1] = sc[g][i][2] = sc[g][i][3] = 0.0f;
         const uint32_t k_addr = kt + ((lane % 8 + lane / 16 * 8) * G::LQ + (lane / 8 % 2) * 8) * 2;
 #pragma unroll
         for (int kk = 0; kk < DQ / 16; kk++) {
-            uint32_t qa[4];
-            ldsm4(qa, q_addr + kk * 32);
+            uint32_t q0[4], q1[4];
+            ldsm4(q0, q_addr + kk * 32);
+            ldsm4(q1, q_addr + 16 * G::LQ * 2 + kk * 32);
 #pragma unroll
             for (int n = 0; n < PF_KEYS / 16; n++) {
                 uint32_t kb[4];
                 ldsm4(kb, k_addr + (n * 16 * G::LQ + kk * 16) * 2);
-                mma16816(sc[2 * n], qa, kb[0], kb[1]);
-                mma16816(sc[2 * n + 1], qa, kb[2], kb[3]);
+                mma16816(sc[0][2 * n], q0, kb[0], kb[1]);
+                mma16816(sc[0][2 * n + 1], q0, kb[2], kb[3]);
+                mma16816(sc[1][2 * n], q1, kb[0], kb[1]);
+                mma16816(sc[1][2 * n + 1], q1, kb[2], kb[3]);
             }
         }
         const uint32_t j0 = tile * PF_KEYS + (lane & 3) * 2;
-        float top0 = m[0], top1 = m[1];
-        const bool edge = tile * PF_KEYS + PF_KEYS > p0 + t0 + warp * 16;   // some key of the tile is hidden from some row of the warp
+        const bool edge = tile * PF_KEYS + PF_KEYS > p0 + t0 + warp * 32;   // some key of the tile is hidden from some row of the warp
 #pragma unroll
-        for (int i = 0; i < PF_KEYS / 8; i++) {
+        for (int g = 0; g < 2; g++) {
+            float top0 = m[g][0], top1 = m[g][1];
 #pragma unroll
-            for (int e = 0; e < 4; e++) {
-                float v = sc[i][e] * scale;
-                if (edge && j0 + i * 8 + (e & 1) > (e < 2 ? see0 : see1)) v = -INFINITY;
-                sc[i][e] = v;
+            for (int i = 0; i < PF_KEYS / 8; i++) {
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    float v = sc[g][i][e] * scale;
+                    if (edge && j0 + i * 8 + (e & 1) > see + g * 16 + (e < 2 ? 0 : 8)) v = -INFINITY;
+                    sc[g][i][e] = v;
+                }
+                top0 = fmaxf(top0, fmaxf(sc[g][i][0], sc[g][i][1]));
+                top1 = fmaxf(top1, fmaxf(sc[g][i][2], sc[g][i][3]));
             }
-            top0 = fmaxf(top0, fmaxf(sc[i][0], sc[i][1]));
-            top1 = fmaxf(top1, fmaxf(sc[i][2], sc[i][3]));
-        }
 #pragma unroll
-        for (int x = 1; x <= 2; x *= 2) {
-            top0 = fmaxf(top0, __shfl_xor_sync(0xffffffffu, top0, x));
-            top1 = fmaxf(top1, __shfl_xor_sync(0xffffffffu, top1, x));
-        }
-        const float f0 = exp2f(m[0] - top0), f1 = exp2f(m[1] - top1);
-        m[0] = top0; m[1] = top1;
-        l[0] *= f0; l[1] *= f1;
+            for (int x = 1; x <= 2; x *= 2) {
+                top0 = fmaxf(top0, __shfl_xor_sync(0xffffffffu, top0, x));
+                top1 = fmaxf(top1, __shfl_xor_sync(0xffffffffu, top1, x));
+            }
+            const float f0 = exp2f(m[g][0] - top0), f1 = exp2f(m[g][1] - top1);
+            if (__any_sync(0xffffffffu, f0 != 1.0f || f1 != 1.0f)) {
 #pragma unroll
-        for (int i = 0; i < DV / 8; i++) { o[i][0] *= f0; o[i][1] *= f0; o[i][2] *= f1; o[i][3] *= f1; }
+                for (int i = 0; i < DV / 8; i++) { o[g][i][0] *= f0; o[g][i][1] *= f0; o[g][i][2] *= f1; o[g][i][3] *= f1; }
+            }
+            m[g][0] = top0; m[g][1] = top1;
+            l[g][0] *= f0; l[g][1] *= f1;
 #pragma unroll
-        for (int i = 0; i < PF_KEYS / 8; i++) {
-            sc[i][0] = exp2f(sc[i][0] - top0); sc[i][1] = exp2f(sc[i][1] - top0);
-            sc[i][2] = exp2f(sc[i][2] - top1); sc[i][3] = exp2f(sc[i][3] - top1);
-            l[0] += sc[i][0] + sc[i][1]; l[1] += sc[i][2] + sc[i][3];
+            for (int i = 0; i < PF_KEYS / 8; i++) {
+                sc[g][i][0] = exp2f(sc[g][i][0] - top0); sc[g][i][1] = exp2f(sc[g][i][1] - top0);
+                sc[g][i][2] = exp2f(sc[g][i][2] - top1); sc[g][i][3] = exp2f(sc[g][i][3] - top1);
+                l[g][0] += sc[g][i][0] + sc[g][i][1]; l[g][1] += sc[g][i][2] + sc[g][i][3];
+            }
         }
         const uint32_t v_addr = vt + ((lane % 16) * G::LV + lane / 16 * 8) * 2;
 #pragma unroll
         for (int kk = 0; kk < PF_KEYS / 16; kk++) {
-            uint32_t hi[4], lo[4];
+            uint32_t hi[2][4], lo[2][4];
 #pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const float x = sc[2 * kk + e / 2][(e & 1) * 2], y = sc[2 * kk + e / 2][(e & 1) * 2 + 1];
-                hi[e] = pack_bf16(x, y);
-                const float2 r = bf2(hi[e]);
-                lo[e] = pack_bf16(x - r.x, y - r.y);
-            }
+            for (int g = 0; g < 2; g++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    const float x = sc[g][2 * kk + e / 2][(e & 1) * 2], y = sc[g][2 * kk + e / 2][(e & 1) * 2 + 1];
+                    hi[g][e] = pack_bf16(x, y);
+                    const float2 r = bf2(hi[g][e]);
+                    lo[g][e] = pack_bf16(x - r.x, y - r.y);
+                }
 #pragma unroll
             for (int n = 0; n < DV / 16; n++) {
                 uint32_t vb[4];
                 ldsm4t(vb, v_addr + (kk * 16 * G::LV + n * 16) * 2);
-                mma16816(o[2 * n], hi, vb[0], vb[1]);
-                mma16816(o[2 * n + 1], hi, vb[2], vb[3]);
-                mma16816(o[2 * n], lo, vb[0], vb[1]);
-                mma16816(o[2 * n + 1], lo, vb[2], vb[3]);
+#pragma unroll
+                for (int g = 0; g < 2; g++) {
+                    mma16816(o[g][2 * n], hi[g], vb[0], vb[1]);
+                    mma16816(o[g][2 * n + 1], hi[g], vb[2], vb[3]);
+                    mma16816(o[g][2 * n], lo[g], vb[0], vb[1]);
+                    mma16816(o[g][2 * n + 1], lo[g], vb[2], vb[3]);
+                }
             }
         }
         __syncthreads();
     }
 #pragma unroll
-    for (int r = 0; r < 2; r++) {
-        float den = l[r];
-        den += __shfl_xor_sync(0xffffffffu, den, 1);
-        den += __shfl_xor_sync(0xffffffffu, den, 2);
-        const float inv = __frcp_rn(den);
-        const uint32_t row = row0 + 8 * r;
-        if (row >= rows) continue;
-        const float* gate = a.y + (size_t)(t0 + row) * a.ldy + s.off_g + (size_t)h * s.vdim;
-        bf16* out = static_cast<bf16*>(a.out) + (size_t)(t0 + row) * a.ldo;
+    for (int g = 0; g < 2; g++)
 #pragma unroll
-        for (int i = 0; i < DV / 8; i++) {
-            const uint32_t c = i * 8 + (lane & 3) * 2;
-            if (c < s.vdim)
-                *reinterpret_cast<uint32_t*>(out + (size_t)h * s.vdim + c) =
-                    pack_bf16(o[i][2 * r] * inv * sigmoid_f(gate[c]), o[i][2 * r + 1] * inv * sigmoid_f(gate[c + 1]));
+        for (int r = 0; r < 2; r++) {
+            float den = l[g][r];
+            den += __shfl_xor_sync(0xffffffffu, den, 1);
+            den += __shfl_xor_sync(0xffffffffu, den, 2);
+            const float inv = __frcp_rn(den);
+            const uint32_t row = row0 + 16 * g + 8 * r;
+            if (row >= rows) continue;
+            const float* gate = a.y + (size_t)(t0 + row) * a.ldy + s.off_g + (size_t)h * s.vdim + v0;
+            bf16* out = static_cast<bf16*>(a.out) + (size_t)(t0 + row) * a.ldo;
+#pragma unroll
+            for (int i = 0; i < DV / 8; i++) {
+                const uint32_t c = i * 8 + (lane & 3) * 2;
+                if (c < vn)
+                    *reinterpret_cast<uint32_t*>(out + (size_t)h * s.vdim + v0 + c) =
+                        pack_bf16(o[g][i][2 * r] * inv * sigmoid_f(gate[c]), o[g][i][2 * r + 1] * inv * sigmoid_f(gate[c + 1]));
+            }
+            if (h + 1 == s.heads)   // padding up to the stride
+                for (uint32_t c = s.heads * s.vdim + (lane & 3); c < a.ldo; c += 4) out[c] = __float2bfloat16_rn(0.0f);
         }
-        if (h + 1 == s.heads)   // padding up to the stride
-            for (uint32_t c = s.heads * s.vdim + (lane & 3); c < a.ldo; c += 4) out[c] = __float2bfloat16_rn(0.0f);
-    }
 }
 
 template <int DQ, int DV>
@@ -198,7 +220,7 @@ cudaError_t prefill_inst(const LatentArgs& a, uint32_t tokens, cudaStream_t st, 
     static bool done[64] = {};
     const cudaError_t err = allow_smem(latent_prefill_kernel<DQ, DV>, PfGeom<DQ, DV>::SMEM, done);
     if (err != cudaSuccess) return err;
-    return launch_pdl(latent_prefill_kernel<DQ, DV>, dim3(a.s.heads, (tokens + PF_ROWS - 1) / PF_ROWS), dim3(256), PfGeom<DQ, DV>::SMEM, st, pdl, a, tokens);
+    return launch_pdl(latent_prefill_kernel<DQ, DV>, dim3(a.s.heads, (tokens + PF_ROWS - 1) / PF_ROWS, (a.s.vdim + DV - 1) / DV), dim3(PF_THREADS), PfGeom<DQ, DV>::SMEM, st, pdl, a, tokens);
 }
 
 }  // namespace
@@ -208,8 +230,8 @@ cudaError_t launch_latent_prefill(const LatentArgs& a, uint32_t tokens, cudaStre
     const uint32_t q = a.s.dim + a.s.rot, v = a.s.vdim;
     if (q <= 64 && v <= 64) return prefill_inst<64, 64>(a, tokens, st, pdl);
     if (q <= 128 && v <= 128) return prefill_inst<128, 128>(a, tokens, st, pdl);
-    if (q <= 192 && v <= 128) return prefill_inst<192, 128>(a, tokens, st, pdl);
-    return prefill_inst<256, 256>(a, tokens, st, pdl);
+    if (q <= 192) return prefill_inst<192, 128>(a, tokens, st, pdl);
+    return prefill_inst<256, 128>(a, tokens, st, pdl);
 }
 
 }  // namespace alice
