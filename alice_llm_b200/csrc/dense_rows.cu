@@ -1,8 +1,7 @@
-// One token against dense bfloat16 rows. A warp owns R consecutive rows at a time; every lane streams 16-byte pieces of
-// each (R times the unroll factor in flight; two CTAs of eight warps per SM are enough, which leaves room for the CTAs of the
-// next kernel), the input sits in shared memory as f32. The rows a warp starts with are
-// requested into L2 before the wait for the producing kernel, so under programmatic dependent launch the weights travel
-// while the input is still being made.
+// One token against dense bfloat16 rows. A warp owns R consecutive rows at a time; every lane requests 16-byte pieces in batches
+// of R * 8, so two CTAs of eight warps per SM keep enough bytes in flight and leave room for the CTAs of the next kernel. The
+// input sits in shared memory as f32. The beginning of the rows a warp starts with is requested into L2 before the wait for the
+// producing kernel (a longer prefetch made the stream slower: 4096 x 18432 in 28.7 us without, 34.9 us with whole rows).
 #include "dense_dev.cuh"
 
 namespace alice {
@@ -11,24 +10,37 @@ namespace {
 constexpr int RT = 256, RW = RT / 32;
 
 template <int R, int U>
+__device__ __forceinline__ void dot_batches(const bf16* const (&w)[R], const float* xs, uint32_t& c, uint32_t k, float (&acc)[R]) {
+    for (; c + (U - 1) * 256 < k; c += U * 256) {
+        uint4 v[U][R];
+#pragma unroll
+        for (int u = 0; u < U; u++)
+#pragma unroll
+            for (int r = 0; r < R; r++) v[u][r] = __ldg(reinterpret_cast<const uint4*>(w[r] + c + u * 256));
+#pragma unroll
+        for (int u = 0; u < U; u++) {
+            const float4 x0 = *reinterpret_cast<const float4*>(xs + c + u * 256), x1 = *reinterpret_cast<const float4*>(xs + c + u * 256 + 4);
+#pragma unroll
+            for (int r = 0; r < R; r++) acc[r] = dot8(v[u][r], x0, x1, acc[r]);
+        }
+    }
+}
+// acc[r] = w[r][0 .. k) . xs[0 .. k), the same in every lane
+template <int R>
 __device__ __forceinline__ void dot_rows(const bf16* const (&w)[R], const float* xs, uint32_t k, uint32_t lane, float (&acc)[R]) {
 #pragma unroll
     for (int r = 0; r < R; r++) acc[r] = 0.0f;
-#pragma unroll U
-    for (uint32_t c = lane * 8; c < k; c += 256) {
-        uint4 v[R];
-#pragma unroll
-        for (int r = 0; r < R; r++) v[r] = __ldg(reinterpret_cast<const uint4*>(w[r] + c));
-        const float4 x0 = *reinterpret_cast<const float4*>(xs + c), x1 = *reinterpret_cast<const float4*>(xs + c + 4);
-#pragma unroll
-        for (int r = 0; r < R; r++) acc[r] = dot8(v[r], x0, x1, acc[r]);
-    }
+    uint32_t c = lane * 8;
+    dot_batches<R, 8>(w, xs, c, k, acc);
+    dot_batches<R, 4>(w, xs, c, k, acc);
+    dot_batches<R, 2>(w, xs, c, k, acc);
+    dot_batches<R, 1>(w, xs, c, k, acc);
 #pragma unroll
     for (int r = 0; r < R; r++) acc[r] = warp_sum(acc[r]);
 }
 
 __device__ __forceinline__ void prefetch_row(const bf16* w, uint32_t k, uint32_t lane) {
-    for (uint32_t c = lane * 64; c < k; c += 32 * 64) prefetch_l2(w + c);
+    if (lane * 64 < k) prefetch_l2(w + lane * 64);
 }
 
 // order-preserving image of a float, as the output head's argmax packs it
@@ -80,7 +92,7 @@ __global__ void __launch_bounds__(RT, 2) rows_in_kernel(const __grid_constant__ 
     for (uint32_t item = w_id; item < items; item += warps) {
         item_rows<R>(op, item, items0, w, first, pair);
         float acc[R];
-        dot_rows<R, 4>(w, xs, k, lane, acc);
+        dot_rows<R>(w, xs, k, lane, acc);
         if (!pair) {
 #pragma unroll
             for (int r = 0; r < R; r++) {
@@ -97,32 +109,55 @@ __global__ void __launch_bounds__(RT, 2) rows_in_kernel(const __grid_constant__ 
     if (op.argmax_key && lane == 0 && best) atomicMax(op.argmax_key, best);
 }
 
-// A warp owns one row of [W1 | W2] at a time; the CTA has as many warps as spread the rows evenly over two CTAs per SM.
-constexpr int OUT_MAX_WARPS = 16;
-__global__ void __launch_bounds__(OUT_MAX_WARPS * 32, 2) rows_out_kernel(const __grid_constant__ RowsOut op) {
+template <int R>
+__global__ void __launch_bounds__(RT, 2) rows_out_kernel(const __grid_constant__ RowsOut op) {
     extern __shared__ __align__(16) float xs[];
-    const uint32_t lane = threadIdx.x & 31, nw = blockDim.x >> 5, warps = gridDim.x * nw, w_id = blockIdx.x + (threadIdx.x >> 5) * gridDim.x;
-    const uint32_t n = op.w1.n, k1 = op.w1.k, k2 = op.w2.n ? op.w2.k : 0;
+    const uint32_t lane = threadIdx.x & 31, warps = gridDim.x * RW, w_id = blockIdx.x + (threadIdx.x >> 5) * gridDim.x;
+    const uint32_t n = op.w1.n, k1 = op.w1.k, k2 = op.w2.n ? op.w2.k : 0, items = (n + R - 1) / R;
     pdl_launch_dependents();
-    if (w_id < n) {
-        prefetch_row(op.w1.w + (size_t)w_id * k1, k1, lane);
-        if (k2) prefetch_row(op.w2.w + (size_t)w_id * k2, k2, lane);
-    }
+    if (w_id < items)
+#pragma unroll
+        for (int r = 0; r < R; r++) {
+            const uint32_t row = min(w_id * R + r, n - 1);
+            prefetch_row(op.w1.w + (size_t)row * k1, k1, lane);
+            if (k2) prefetch_row(op.w2.w + (size_t)row * k2, k2, lane);
+        }
     pdl_wait();
-    for (uint32_t i = threadIdx.x * 4; i < k1; i += blockDim.x * 4) *reinterpret_cast<float4*>(xs + i) = __ldcg(reinterpret_cast<const float4*>(op.a + i));
-    for (uint32_t i = threadIdx.x * 4; i < k2; i += blockDim.x * 4) *reinterpret_cast<float4*>(xs + k1 + i) = __ldcg(reinterpret_cast<const float4*>(op.f + i));
+    for (uint32_t i = threadIdx.x * 4; i < k1; i += RT * 4) *reinterpret_cast<float4*>(xs + i) = __ldcg(reinterpret_cast<const float4*>(op.a + i));
+    for (uint32_t i = threadIdx.x * 4; i < k2; i += RT * 4) *reinterpret_cast<float4*>(xs + k1 + i) = __ldcg(reinterpret_cast<const float4*>(op.f + i));
     __syncthreads();
-    for (uint32_t row = w_id; row < n; row += warps) {
-        const bf16 *const u[1] = {op.w1.w + (size_t)row * k1}, *const d[1] = {op.w2.w + (size_t)row * k2};
-        float acc1[1], acc2[1] = {0.0f};
-        if (k2) dot_rows<1, 8>(d, xs + k1, k2, lane, acc2);
-        dot_rows<1, 8>(u, xs, k1, lane, acc1);
-        if (lane == 0) {
-            float v = op.s1[row] * acc1[0];
-            if (k2) v += op.s2[row] * (acc2[0] + op.b2[row]);
-            op.x[row] += v;
+    for (uint32_t item = w_id; item < items; item += warps) {
+        const bf16 *u[R], *d[R];
+#pragma unroll
+        for (int r = 0; r < R; r++) {
+            const uint32_t row = min(item * R + r, n - 1);
+            u[r] = op.w1.w + (size_t)row * k1;
+            d[r] = op.w2.w + (size_t)row * k2;
+        }
+        float acc1[R], acc2[R];
+#pragma unroll
+        for (int r = 0; r < R; r++) acc2[r] = 0.0f;
+        if (k2) dot_rows<R>(d, xs + k1, k2, lane, acc2);
+        dot_rows<R>(u, xs, k1, lane, acc1);
+#pragma unroll
+        for (int r = 0; r < R; r++) {
+            const uint32_t row = item * R + r;
+            if (lane == (uint32_t)r && row < n) {
+                float v = op.s1[row] * acc1[r];
+                if (k2) v += op.s2[row] * (acc2[r] + op.b2[row]);
+                op.x[row] += v;
+            }
         }
     }
+}
+
+template <int R>
+cudaError_t rows_out_r(const RowsOut& op, int num_sms, cudaStream_t st, bool pdl) {
+    static bool done[64] = {};
+    const cudaError_t err = allow_smem(rows_out_kernel<R>, 224 * 1024, done);
+    if (err != cudaSuccess) return err;
+    const uint32_t items = (op.w1.n + R - 1) / R, grid = std::min<uint32_t>((items + RW - 1) / RW, (uint32_t)num_sms * 2);
+    return launch_pdl(rows_out_kernel<R>, dim3(grid), dim3(RT), (size_t)(op.w1.k + (op.w2.n ? op.w2.k : 0)) * 4, st, pdl, op);
 }
 
 template <int R>
@@ -138,21 +173,13 @@ cudaError_t rows_in_r(const RowsIn& op, int num_sms, cudaStream_t st, bool pdl) 
 
 cudaError_t launch_rows_in(const RowsIn& op, int num_sms, cudaStream_t st, bool pdl) {
     if (!op.w0.n || op.w0.k % DENSE_PAD || (op.gu.n && (op.gu.k != op.w0.k || op.gu.n % 128)) || (size_t)op.w0.k * 4 > 220 * 1024) return cudaErrorInvalidValue;
-    // enough items to give every SM two dozen warps: fewer rows per warp for the small matrices
-    if (op.w0.n + op.gu.n >= (uint32_t)num_sms * 24 * 4) return rows_in_r<4>(op, num_sms, st, pdl);
     return rows_in_r<2>(op, num_sms, st, pdl);
 }
 
 cudaError_t launch_rows_out(const RowsOut& op, int num_sms, cudaStream_t st, bool pdl) {
     if (!op.w1.n || op.w1.k % DENSE_PAD || (op.w2.n && (op.w2.n != op.w1.n || op.w2.k % DENSE_PAD))) return cudaErrorInvalidValue;
     if ((size_t)(op.w1.k + (op.w2.n ? op.w2.k : 0)) * 4 > 220 * 1024) return cudaErrorInvalidValue;
-    static bool done[64] = {};
-    const cudaError_t err = allow_smem(rows_out_kernel, 224 * 1024, done);
-    if (err != cudaSuccess) return err;
-    const uint32_t slots = (uint32_t)num_sms * 2, rounds = (op.w1.n + slots * OUT_MAX_WARPS - 1) / (slots * OUT_MAX_WARPS);
-    const uint32_t nw = std::min<uint32_t>(OUT_MAX_WARPS, std::max<uint32_t>(4, (op.w1.n + slots * rounds - 1) / (slots * rounds)));
-    const uint32_t grid = std::min(slots, (op.w1.n + nw - 1) / nw);
-    return launch_pdl(rows_out_kernel, dim3(grid), dim3(nw * 32), (size_t)(op.w1.k + (op.w2.n ? op.w2.k : 0)) * 4, st, pdl, op);
+    return op.w1.n >= (uint32_t)num_sms * 16 ? rows_out_r<2>(op, num_sms, st, pdl) : rows_out_r<1>(op, num_sms, st, pdl);
 }
 
 }  // namespace alice
