@@ -26,7 +26,6 @@ __global__ void __launch_bounds__(PF_THREADS, 2) latent_prefill_kernel(const __g
     const LatentShape& s = a.s;
     const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x;
     const uint32_t t0 = (gridDim.y - 1 - blockIdx.y) * PF_ROWS;   // the longest rows first
-    auto* qs = reinterpret_cast<bf16*>(sm);
     const uint32_t q_sm = smem_u32(sm), k_sm = q_sm + (uint32_t)G::Q, v_sm = k_sm + 2 * (uint32_t)G::K;
     pdl_launch_dependents();
     pdl_wait();
@@ -45,43 +44,24 @@ __global__ void __launch_bounds__(PF_THREADS, 2) latent_prefill_kernel(const __g
         const uint32_t r = i / (DV - vn), c = vn + i % (DV - vn);
         reinterpret_cast<bf16*>(sm + G::Q + 2 * G::K + (r / PF_KEYS) * G::V)[(r % PF_KEYS) * G::LV + c] = __float2bfloat16_rn(0.0f);
     }
+    // rows of 16-byte pieces, a few threads a row
+    constexpr uint32_t TPR = PF_THREADS / PF_KEYS;
+    const uint32_t fr = tid / TPR, fc = tid % TPR, nd = s.dim / 8, nr = s.rot / 8, nv = vn / 8;
     auto fetch = [&](uint32_t tile, uint32_t b) {
-        const uint32_t j0 = tile * PF_KEYS, nd = s.dim / 8, nr = s.rot / 8, nv = vn / 8;
-        const uint32_t kd = k_sm + b * (uint32_t)G::K, vd = v_sm + b * (uint32_t)G::V;
-        for (uint32_t i = tid; i < PF_KEYS * nd; i += PF_THREADS) {
-            const uint32_t r = i / nd, c = i % nd * 8, j = min(j0 + r, keys - 1);
-            cp16(kd + (r * G::LQ + c) * 2, a.k_all + (size_t)j * kw + (size_t)h * s.dim + c, j0 + r < keys);
-        }
-        for (uint32_t i = tid; i < PF_KEYS * nr; i += PF_THREADS) {
-            const uint32_t r = i / nr, c = i % nr * 8, j = min(j0 + r, keys - 1);
-            cp16(kd + (r * G::LQ + s.dim + c) * 2, cache + (size_t)j * cw + s.cp + c, j0 + r < keys);
-        }
-        for (uint32_t i = tid; i < PF_KEYS * nv; i += PF_THREADS) {
-            const uint32_t r = i / nv, c = i % nv * 8, j = min(j0 + r, keys - 1);
-            cp16(vd + (r * G::LV + c) * 2, a.v_all + (size_t)j * vw + (size_t)h * s.vdim + v0 + c, j0 + r < keys);
-        }
+        const uint32_t j = min(tile * PF_KEYS + fr, keys - 1);
+        const bool ok = tile * PF_KEYS + fr < keys;
+        const uint32_t kd = k_sm + b * (uint32_t)G::K + fr * G::LQ * 2, vd = v_sm + b * (uint32_t)G::V + fr * G::LV * 2;
+        const bf16 *kp = a.k_all + (size_t)j * kw + (size_t)h * s.dim, *rp = cache + (size_t)j * cw + s.cp, *vp = a.v_all + (size_t)j * vw + (size_t)h * s.vdim + v0;
+        for (uint32_t c = fc; c < nd; c += TPR) cp16(kd + c * 16, kp + c * 8, ok);
+        for (uint32_t c = fc; c < nr; c += TPR) cp16(kd + (nd + c) * 16, rp + c * 8, ok);
+        for (uint32_t c = fc; c < nv; c += TPR) cp16(vd + c * 16, vp + c * 8, ok);
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    fetch(0, 0);
-    // queries, the rotated part turned to its position on the way
-    const uint32_t half = s.rot_dims / 2;
-    for (uint32_t i = tid; i < PF_ROWS * DQ; i += PF_THREADS) {
-        const uint32_t r = i / DQ, c = i % DQ;
-        float v = 0.0f;
-        if (r < rows && c < qd) {
-            const float* q = a.q + ((size_t)(t0 + r) * s.heads + h) * qd;
-            if (c >= s.dim && c < s.dim + s.rot_dims) {
-                const uint32_t d = c - s.dim, j = d < half ? d : d - half;
-                float sn, cs;
-                sincosf((float)(p0 + t0 + r) * a.freq[j], &sn, &cs);
-                const float x = q[s.dim + j], y = q[s.dim + half + j];
-                v = d < half ? x * cs - y * sn : y * cs + x * sn;
-            } else {
-                v = q[c];
-            }
-        }
-        qs[r * G::LQ + c] = __float2bfloat16_rn(v);
+    for (uint32_t r = fr; r < PF_ROWS; r += PF_KEYS) {   // queries, part of the first copy group
+        const bf16* q = a.q_rot + ((size_t)(t0 + min(r, rows - 1)) * s.heads + h) * qd;
+        for (uint32_t c = fc; c < DQ / 8; c += TPR) cp16(q_sm + r * G::LQ * 2 + c * 16, q + min(c * 8, qd - 8), r < rows && c * 8 < qd);
     }
+    fetch(0, 0);
 
     // a thread's rows are lane / 4 and lane / 4 + 8 of each of its warp's two 16-row tiles
     constexpr float LOG2E = 1.4426950408889634f;
@@ -215,6 +195,38 @@ __global__ void __launch_bounds__(PF_THREADS, 2) latent_prefill_kernel(const __g
         }
 }
 
+// Queries in bf16 with the rotated part turned to its position. One CTA per token.
+__global__ void __launch_bounds__(256) latent_rotate_kernel(const __grid_constant__ LatentArgs a, bf16* out) {
+    extern __shared__ float2 cs[];   // (cos, sin) per pair
+    const LatentShape& s = a.s;
+    const uint32_t t = blockIdx.x, half = s.rot_dims / 2, qd = s.dim + s.rot, n = s.heads * qd;
+    pdl_launch_dependents();
+    pdl_wait();
+    const float p = (float)((uint32_t)*a.pos + t);
+    for (uint32_t i = threadIdx.x; i < half; i += 256) {
+        float sn, c;
+        sincosf(p * a.freq[i], &sn, &c);
+        cs[i] = make_float2(c, sn);
+    }
+    __syncthreads();
+    const float* q = a.q + (size_t)t * n;
+    for (uint32_t i = threadIdx.x * 2; i < n; i += 512) {   // head sizes are even
+        float v[2];
+        const uint32_t c = i % qd;
+        const float2 x = *reinterpret_cast<const float2*>(q + i);
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+            v[e] = e ? x.y : x.x;
+            if (c + e >= s.dim && c + e < s.dim + s.rot_dims) {
+                const uint32_t d = c + e - s.dim;
+                if (d < half) v[e] = v[e] * cs[d].x - q[i + e + half] * cs[d].y;
+                else v[e] = v[e] * cs[d - half].x + q[i + e - half] * cs[d - half].y;
+            }
+        }
+        *reinterpret_cast<uint32_t*>(out + (size_t)t * n + i) = pack_bf16(v[0], v[1]);
+    }
+}
+
 template <int DQ, int DV>
 cudaError_t prefill_inst(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
     static bool done[64] = {};
@@ -228,6 +240,8 @@ cudaError_t prefill_inst(const LatentArgs& a, uint32_t tokens, cudaStream_t st, 
 cudaError_t launch_latent_prefill(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
     if (!latent_prefill_fits(a.s) || !a.cache_bf16 || !a.act_bf16) return cudaErrorInvalidValue;
     const uint32_t q = a.s.dim + a.s.rot, v = a.s.vdim;
+    const cudaError_t err = launch_pdl(latent_rotate_kernel, dim3(tokens), dim3(256), (size_t)(a.s.rot_dims / 2) * sizeof(float2), st, pdl, a, a.q_rot);
+    if (err != cudaSuccess) return err;
     if (q <= 64 && v <= 64) return prefill_inst<64, 64>(a, tokens, st, pdl);
     if (q <= 128 && v <= 128) return prefill_inst<128, 128>(a, tokens, st, pdl);
     if (q <= 192) return prefill_inst<192, 128>(a, tokens, st, pdl);

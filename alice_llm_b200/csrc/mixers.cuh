@@ -105,6 +105,7 @@ struct LatentArgs {
     uint32_t ldo = 0;
     // tiled prefill: keys and values of every cached token, made from the latent rows
     const bf16 *k_all = nullptr, *v_all = nullptr;   // [ctx][heads * dim], [ctx][heads * vdim]
+    bf16* q_rot = nullptr;                           // [t][heads * (dim + rot)], room for the rotated queries
 };
 // Whether the tensor-core prefill covers these sizes (others take the latent-space path).
 inline bool latent_prefill_fits(const LatentShape& s) {

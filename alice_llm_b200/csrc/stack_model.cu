@@ -34,7 +34,7 @@ struct Scratch {
     // latent
     float *q = nullptr, *ql = nullptr, *part = nullptr, *mix = nullptr;
     void* cqn = nullptr;
-    bf16 *k_all = nullptr, *v_all = nullptr;         // keys and values of the whole context (tiled prefill)
+    bf16 *k_all = nullptr, *v_all = nullptr, *q_rot = nullptr;   // keys and values of the whole context and rotated queries (tiled prefill)
     // delta
     float *qn = nullptr, *kn = nullptr, *pair_inv = nullptr, *pair_b = nullptr, *v = nullptr, *beta = nullptr, *g = nullptr, *gate = nullptr, *o = nullptr;
     bf16* low = nullptr;                             // bf16 copy of the low-rank columns
@@ -144,7 +144,7 @@ struct LatentMixer final : Mixer {
             op.w = uv; op.out = s.v_all; op.ldo = uv.n;
             if (!erc) erc = m->product(op);
             if (erc) return erc;
-            a.k_all = s.k_all; a.v_all = s.v_all;
+            a.k_all = s.k_all; a.v_all = s.v_all; a.q_rot = s.q_rot;
             MCU(launch_latent_prefill(a, n, st, pdl));
             return ALICE_OK;
         }
@@ -459,6 +459,7 @@ void build_scratch(Builder& b) {
     s.part = b.zeros<float>((size_t)std::max(ML, DECODE_SPLITS) * part);
     s.mix = b.zeros<float>((size_t)ML * mix);
     s.k_all = b.zeros<bf16>((size_t)m->max_seq * k_all);
+    s.q_rot = b.zeros<bf16>(k_all ? (size_t)M * q : 0);
     s.v_all = b.zeros<bf16>((size_t)m->max_seq * v_all);
     s.qn = b.zeros<float>((size_t)M * kd); s.kn = b.zeros<float>((size_t)M * kd);
     s.pair_inv = b.zeros<float>((size_t)M * h * DELTA_BLOCK); s.pair_b = b.zeros<float>((size_t)M * h * DELTA_BLOCK);
