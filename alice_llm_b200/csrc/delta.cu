@@ -611,7 +611,7 @@ cudaError_t launch_delta_scan(const DeltaArgs& a, uint32_t tokens, cudaStream_t 
 }
 
 cudaError_t launch_delta_step(const DeltaStepArgs& a, cudaStream_t st, bool pdl) {
-    if (!delta_step_fits(a.d.s) || (size_t)(a.a2.k + a.g2.k) * 4 > 32 * 1024) return cudaErrorInvalidValue;
+    if (!delta_step_fits(a)) return cudaErrorInvalidValue;
     switch (a.d.s.dp) {
         case 64: return step_e<8>(a, st, pdl);
         case 128: return step_e<16>(a, st, pdl);

@@ -300,6 +300,7 @@ cudaError_t attn_type(const LatentArgs& a, uint32_t tokens, cudaStream_t st, boo
     const bool few = a.s.heads <= 8;
     if (a.s.cp <= 128) return few ? attn_inst<CT, 1, 4>(a, tokens, st, pdl) : attn_inst<CT, 4, 4>(a, tokens, st, pdl);
     if (a.s.cp <= 512) return few ? attn_inst<CT, 1, 16>(a, tokens, st, pdl) : attn_inst<CT, 4, 16>(a, tokens, st, pdl);
+    if (a.s.cp <= 1024) return attn_inst<CT, 1, 32>(a, tokens, st, pdl);
     return cudaErrorInvalidValue;
 }
 

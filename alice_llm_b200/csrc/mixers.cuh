@@ -71,7 +71,7 @@ struct DeltaStepArgs {
     uint32_t off_a = 0, off_g = 0;    // columns of their low-rank inputs in y
     const float *a_log = nullptr, *dt_bias = nullptr;
 };
-inline bool delta_step_fits(const DeltaShape& s) { return s.vp <= 256; }
+inline bool delta_step_fits(const DeltaStepArgs& a) { return a.d.s.vp <= 256 && a.a2.k + a.g2.k <= 8192; }
 cudaError_t launch_delta_step(const DeltaStepArgs& a, cudaStream_t st, bool pdl);
 
 // ---- latent.cu: attention over a cached latent ---------------------------------------------------
@@ -81,7 +81,7 @@ struct LatentShape {
     uint32_t off_q, off_kv, off_g;    // columns of the projection output
     float scale;
 };
-constexpr uint32_t LATENT_MAX_RANK = 512;
+constexpr uint32_t LATENT_MAX_RANK = 1024;
 
 struct LatentArgs {
     LatentShape s;

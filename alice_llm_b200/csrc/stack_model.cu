@@ -181,9 +181,9 @@ struct DeltaMixer final : Mixer {
         a.s = sh; a.y = s.y; a.ldy = s.ldy; a.conv_w = conv; a.conv_state = states[pass].conv; a.state = states[pass].s;
         a.qn = s.qn; a.kn = s.kn; a.pair_inv = s.pair_inv; a.pair_b = s.pair_b; a.v = s.v; a.beta = s.beta; a.g = s.g; a.o = s.o; a.gate = s.gate; a.norm_w = norm; a.eps = m->cfg.eps;
         a.out = s.a; a.ldo = o.k; a.out_bf16 = low; a.pos = m->d_pos;
-        if (n == 1 && delta_step_fits(sh)) {
-            DeltaStepArgs sa;
-            sa.d = a; sa.a2 = a2; sa.g2 = g2; sa.off_a = off_a; sa.off_g = off_g; sa.a_log = a_log; sa.dt_bias = dt_bias;
+        DeltaStepArgs sa;
+        sa.d = a; sa.a2 = a2; sa.g2 = g2; sa.off_a = off_a; sa.off_g = off_g; sa.a_log = a_log; sa.dt_bias = dt_bias;
+        if (n == 1 && delta_step_fits(sa)) {
             MCU(launch_delta_step(sa, st, pdl));
             return ALICE_OK;
         }
@@ -376,7 +376,7 @@ void build_latent(Builder& b, const alice_stack_layer& L, uint32_t wp, uint32_t 
     LatentShape& s = mx.sh;
     if (!L.heads || !L.dim || !L.vdim || !L.q_rank || !L.kv_rank) return b.shape("latent mixer with a zero size");
     if (L.rot_dims % 2 || L.rot_dims > L.rot_dim) return b.shape("rotated dimensions must be even and lie within rot_dim");
-    if (L.kv_rank > LATENT_MAX_RANK) return b.shape("kv_rank above 512");
+    if (L.kv_rank > LATENT_MAX_RANK) return b.shape("kv_rank above 1024");
     s.heads = L.heads; s.dim = L.dim; s.rot = L.rot_dim; s.rot_dims = L.rot_dims; s.vdim = L.vdim; s.q_rank = L.q_rank; s.kv_rank = L.kv_rank;
     s.qp = P(L.q_rank); s.cp = P(L.kv_rank); s.rp = pad_to(L.rot_dim, 16); s.scale = L.scale;
     s.off_q = 0; s.off_kv = s.qp; s.off_g = s.off_kv + P(L.kv_rank + L.rot_dim);

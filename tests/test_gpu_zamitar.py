@@ -65,6 +65,8 @@ ALONE = {
     "latent attention, 128 / 128": zm.config([zm.latent(heads=3, dim=72, rot=56, vdim=128, ff=0)]),
     "latent attention, 192 / 128": zm.config([zm.latent(heads=3, dim=128, rot=64, vdim=112, kv_rank=500, ff=0)]),
     "latent attention, 256 / 256": zm.config([zm.latent(heads=2, dim=200, rot=48, vdim=248, ff=0)]),
+    "latent attention, a latent of 600": zm.config([zm.latent(heads=3, kv_rank=600, ff=0)]),
+    "latent attention, wide rotated part": zm.config([zm.latent(heads=2, dim=8, rot=128, kv_rank=512, ff=0)]),
     "delta rule": zm.config([zm.delta(ff=0)]),
     "delta rule, one tap": zm.config([zm.delta(conv=1, ff=0)]),
     "delta rule, seven taps": zm.config([zm.delta(conv=7, ff=0)]),
