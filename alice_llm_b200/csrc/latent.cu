@@ -219,11 +219,13 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const __grid_constant_
     }
 }
 
-// Joins the shares of the context and the sink: weighted latent of every head. grid (heads, cp / 64, tokens), 64 threads.
-__global__ void __launch_bounds__(64) latent_join_kernel(const __grid_constant__ LatentArgs a) {
+// Joins the shares of the context and the sink: weighted latent of every head. grid (heads, cp / 64, tokens), 256 threads: 64
+// columns, the shares dealt to four groups.
+__global__ void __launch_bounds__(256) latent_join_kernel(const __grid_constant__ LatentArgs a) {
     extern __shared__ float wt[];   // one weight per share
+    __shared__ float sum[4][64];
     const LatentShape& s = a.s;
-    const uint32_t h = blockIdx.x, t = blockIdx.z, lane = threadIdx.x & 31, c = blockIdx.y * 64 + threadIdx.x;
+    const uint32_t h = blockIdx.x, t = blockIdx.z, lane = threadIdx.x & 31, g = threadIdx.x >> 6, c = blockIdx.y * 64 + (threadIdx.x & 63);
     pdl_launch_dependents();
     pdl_wait();
     const float* part = a.part + ((size_t)t * a.splits * s.heads + h) * (s.cp + 2);
@@ -247,11 +249,13 @@ __global__ void __launch_bounds__(64) latent_join_kernel(const __grid_constant__
     __syncthreads();
     float v = 0.0f;
 #pragma unroll 16
-    for (uint32_t k = 0; k < shares; k++) {
+    for (uint32_t k = g; k < shares; k += 4) {
         const float x = part[k * step + c], w = wt[k];
         v = w != 0.0f ? fmaf(w, x, v) : v;   // an empty share holds no sums
     }
-    a.mix[((size_t)t * s.heads + h) * s.cp + c] = v;
+    sum[g][threadIdx.x & 63] = v;
+    __syncthreads();
+    if (g == 0) a.mix[((size_t)t * s.heads + h) * s.cp + c] = (sum[0][threadIdx.x] + sum[1][threadIdx.x]) + (sum[2][threadIdx.x] + sum[3][threadIdx.x]);
 }
 
 // Value rows of the weighted latent and the output gate. grid (heads, groups of 16 rows, tokens), 8 warps of two rows.
@@ -322,7 +326,7 @@ cudaError_t launch_latent_attn(const LatentArgs& a, uint32_t tokens, cudaStream_
     return a.cache_bf16 ? attn_type<bf16>(a, tokens, st, pdl) : attn_type<float>(a, tokens, st, pdl);
 }
 cudaError_t launch_latent_out(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
-    const cudaError_t err = launch_pdl(latent_join_kernel, dim3(a.s.heads, a.s.cp / 64, tokens), dim3(64), (size_t)a.splits * 4, st, pdl, a);
+    const cudaError_t err = launch_pdl(latent_join_kernel, dim3(a.s.heads, a.s.cp / 64, tokens), dim3(256), (size_t)a.splits * 4, st, pdl, a);
     if (err != cudaSuccess) return err;
     const dim3 grid(a.s.heads, (a.s.vdim + 15) / 16, tokens);
     return a.act_bf16 ? launch_pdl(latent_value_kernel<bf16>, grid, dim3(256), (size_t)a.s.cp * 4, st, pdl, a)

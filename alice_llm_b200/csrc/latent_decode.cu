@@ -8,20 +8,20 @@
 namespace alice {
 namespace {
 
-constexpr uint32_t LD_KEYS = 64, LD_HEADS = 16;
+constexpr uint32_t LD_KEYS = 32, LD_HEADS = 16, LD_STAGES = 2;   // a deeper ring measured no faster
 
 // grid (head groups of 16, splits, tokens), 8 warps. NT: 8-column tiles of the weighted sum per warp (8 * NT * 8 >= cp).
 template <int NT>
 __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const __grid_constant__ LatentArgs a) {
     extern __shared__ __align__(128) uint8_t sm[];
-    __shared__ float sc[LD_HEADS][LD_KEYS + 4], mrow[LD_HEADS], lrow[LD_HEADS], frow[LD_HEADS];
+    __shared__ float sc[2][LD_HEADS][LD_KEYS + 4], mrow[LD_HEADS], lrow[LD_HEADS], frow[LD_HEADS];
     __shared__ __align__(16) bf16 ph[LD_HEADS][LD_KEYS + 8], pl[LD_HEADS][LD_KEYS + 8];
     const LatentShape& s = a.s;
     const uint32_t width = s.cp + s.rp, ld = width + 8;   // row stride: eight rows in different banks (width is a multiple of 16)
     const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, t = blockIdx.z, h0 = blockIdx.x * LD_HEADS;
     auto* qh = reinterpret_cast<bf16*>(sm);
     bf16* ql = qh + LD_HEADS * ld;
-    bf16* kt = ql + LD_HEADS * ld;                        // two tiles of [64][ld]
+    bf16* kt = ql + LD_HEADS * ld;                        // LD_STAGES tiles of [LD_KEYS][ld]
     const uint32_t qh_s = smem_u32(qh), ql_s = smem_u32(ql), kt_s = smem_u32(kt), tile_bytes = LD_KEYS * ld * 2;
     pdl_launch_dependents();
     pdl_wait();
@@ -35,20 +35,29 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const __grid_cons
     }
     const bf16* cache = static_cast<const bf16*>(a.cache);
     auto fetch = [&](uint32_t k0, uint32_t b) {
-        const uint32_t nc = width / 8;
-        for (uint32_t i = tid; i < LD_KEYS * nc; i += 256) {
-            const uint32_t r = i / nc, c = i % nc * 8, j = min(k0 + r, hi - 1);
-            cp16(kt_s + b * tile_bytes + (r * ld + c) * 2, cache + (size_t)j * width + c, k0 + r < hi);
-        }
+        const uint32_t row = tid / 8, j = min(k0 + row, hi - 1);   // eight threads a row
+        const bf16* src = cache + (size_t)j * width;
+        const uint32_t dst = kt_s + b * tile_bytes + row * ld * 2;
+        if (k0 < hi)
+            for (uint32_t c = tid % 8 * 8; c < width; c += 64) cp16(dst + c * 2, src + c, k0 + row < hi);
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    fetch(lo, 0);
-    for (uint32_t i = tid; i < LD_HEADS * width; i += 256) {
-        const uint32_t r = i / width, c = i % width;
-        const float v = h0 + r < s.heads ? a.ql[((size_t)t * s.heads + h0 + r) * width + c] * s.scale : 0.0f;
-        const bf16 b = __float2bfloat16_rn(v);
-        qh[r * ld + c] = b;
-        ql[r * ld + c] = __float2bfloat16_rn(v - __bfloat162float(b));
+#pragma unroll
+    for (uint32_t i = 0; i + 1 < LD_STAGES; i++) fetch(lo + i * LD_KEYS, i);
+    static_assert(LD_KEYS * 8 == 256, "a tile is fetched in one round of rows");
+#pragma unroll
+    for (uint32_t r = warp; r < LD_HEADS; r += 8) {
+        const float* q = a.ql + ((size_t)t * s.heads + min(h0 + r, s.heads - 1)) * width;
+        const float f = h0 + r < s.heads ? s.scale : 0.0f;
+#pragma unroll 5
+        for (uint32_t c = lane * 4; c < width; c += 128) {
+            const float4 v = *reinterpret_cast<const float4*>(q + c);
+            const float x0 = v.x * f, x1 = v.y * f, x2 = v.z * f, x3 = v.w * f;
+            const uint2 hw = make_uint2(pack_bf16(x0, x1), pack_bf16(x2, x3));
+            const float2 h01 = bf2(hw.x), h23 = bf2(hw.y);
+            *reinterpret_cast<uint2*>(qh + r * ld + c) = hw;
+            *reinterpret_cast<uint2*>(ql + r * ld + c) = make_uint2(pack_bf16(x0 - h01.x, x1 - h01.y), pack_bf16(x2 - h23.x, x3 - h23.y));
+        }
     }
     if (tid < LD_HEADS) { mrow[tid] = -INFINITY; lrow[tid] = 0.0f; }
     float o[NT][4];
@@ -56,48 +65,47 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const __grid_cons
     for (int i = 0; i < NT; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
     const uint32_t c0 = warp * NT * 8;                    // this warp's latent columns
 
-    for (uint32_t k0 = lo, b = 0; k0 < hi; k0 += LD_KEYS, b ^= 1) {
-        if (k0 + LD_KEYS < hi) {
-            fetch(k0 + LD_KEYS, b ^ 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
+    for (uint32_t k0 = lo, b = 0; k0 < hi; k0 += LD_KEYS, b = (b + 1) % LD_STAGES) {
+        fetch(k0 + (LD_STAGES - 1) * LD_KEYS, (b + LD_STAGES - 1) % LD_STAGES);   // into the tile that was read last
+        asm volatile("cp.async.wait_group %0;" ::"n"(LD_STAGES - 1) : "memory");
         __syncthreads();
         const uint32_t kb = kt_s + b * tile_bytes;
-        {   // scores of the warp's eight keys; two k-steps of the key operand per load
-            float d0[4] = {}, d1[4] = {};
-            const uint32_t qa = ((lane % 16) * ld + lane / 16 * 8) * 2, ka = kb + ((warp * 8 + lane % 8) * ld + lane / 8 * 8) * 2;
-            uint32_t kk = 0;
-            for (; kk + 32 <= width; kk += 32) {
+        {   // scores: four warps of eight keys over the first half of the columns, four over the second
+            float d[4][4] = {};
+            const uint32_t nt = warp & 3, mid = width / 64 * 32, stop = warp < 4 ? mid : width;
+            const uint32_t qa = ((lane % 16) * ld + lane / 16 * 8) * 2, ka = kb + ((nt * 8 + lane % 8) * ld + lane / 8 * 8) * 2;
+            uint32_t kk = warp < 4 ? 0 : mid;
+#pragma unroll 3
+            for (; kk + 32 <= stop; kk += 32) {   // two k-steps of the key operand per load
                 uint32_t k4[4], q4[4];
                 ldsm4(k4, ka + kk * 2);
-                ldsm4(q4, qh_s + qa + kk * 2); mma16816(d0, q4, k4[0], k4[1]);
-                ldsm4(q4, ql_s + qa + kk * 2); mma16816(d1, q4, k4[0], k4[1]);
-                ldsm4(q4, qh_s + qa + kk * 2 + 32); mma16816(d0, q4, k4[2], k4[3]);
-                ldsm4(q4, ql_s + qa + kk * 2 + 32); mma16816(d1, q4, k4[2], k4[3]);
+                ldsm4(q4, qh_s + qa + kk * 2); mma16816(d[0], q4, k4[0], k4[1]);
+                ldsm4(q4, ql_s + qa + kk * 2); mma16816(d[1], q4, k4[0], k4[1]);
+                ldsm4(q4, qh_s + qa + kk * 2 + 32); mma16816(d[2], q4, k4[2], k4[3]);
+                ldsm4(q4, ql_s + qa + kk * 2 + 32); mma16816(d[3], q4, k4[2], k4[3]);
             }
-            if (kk < width) {   // an odd k-step: its second half would lie past the row
+            if (kk < stop) {   // an odd k-step: its second half would lie past the row
                 uint32_t k2[2], q4[4];
-                ldsm2(k2, kb + ((warp * 8 + lane % 8) * ld + (lane / 8 & 1) * 8) * 2 + kk * 2);
-                ldsm4(q4, qh_s + qa + kk * 2); mma16816(d0, q4, k2[0], k2[1]);
-                ldsm4(q4, ql_s + qa + kk * 2); mma16816(d1, q4, k2[0], k2[1]);
+                ldsm2(k2, kb + ((nt * 8 + lane % 8) * ld + (lane / 8 & 1) * 8) * 2 + kk * 2);
+                ldsm4(q4, qh_s + qa + kk * 2); mma16816(d[0], q4, k2[0], k2[1]);
+                ldsm4(q4, ql_s + qa + kk * 2); mma16816(d[1], q4, k2[0], k2[1]);
             }
-            const uint32_t r = lane / 4, c = warp * 8 + (lane & 3) * 2;
-            sc[r][c] = d0[0] + d1[0]; sc[r][c + 1] = d0[1] + d1[1];
-            sc[r + 8][c] = d0[2] + d1[2]; sc[r + 8][c + 1] = d0[3] + d1[3];
+            const uint32_t r = lane / 4, c = nt * 8 + (lane & 3) * 2;
+            float (&out_sc)[LD_HEADS][LD_KEYS + 4] = sc[warp >> 2];
+            out_sc[r][c] = (d[0][0] + d[2][0]) + (d[1][0] + d[3][0]); out_sc[r][c + 1] = (d[0][1] + d[2][1]) + (d[1][1] + d[3][1]);
+            out_sc[r + 8][c] = (d[0][2] + d[2][2]) + (d[1][2] + d[3][2]); out_sc[r + 8][c + 1] = (d[0][3] + d[2][3]) + (d[1][3] + d[3][3]);
         }
         __syncthreads();
 #pragma unroll
-        for (int i = 0; i < 2; i++) {   // softmax of two heads per warp
+        for (int i = 0; i < 2; i++) {   // softmax of two heads per warp, a key per lane
             const uint32_t r = warp * 2 + i;
-            float x = k0 + lane < hi ? sc[r][lane] : -INFINITY, y = k0 + 32 + lane < hi ? sc[r][lane + 32] : -INFINITY;
-            const float m0 = mrow[r], top = fmaxf(m0, warp_max(fmaxf(x, y))), f = expf(m0 - top);
-            x = expf(x - top); y = expf(y - top);
-            const float sum = warp_sum(x + y);
-            const bf16 xb = __float2bfloat16_rn(x), yb = __float2bfloat16_rn(y);
-            ph[r][lane] = xb; pl[r][lane] = __float2bfloat16_rn(x - __bfloat162float(xb));
-            ph[r][lane + 32] = yb; pl[r][lane + 32] = __float2bfloat16_rn(y - __bfloat162float(yb));
+            float x = k0 + lane < hi ? sc[0][r][lane] + sc[1][r][lane] : -INFINITY;
+            const float m0 = mrow[r], top = fmaxf(m0, warp_max(x)), f = expf(m0 - top);
+            x = expf(x - top);
+            const float sum = warp_sum(x);
+            const bf16 xb = __float2bfloat16_rn(x);
+            ph[r][lane] = xb;
+            pl[r][lane] = __float2bfloat16_rn(x - __bfloat162float(xb));
             __syncwarp();
             if (lane == 0) { mrow[r] = top; lrow[r] = fmaf(lrow[r], f, sum); frow[r] = f; }
         }
@@ -137,7 +145,7 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const __grid_cons
     if (tid < LD_HEADS && h0 + tid < s.heads) { out[(size_t)(h0 + tid) * (s.cp + 2) + s.cp] = mrow[tid]; out[(size_t)(h0 + tid) * (s.cp + 2) + s.cp + 1] = lrow[tid]; }
 }
 
-size_t decode_smem(const LatentShape& s) { return (size_t)(2 * LD_HEADS + 2 * LD_KEYS) * (s.cp + s.rp + 8) * 2; }
+size_t decode_smem(const LatentShape& s) { return (size_t)(2 * LD_HEADS + LD_STAGES * LD_KEYS) * (s.cp + s.rp + 8) * 2; }
 
 template <int NT>
 cudaError_t decode_inst(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {

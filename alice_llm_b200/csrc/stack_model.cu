@@ -15,7 +15,7 @@ using namespace alice;
 namespace {
 
 constexpr uint32_t CHUNK_SMALL = 256, CHUNK = 2048, TRACE_TOKENS = 256;
-constexpr uint32_t DECODE_SPLITS = 64;   // shares of the context one decoded token's attention is cut into
+constexpr uint32_t DECODE_SPLITS = 128;  // most shares of the context one decoded token's attention is cut into
 constexpr uint32_t FEW_TOKENS = 4;       // up to here attention runs in the latent space also where the tiled form exists
 
 struct StackModel;
@@ -124,7 +124,8 @@ struct LatentMixer final : Mixer {
         a.s = sh; a.y = s.y; a.ldy = s.ldy; a.q_norm = q_norm; a.kv_norm = kv_norm; a.sink = sink; a.freq = freq; a.eps = m->cfg.eps;
         a.uk = uk.w; a.uv = uv.w; a.pos = m->d_pos; a.cache = cache[pass]; a.cache_bf16 = !m->exact();
         a.cqn = s.cqn; a.act_bf16 = m->tiled_bf16(n); a.q = s.q; a.ql = s.ql; a.part = s.part; a.mix = s.mix; a.out = s.a; a.ldo = o.k;
-        a.splits = n <= FEW_TOKENS ? DECODE_SPLITS / n : 1;
+        // one CTA per SM: shares of the context times groups of 16 heads times tokens
+        a.splits = n <= FEW_TOKENS ? std::max<uint32_t>(1, std::min(DECODE_SPLITS, (uint32_t)m->e->num_sms / ((sh.heads + 15) / 16)) / n) : 1;
         if (n == 1) {
             RowsIn in;
             in.x = s.y + sh.off_q; in.n_x = sh.q_rank; in.norm = NORM_RMS; in.norm_w = q_norm; in.eps = m->cfg.eps; in.w0 = uq; in.y0 = s.q;
