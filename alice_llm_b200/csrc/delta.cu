@@ -213,7 +213,13 @@ __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
           "l"(*reinterpret_cast<const unsigned long long*>(&c)));
     return d;
 }
-__device__ __forceinline__ float2 mul2(float2 a, float2 b) { return make_float2(a.x * b.x, a.y * b.y); }
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+    float2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;"
+        : "=l"(*reinterpret_cast<unsigned long long*>(&d))
+        : "l"(*reinterpret_cast<const unsigned long long*>(&a)), "l"(*reinterpret_cast<const unsigned long long*>(&b)));
+    return d;
+}
 
 // Sums 64 values over each half-warp; lane l of it is left with those of index 4 l .. 4 l + 3.
 __device__ __forceinline__ float4 reduce64(float (&v)[64], uint32_t lane) {
@@ -316,7 +322,7 @@ __global__ void __launch_bounds__(NW * 32) delta_scan_kernel(const __grid_consta
             }
         }
         __syncthreads();
-#pragma unroll
+#pragma unroll 1
         for (int pass = 0; pass < 2; pass++) {   // S^T (G k), then S^T (G q)
             float v[64];
 #pragma unroll
@@ -379,7 +385,7 @@ __global__ void __launch_bounds__(NW * 32) delta_scan_kernel(const __grid_consta
         for (int c = 0; c < 4; c++)
 #pragma unroll
             for (int i = 0; i < NP; i++) S[c][i] = mul2(e[i], S[c][i]);
-#pragma unroll
+#pragma unroll 4
         for (int t = 0; t < W; t++) {
             float2 x[NP];
             rows(st.g[t] + dg * 4, x);
