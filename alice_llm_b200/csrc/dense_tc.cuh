@@ -110,13 +110,16 @@ __device__ __forceinline__ void epi_32(const GemmOp& op, uint32_t t, uint32_t n,
     } else {
         if (whole) {
             float4* p = reinterpret_cast<float4*>(static_cast<float*>(op.out) + o);
+            const uint32_t head = EPI == EPI_DECAY ? n / op.dim : 0;
+            const bool one = EPI == EPI_DECAY && (n + 31) / op.dim == head;   // one head in these columns: one rate
+            const float rate = one ? expf(__ldg(op.a_log + head)) : 0.0f;
 #pragma unroll
             for (int i = 0; i < 8; i++) {
                 float r[4];
 #pragma unroll
                 for (int j = 0; j < 4; j++) {
                     const uint32_t c = n + 4 * i + j;
-                    if constexpr (EPI == EPI_DECAY) r[j] = expf(-expf(__ldg(op.a_log + c / op.dim)) * softplus_f(v[4 * i + j] + __ldg(op.bias + c)));
+                    if constexpr (EPI == EPI_DECAY) r[j] = expf(-(one ? rate : expf(__ldg(op.a_log + c / op.dim))) * softplus_f(v[4 * i + j] + __ldg(op.bias + c)));
                     else r[j] = sigmoid_f(v[4 * i + j]);
                 }
                 p[i] = make_float4(r[0], r[1], r[2], r[3]);
