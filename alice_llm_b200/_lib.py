@@ -106,16 +106,18 @@ class LayerWeights(C.Structure):
 class StackLayer(C.Structure):
     """alice_stack_layer"""
     _fields_ = [(n, C.c_uint32) for n in ("mixer", "heads", "kv_heads", "dim", "vdim", "q_rank", "kv_rank", "rot_dim", "rot_dims", "conv_taps",
-                                          "decay_rank", "gate_rank", "ff")] + \
-               [("scale", C.c_float), ("rot_base", C.c_double)] + \
-               [(n, C.c_void_p) for n in ("in_", "uq", "uk", "uv", "a2", "g2", "o", "gu", "down", "norm", "ls1", "ls2", "gate_bias", "up_bias",
+                                          "decay_rank", "gate_rank", "ff", "unit_qk")] + \
+               [("scale", C.c_float), ("softcap", C.c_float)] + \
+               [(n, C.c_double) for n in ("rot_base", "rot_factor", "rot_low", "rot_high", "rot_original")] + \
+               [(n, C.c_void_p) for n in ("in_", "uq", "uk", "uv", "a2", "g2", "o", "gu", "down", "norm", "norm2", "ls1", "ls2", "gate_bias", "up_bias",
                                           "down_bias", "q_norm", "kv_norm", "sink", "conv", "a_log", "dt_bias", "head_norm")]
 
 
 class StackConfig(C.Structure):
     """alice_stack_config"""
-    _fields_ = [(n, C.c_uint32) for n in ("num_layers", "width", "vocab_size", "max_seq_len", "loop_start", "loop_stop", "loop_times", "exact")] + \
-               [("eps", C.c_float), ("embed_scale", C.c_float), ("loop_step", C.c_void_p)]
+    _fields_ = [(n, C.c_uint32) for n in ("num_layers", "width", "vocab_size", "max_seq_len", "loop_start", "loop_stop", "loop_times", "exact", "block",
+                                          "norm")] + \
+               [("eps", C.c_float), ("embed_scale", C.c_float), ("alpha", C.c_float), ("loop_step", C.c_void_p), ("head", C.c_void_p)]
 
 
 class AliceError(RuntimeError):

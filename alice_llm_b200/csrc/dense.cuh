@@ -20,7 +20,8 @@ struct DenseMat {
 
 enum InputNorm : int { NORM_NONE = 0, NORM_LAYER = 1, NORM_RMS = 2 };
 
-// One token: y0 = W0 h and y1 = act(gate h) * (up h), both of the same h, which every CTA derives from x itself.
+// One token: y0 = W0 h and y1 = act(gate h) * (up h), both of the same h, which every CTA derives from x itself. Either product
+// may be absent.
 struct RowsIn {
     const float* x = nullptr;
     uint32_t n_x = 0;             // true length; elements [n_x, k) of h are zero
@@ -30,24 +31,27 @@ struct RowsIn {
     DenseMat w0;
     float* y0 = nullptr;
     DenseMat gu;                  // 64 gate rows, 64 up rows, 64 gate rows, ... (gu.n = 2 * ff padded), or empty
-    const float *gate_b = nullptr, *up_b = nullptr;
+    const float *gate_b = nullptr, *up_b = nullptr;   // null: no biases
     float* y1 = nullptr;
+    float* h_out = nullptr;       // not x: h itself is left here too, n_x elements
     unsigned long long* argmax_key = nullptr;   // of y0's rows: atomicMax of (order-preserving value, ~row)
 };
-// One token: x += s1 * (W1 a) + s2 * (W2 f + b2).
+// One token: out = alpha * x + s1 * (W1 a) + s2 * (W2 f + b2); out and x may be the same vector.
 struct RowsOut {
     DenseMat w1, w2;              // w2 may be empty
+    float alpha = 1.f;
     const float *a = nullptr, *f = nullptr;
-    const float *s1 = nullptr, *s2 = nullptr, *b2 = nullptr;
-    float* x = nullptr;
+    const float *s1 = nullptr, *s2 = nullptr, *b2 = nullptr;   // s1 null: all ones
+    const float* x = nullptr;
+    float* out = nullptr;
 };
 cudaError_t launch_rows_in(const RowsIn& op, int num_sms, cudaStream_t st, bool pdl);
 cudaError_t launch_rows_out(const RowsOut& op, int num_sms, cudaStream_t st, bool pdl);
 
 enum DenseEpilogue : int {
     EPI_STORE = 0,     // out[t][n] = acc (and, for n >= col2, a bf16 copy in out2)
-    EPI_SWIGLU = 1,    // w holds interleaved gate / up rows; out[t][c] = silu(gate + gate_b) * (up + up_b)
-    EPI_RESID = 2,     // out[t][n] += scale[n] * (acc + bias[n])
+    EPI_SWIGLU = 1,    // w holds interleaved gate / up rows; out[t][c] = silu(gate + gate_b) * (up + up_b), biases may be null
+    EPI_RESID = 2,     // out[t][n] = alpha * out[t][n] + scale[n] * (acc + bias[n]); scale and bias may be null
     EPI_DECAY = 3,     // out[t][n] = exp(-exp(a_log[n / dim]) * softplus(acc + bias[n]))
     EPI_SIGMOID = 4,   // out[t][n] = sigmoid(acc)
 };
@@ -66,6 +70,7 @@ struct GemmOp {
     bf16* out2 = nullptr;
     uint32_t col2 = 0, ld2 = 0;
     const float *bias = nullptr, *bias2 = nullptr, *scale = nullptr, *a_log = nullptr;
+    float alpha = 1.f;
     uint32_t dim = 1;
 };
 // bf16 inputs run on the tensor cores, f32 inputs in f32 arithmetic throughout.

@@ -12,7 +12,9 @@ __device__ __forceinline__ void epi_one(const GemmOp& op, uint32_t t, uint32_t n
         else static_cast<float*>(op.out)[o] = v;
         if (op.out2 && n >= op.col2) put(op.out2 + (size_t)t * op.ld2 + (n - op.col2), v);
     } else if constexpr (EPI == EPI_RESID) {
-        static_cast<float*>(op.out)[o] += op.scale[n] * (op.bias ? v + op.bias[n] : v);
+        float* x = static_cast<float*>(op.out) + o;
+        const float r = op.bias ? v + op.bias[n] : v;
+        *x = op.alpha * *x + (op.scale ? op.scale[n] * r : r);
     } else if constexpr (EPI == EPI_DECAY) {
         static_cast<float*>(op.out)[o] = expf(-expf(op.a_log[n / op.dim]) * softplus_f(v + op.bias[n]));
     } else if constexpr (EPI == EPI_SIGMOID) {
@@ -21,7 +23,7 @@ __device__ __forceinline__ void epi_one(const GemmOp& op, uint32_t t, uint32_t n
 }
 
 __device__ __forceinline__ void epi_swiglu(const GemmOp& op, uint32_t t, uint32_t c, float gate, float up) {
-    const float v = silu_ref(gate + op.bias[c]) * (up + op.bias2[c]);
+    const float v = op.bias ? silu_ref(gate + op.bias[c]) * (up + op.bias2[c]) : silu_ref(gate) * up;
     const size_t o = (size_t)t * op.ldo + c;
     if (op.out_bf16) put(static_cast<bf16*>(op.out) + o, v);
     else static_cast<float*>(op.out)[o] = v;

@@ -76,7 +76,7 @@ __global__ void __launch_bounds__(RT, 2) rows_in_kernel(const __grid_constant__ 
     const uint32_t lane = threadIdx.x & 31, warps = gridDim.x * RW;
     const uint32_t items0 = (op.w0.n + R - 1) / R, items = items0 + op.gu.n / R;
     const uint32_t w_id = blockIdx.x + (threadIdx.x >> 5) * gridDim.x;
-    const uint32_t k = op.w0.k;
+    const uint32_t k = op.w0.n ? op.w0.k : op.gu.k;
     const bf16* w[R];
     uint32_t first;
     bool pair;
@@ -88,6 +88,8 @@ __global__ void __launch_bounds__(RT, 2) rows_in_kernel(const __grid_constant__ 
     }
     pdl_wait();
     load_normed<RW>(xs, op.x, op.n_x, k, op.norm, op.norm_w, op.eps, red);
+    if (op.h_out && blockIdx.x == 0)
+        for (uint32_t i = threadIdx.x; i < op.n_x; i += RT) op.h_out[i] = xs[i];
     unsigned long long best = 0ull;
     for (uint32_t item = w_id; item < items; item += warps) {
         item_rows<R>(op, item, items0, w, first, pair);
@@ -103,7 +105,10 @@ __global__ void __launch_bounds__(RT, 2) rows_in_kernel(const __grid_constant__ 
         } else {
 #pragma unroll
             for (int r = 0; r < R / 2; r++)
-                if (lane == (uint32_t)r) op.y1[first + r] = silu_ref(acc[r] + op.gate_b[first + r]) * (acc[R / 2 + r] + op.up_b[first + r]);
+                if (lane == (uint32_t)r) {
+                    const float g = op.gate_b ? acc[r] + op.gate_b[first + r] : acc[r], u = op.up_b ? acc[R / 2 + r] + op.up_b[first + r] : acc[R / 2 + r];
+                    op.y1[first + r] = silu_ref(g) * u;
+                }
         }
     }
     if (op.argmax_key && lane == 0 && best) atomicMax(op.argmax_key, best);
@@ -143,9 +148,9 @@ __global__ void __launch_bounds__(RT, 2) rows_out_kernel(const __grid_constant__
         for (int r = 0; r < R; r++) {
             const uint32_t row = item * R + r;
             if (lane == (uint32_t)r && row < n) {
-                float v = op.s1[row] * acc1[r];
+                float v = op.s1 ? op.s1[row] * acc1[r] : acc1[r];
                 if (k2) v += op.s2[row] * (acc2[r] + op.b2[row]);
-                op.x[row] += v;
+                op.out[row] = op.alpha * op.x[row] + v;
             }
         }
     }
@@ -167,12 +172,14 @@ cudaError_t rows_in_r(const RowsIn& op, int num_sms, cudaStream_t st, bool pdl) 
     if (err != cudaSuccess) return err;
     const uint32_t items = (op.w0.n + R - 1) / R + op.gu.n / R;
     const uint32_t grid = std::min<uint32_t>((items + RW - 1) / RW, (uint32_t)num_sms * 2);
-    return launch_pdl(rows_in_kernel<R>, dim3(grid), dim3(RT), (size_t)op.w0.k * 4, st, pdl, op);
+    return launch_pdl(rows_in_kernel<R>, dim3(grid), dim3(RT), (size_t)(op.w0.n ? op.w0.k : op.gu.k) * 4, st, pdl, op);
 }
 }  // namespace
 
 cudaError_t launch_rows_in(const RowsIn& op, int num_sms, cudaStream_t st, bool pdl) {
-    if (!op.w0.n || op.w0.k % DENSE_PAD || (op.gu.n && (op.gu.k != op.w0.k || op.gu.n % 128)) || (size_t)op.w0.k * 4 > 220 * 1024) return cudaErrorInvalidValue;
+    const uint32_t k = op.w0.n ? op.w0.k : op.gu.k;
+    if ((!op.w0.n && !op.gu.n) || k % DENSE_PAD || (op.gu.n && (op.gu.k != k || op.gu.n % 128)) || (size_t)k * 4 > 220 * 1024) return cudaErrorInvalidValue;
+    if (op.h_out == op.x) return cudaErrorInvalidValue;   // other CTAs still read x
     return rows_in_r<2>(op, num_sms, st, pdl);
 }
 

@@ -100,9 +100,10 @@ __device__ __forceinline__ void epi_32(const GemmOp& op, uint32_t t, uint32_t n,
 #pragma unroll
             for (int i = 0; i < 8; i++) {
                 float4 x = p[i];
-                const float4 s = __ldg(reinterpret_cast<const float4*>(op.scale + n) + i);
+                const float4 s = op.scale ? __ldg(reinterpret_cast<const float4*>(op.scale + n) + i) : make_float4(1.f, 1.f, 1.f, 1.f);
                 const float4 b = op.bias ? __ldg(reinterpret_cast<const float4*>(op.bias + n) + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-                x.x += s.x * (v[4 * i] + b.x); x.y += s.y * (v[4 * i + 1] + b.y); x.z += s.z * (v[4 * i + 2] + b.z); x.w += s.w * (v[4 * i + 3] + b.w);
+                x.x = op.alpha * x.x + s.x * (v[4 * i] + b.x); x.y = op.alpha * x.y + s.y * (v[4 * i + 1] + b.y);
+                x.z = op.alpha * x.z + s.z * (v[4 * i + 2] + b.z); x.w = op.alpha * x.w + s.w * (v[4 * i + 3] + b.w);
                 p[i] = x;
             }
             return;
@@ -140,7 +141,7 @@ __device__ __forceinline__ void epi_swiglu_32(const GemmOp& op, uint32_t t, uint
 #pragma unroll
         for (int j = 0; j < 8; j++) {
             const int k = 8 * i + j;
-            r[j] = silu_ref(g[k] + __ldg(op.bias + c + k)) * (u[k] + __ldg(op.bias2 + c + k));
+            r[j] = op.bias ? silu_ref(g[k] + __ldg(op.bias + c + k)) * (u[k] + __ldg(op.bias2 + c + k)) : silu_ref(g[k]) * u[k];
         }
         uint32_t w[4];
 #pragma unroll

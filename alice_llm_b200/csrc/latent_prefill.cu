@@ -1,199 +1,9 @@
-// Causal attention of many tokens over keys and values made from the cached latent rows, on the tensor cores: bf16 queries,
-// keys and values, f32 scores, softmax and sums. The softmax weights enter the weighted sum as a bf16 pair (value and
-// remainder), so they are not cut to eight bits. The sink of a head is the state the online softmax starts from: a key that
-// scores `sink` and has no value.
-#include "dense_dev.cuh"
-#include "mixers.cuh"
-#include "mma_sync.cuh"
+// Attention of many tokens over a cached latent: keys and values of the whole context have been made from the latent rows,
+// the rotated key part is read from the cache itself.
+#include "attn_prefill.cuh"
 
 namespace alice {
 namespace {
-
-constexpr int PF_KEYS = 32, PF_ROWS = 128, PF_THREADS = 128;   // keys per tile; queries per CTA, 32 per warp: each key fragment serves two row tiles
-
-// DQ, DV: query / key and value dimensions the tiles have room for (multiples of 16, zero beyond the true sizes). Values wider
-// than DV are cut into slices (blockIdx.z), each with its own pass over the scores.
-template <int DQ, int DV>
-struct PfGeom {
-    static constexpr int LQ = DQ + 8, LV = DV + 8;   // row strides: eight rows land in different banks
-    static constexpr size_t Q = (size_t)PF_ROWS * LQ * 2, K = (size_t)PF_KEYS * LQ * 2, V = (size_t)PF_KEYS * LV * 2, SMEM = Q + 2 * (K + V);
-};
-
-template <int DQ, int DV>
-__global__ void __launch_bounds__(PF_THREADS, 2) latent_prefill_kernel(const __grid_constant__ LatentArgs a, uint32_t tokens) {
-    using G = PfGeom<DQ, DV>;
-    extern __shared__ __align__(128) uint8_t sm[];
-    const LatentShape& s = a.s;
-    const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x;
-    const uint32_t t0 = (gridDim.y - 1 - blockIdx.y) * PF_ROWS;   // the longest rows first
-    const uint32_t q_sm = smem_u32(sm), k_sm = q_sm + (uint32_t)G::Q, v_sm = k_sm + 2 * (uint32_t)G::K;
-    pdl_launch_dependents();
-    pdl_wait();
-    const uint32_t p0 = (uint32_t)*a.pos, qd = s.dim + s.rot;
-    const uint32_t rows = min((uint32_t)PF_ROWS, tokens - t0), keys = p0 + t0 + rows, ntiles = (keys + PF_KEYS - 1) / PF_KEYS;
-    const bf16* cache = static_cast<const bf16*>(a.cache);
-    const uint32_t cw = s.cp + s.rp, kw = s.heads * s.dim, vw = s.heads * s.vdim;
-    const uint32_t v0 = blockIdx.z * DV, vn = min(s.vdim - v0, (uint32_t)DV);   // this slice of the values
-
-    // zero what lies beyond the true sizes once (the copies below never touch it)
-    for (uint32_t i = tid; i < 2 * PF_KEYS * (DQ - qd); i += PF_THREADS) {
-        const uint32_t r = i / (DQ - qd), c = qd + i % (DQ - qd);
-        reinterpret_cast<bf16*>(sm + G::Q + (r / PF_KEYS) * G::K)[(r % PF_KEYS) * G::LQ + c] = __float2bfloat16_rn(0.0f);
-    }
-    for (uint32_t i = tid; i < 2 * PF_KEYS * (DV - vn); i += PF_THREADS) {
-        const uint32_t r = i / (DV - vn), c = vn + i % (DV - vn);
-        reinterpret_cast<bf16*>(sm + G::Q + 2 * G::K + (r / PF_KEYS) * G::V)[(r % PF_KEYS) * G::LV + c] = __float2bfloat16_rn(0.0f);
-    }
-    // rows of 16-byte pieces, a few threads a row
-    constexpr uint32_t TPR = PF_THREADS / PF_KEYS;
-    const uint32_t fr = tid / TPR, fc = tid % TPR, nd = s.dim / 8, nr = s.rot / 8, nv = vn / 8;
-    auto fetch = [&](uint32_t tile, uint32_t b) {
-        const uint32_t j = min(tile * PF_KEYS + fr, keys - 1);
-        const bool ok = tile * PF_KEYS + fr < keys;
-        const uint32_t kd = k_sm + b * (uint32_t)G::K + fr * G::LQ * 2, vd = v_sm + b * (uint32_t)G::V + fr * G::LV * 2;
-        const bf16 *kp = a.k_all + (size_t)j * kw + (size_t)h * s.dim, *rp = cache + (size_t)j * cw + s.cp, *vp = a.v_all + (size_t)j * vw + (size_t)h * s.vdim + v0;
-        for (uint32_t c = fc; c < nd; c += TPR) cp16(kd + c * 16, kp + c * 8, ok);
-        for (uint32_t c = fc; c < nr; c += TPR) cp16(kd + (nd + c) * 16, rp + c * 8, ok);
-        for (uint32_t c = fc; c < nv; c += TPR) cp16(vd + c * 16, vp + c * 8, ok);
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    };
-    for (uint32_t r = fr; r < PF_ROWS; r += PF_KEYS) {   // queries, part of the first copy group
-        const bf16* q = a.q_rot + ((size_t)(t0 + min(r, rows - 1)) * s.heads + h) * qd;
-        for (uint32_t c = fc; c < DQ / 8; c += TPR) cp16(q_sm + r * G::LQ * 2 + c * 16, q + min(c * 8, qd - 8), r < rows && c * 8 < qd);
-    }
-    fetch(0, 0);
-
-    // a thread's rows are lane / 4 and lane / 4 + 8 of each of its warp's two 16-row tiles
-    constexpr float LOG2E = 1.4426950408889634f;
-    const float scale = s.scale * LOG2E;
-    float m[2][2], l[2][2], o[2][DV / 8][4];
-#pragma unroll
-    for (int g = 0; g < 2; g++) {
-        m[g][0] = m[g][1] = a.sink[h] * LOG2E;
-        l[g][0] = l[g][1] = (lane & 3) == 0 ? 1.0f : 0.0f;
-#pragma unroll
-        for (int i = 0; i < DV / 8; i++) o[g][i][0] = o[g][i][1] = o[g][i][2] = o[g][i][3] = 0.0f;
-    }
-    const uint32_t row0 = warp * 32 + lane / 4, see = p0 + t0 + row0;   // last key the first of them sees
-    const uint32_t q_addr = q_sm + ((warp * 32 + lane % 16) * G::LQ + lane / 16 * 8) * 2;
-
-    for (uint32_t tile = 0; tile < ntiles; tile++) {
-        const uint32_t b = tile & 1;
-        if (tile + 1 < ntiles) {
-            fetch(tile + 1, b ^ 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();
-        const uint32_t kt = k_sm + b * (uint32_t)G::K, vt = v_sm + b * (uint32_t)G::V;
-        float sc[2][PF_KEYS / 8][4];
-#pragma unroll
-        for (int g = 0; g < 2; g++)
-#pragma unroll
-            for (int i = 0; i < PF_KEYS / 8; i++) sc[g][i][0] = sc[g][i][1] = sc[g][i][2] = sc[g][i][3] = 0.0f;
-        const uint32_t k_addr = kt + ((lane % 8 + lane / 16 * 8) * G::LQ + (lane / 8 % 2) * 8) * 2;
-#pragma unroll
-        for (int kk = 0; kk < DQ / 16; kk++) {
-            uint32_t q0[4], q1[4];
-            ldsm4(q0, q_addr + kk * 32);
-            ldsm4(q1, q_addr + 16 * G::LQ * 2 + kk * 32);
-#pragma unroll
-            for (int n = 0; n < PF_KEYS / 16; n++) {
-                uint32_t kb[4];
-                ldsm4(kb, k_addr + (n * 16 * G::LQ + kk * 16) * 2);
-                mma16816(sc[0][2 * n], q0, kb[0], kb[1]);
-                mma16816(sc[0][2 * n + 1], q0, kb[2], kb[3]);
-                mma16816(sc[1][2 * n], q1, kb[0], kb[1]);
-                mma16816(sc[1][2 * n + 1], q1, kb[2], kb[3]);
-            }
-        }
-        const uint32_t j0 = tile * PF_KEYS + (lane & 3) * 2;
-        const bool edge = tile * PF_KEYS + PF_KEYS > p0 + t0 + warp * 32;   // some key of the tile is hidden from some row of the warp
-#pragma unroll
-        for (int g = 0; g < 2; g++) {
-            float top0 = m[g][0], top1 = m[g][1];
-#pragma unroll
-            for (int i = 0; i < PF_KEYS / 8; i++) {
-#pragma unroll
-                for (int e = 0; e < 4; e++) {
-                    float v = sc[g][i][e] * scale;
-                    if (edge && j0 + i * 8 + (e & 1) > see + g * 16 + (e < 2 ? 0 : 8)) v = -INFINITY;
-                    sc[g][i][e] = v;
-                }
-                top0 = fmaxf(top0, fmaxf(sc[g][i][0], sc[g][i][1]));
-                top1 = fmaxf(top1, fmaxf(sc[g][i][2], sc[g][i][3]));
-            }
-#pragma unroll
-            for (int x = 1; x <= 2; x *= 2) {
-                top0 = fmaxf(top0, __shfl_xor_sync(0xffffffffu, top0, x));
-                top1 = fmaxf(top1, __shfl_xor_sync(0xffffffffu, top1, x));
-            }
-            const float f0 = exp2f(m[g][0] - top0), f1 = exp2f(m[g][1] - top1);
-            if (__any_sync(0xffffffffu, f0 != 1.0f || f1 != 1.0f)) {
-#pragma unroll
-                for (int i = 0; i < DV / 8; i++) { o[g][i][0] *= f0; o[g][i][1] *= f0; o[g][i][2] *= f1; o[g][i][3] *= f1; }
-            }
-            m[g][0] = top0; m[g][1] = top1;
-            l[g][0] *= f0; l[g][1] *= f1;
-#pragma unroll
-            for (int i = 0; i < PF_KEYS / 8; i++) {
-                sc[g][i][0] = exp2f(sc[g][i][0] - top0); sc[g][i][1] = exp2f(sc[g][i][1] - top0);
-                sc[g][i][2] = exp2f(sc[g][i][2] - top1); sc[g][i][3] = exp2f(sc[g][i][3] - top1);
-                l[g][0] += sc[g][i][0] + sc[g][i][1]; l[g][1] += sc[g][i][2] + sc[g][i][3];
-            }
-        }
-        const uint32_t v_addr = vt + ((lane % 16) * G::LV + lane / 16 * 8) * 2;
-#pragma unroll
-        for (int kk = 0; kk < PF_KEYS / 16; kk++) {
-            uint32_t hi[2][4], lo[2][4];
-#pragma unroll
-            for (int g = 0; g < 2; g++)
-#pragma unroll
-                for (int e = 0; e < 4; e++) {
-                    const float x = sc[g][2 * kk + e / 2][(e & 1) * 2], y = sc[g][2 * kk + e / 2][(e & 1) * 2 + 1];
-                    hi[g][e] = pack_bf16(x, y);
-                    const float2 r = bf2(hi[g][e]);
-                    lo[g][e] = pack_bf16(x - r.x, y - r.y);
-                }
-#pragma unroll
-            for (int n = 0; n < DV / 16; n++) {
-                uint32_t vb[4];
-                ldsm4t(vb, v_addr + (kk * 16 * G::LV + n * 16) * 2);
-#pragma unroll
-                for (int g = 0; g < 2; g++) {
-                    mma16816(o[g][2 * n], hi[g], vb[0], vb[1]);
-                    mma16816(o[g][2 * n + 1], hi[g], vb[2], vb[3]);
-                    mma16816(o[g][2 * n], lo[g], vb[0], vb[1]);
-                    mma16816(o[g][2 * n + 1], lo[g], vb[2], vb[3]);
-                }
-            }
-        }
-        __syncthreads();
-    }
-#pragma unroll
-    for (int g = 0; g < 2; g++)
-#pragma unroll
-        for (int r = 0; r < 2; r++) {
-            float den = l[g][r];
-            den += __shfl_xor_sync(0xffffffffu, den, 1);
-            den += __shfl_xor_sync(0xffffffffu, den, 2);
-            const float inv = __frcp_rn(den);
-            const uint32_t row = row0 + 16 * g + 8 * r;
-            if (row >= rows) continue;
-            const float* gate = a.y + (size_t)(t0 + row) * a.ldy + s.off_g + (size_t)h * s.vdim + v0;
-            bf16* out = static_cast<bf16*>(a.out) + (size_t)(t0 + row) * a.ldo;
-#pragma unroll
-            for (int i = 0; i < DV / 8; i++) {
-                const uint32_t c = i * 8 + (lane & 3) * 2;
-                if (c < vn)
-                    *reinterpret_cast<uint32_t*>(out + (size_t)h * s.vdim + v0 + c) =
-                        pack_bf16(o[g][i][2 * r] * inv * sigmoid_f(gate[c]), o[g][i][2 * r + 1] * inv * sigmoid_f(gate[c + 1]));
-            }
-            if (h + 1 == s.heads)   // padding up to the stride
-                for (uint32_t c = s.heads * s.vdim + (lane & 3); c < a.ldo; c += 4) out[c] = __float2bfloat16_rn(0.0f);
-        }
-}
 
 // Queries in bf16 with the rotated part turned to its position. One CTA per token.
 __global__ void __launch_bounds__(256) latent_rotate_kernel(const __grid_constant__ LatentArgs a, bf16* out) {
@@ -227,25 +37,20 @@ __global__ void __launch_bounds__(256) latent_rotate_kernel(const __grid_constan
     }
 }
 
-template <int DQ, int DV>
-cudaError_t prefill_inst(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
-    static bool done[64] = {};
-    const cudaError_t err = allow_smem(latent_prefill_kernel<DQ, DV>, PfGeom<DQ, DV>::SMEM, done);
-    if (err != cudaSuccess) return err;
-    return launch_pdl(latent_prefill_kernel<DQ, DV>, dim3(a.s.heads, (tokens + PF_ROWS - 1) / PF_ROWS, (a.s.vdim + DV - 1) / DV), dim3(PF_THREADS), PfGeom<DQ, DV>::SMEM, st, pdl, a, tokens);
-}
-
 }  // namespace
 
 cudaError_t launch_latent_prefill(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
     if (!latent_prefill_fits(a.s) || !a.cache_bf16 || !a.act_bf16) return cudaErrorInvalidValue;
-    const uint32_t q = a.s.dim + a.s.rot, v = a.s.vdim;
     const cudaError_t err = launch_pdl(latent_rotate_kernel, dim3(tokens), dim3(256), (size_t)(a.s.rot_dims / 2) * sizeof(float2), st, pdl, a, a.q_rot);
     if (err != cudaSuccess) return err;
-    if (q <= 64 && v <= 64) return prefill_inst<64, 64>(a, tokens, st, pdl);
-    if (q <= 128 && v <= 128) return prefill_inst<128, 128>(a, tokens, st, pdl);
-    if (q <= 192) return prefill_inst<192, 128>(a, tokens, st, pdl);
-    return prefill_inst<256, 128>(a, tokens, st, pdl);
+    const LatentShape& z = a.s;
+    PrefillArgs p;
+    p.heads = z.heads; p.vdim = p.v_cols = z.vdim; p.q = a.q_rot; p.pos = a.pos; p.sink = a.sink; p.scale = z.scale;
+    p.k1 = a.k_all; p.k1_cols = z.dim; p.k1_row = (size_t)z.heads * z.dim; p.k1_head = z.dim;
+    p.k2 = static_cast<const bf16*>(a.cache) + z.cp; p.k2_cols = z.rot; p.k2_row = z.cp + z.rp;
+    p.v = a.v_all; p.v_row = (size_t)z.heads * z.vdim; p.v_head = z.vdim;
+    p.gate = a.y + z.off_g; p.ld_gate = a.ldy; p.out = static_cast<bf16*>(a.out); p.ldo = a.ldo;
+    return launch_attn_prefill<false>(p, tokens, st, pdl);
 }
 
 }  // namespace alice

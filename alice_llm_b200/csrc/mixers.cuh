@@ -1,4 +1,4 @@
-// Token mixers of layer-stack models (csrc/delta.cu, csrc/latent.cu) and the small per-token kernels around them
+// Token mixers of layer-stack models (csrc/delta.cu, csrc/latent.cu, csrc/grouped.cu) and the small per-token kernels around them
 // (csrc/stack_ops.cu). Sizes are run-time values; positions come from device memory so that a captured step can be replayed.
 #pragma once
 #include "dense.cuh"
@@ -21,15 +21,17 @@ cudaError_t launch_enter(const EnterArgs& a, uint32_t tokens, cudaStream_t st, b
 constexpr uint32_t MAX_NORM_ROWS = 64;
 struct NormArgs {
     const float* x = nullptr;
-    uint32_t ldx = 0, n = 0, k = 0;   // true and padded length; out rows are k apart, zero beyond n
+    uint32_t ldx = 0, n = 0, k = 0;   // true and padded length (a row holds k floats); out rows are k apart, zero beyond n
+    int norm = NORM_LAYER;            // NORM_NONE: a plain copy
     const float* w = nullptr;
     float eps = 0.f;
-    void* out = nullptr;
+    void* out = nullptr;              // may be null
     bool out_bf16 = false;
+    float* x_out = nullptr;           // f32 result, rows ldx apart; may be x
     bool gather = false;              // read rows idx[i] instead of i (at most MAX_NORM_ROWS)
     uint32_t idx[MAX_NORM_ROWS] = {};
 };
-cudaError_t launch_layer_norm(const NormArgs& a, uint32_t rows, cudaStream_t st, bool pdl);
+cudaError_t launch_norm(const NormArgs& a, uint32_t rows, cudaStream_t st, bool pdl);
 
 // ---- delta.cu: delta rule with one decay per key channel ----------------------------------------
 struct DeltaShape {
@@ -119,5 +121,48 @@ bool latent_decode_fits(const LatentShape& s);
 cudaError_t launch_latent_decode(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 cudaError_t launch_latent_attn(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 cudaError_t launch_latent_out(const LatentArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
+
+// ---- grouped.cu: attention whose key / value heads serve groups of query heads ---------------------
+struct GroupedShape {
+    uint32_t heads, kv_heads, dim, vdim, rot_dims;
+    uint32_t dp, vp;                  // dim and vdim padded to 16
+    uint32_t off_k, off_v;            // columns of the projection output (queries start at 0)
+    float scale, softcap;             // softcap 0: none
+    bool unit_qk;                     // rotated queries and keys over their root mean square
+    uint32_t group() const { return heads / kv_heads; }
+    // A cache row is [key dp | value vp | 8 unused]: eight rows start in different shared-memory banks as they lie.
+    __host__ __device__ uint32_t ld() const { return dp + vp + 8; }
+};
+constexpr uint32_t GROUPED_MAX_DIM = 512, GROUPED_TILE = 16;   // keys are read in whole tiles: planes of the cache hold multiples of it
+
+struct GroupedArgs {
+    GroupedShape s;
+    const float* y = nullptr;         // projections [t][ldy]: q | k | v
+    uint32_t ldy = 0;
+    const float *sink = nullptr, *freq = nullptr;   // sink [heads], -inf for none
+    float eps = 0.f;
+    const int* pos = nullptr;
+    void* cache = nullptr;            // [kv_heads][plane_rows][ld]
+    uint32_t plane_rows = 0;
+    bool cache_bf16 = false;
+    void* q = nullptr;                // prepared queries [t][heads][dp], of the cache's type
+    void* out = nullptr;              // [t][ldo]
+    uint32_t ldo = 0;
+    bool act_bf16 = false;            // type of out
+    // grouped_decode.cu
+    bool append = false;              // one token: its cache row is made here too
+    uint32_t splits = 1;
+    float* part = nullptr;            // [t][splits][heads][vp + 4]
+    unsigned int* tickets = nullptr;  // [t][kv_heads * groups of 16 heads], zero between launches
+    int* status = nullptr;
+};
+// Rotation and norm of queries and keys; queries to a.q, keys and values into the cache.
+cudaError_t launch_grouped_prepare(const GroupedArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
+// In f32 arithmetic throughout, prepared queries and cache of either type.
+cudaError_t launch_grouped_attn(const GroupedArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
+// On the tensor cores, bf16 cache: many tokens (prepared queries), few tokens (queries straight from the projections).
+inline bool grouped_tiled_fits(const GroupedShape& s) { return s.dp <= 256 && s.vp <= 256; }
+cudaError_t launch_grouped_prefill(const GroupedArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
+cudaError_t launch_grouped_decode(const GroupedArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 
 }  // namespace alice

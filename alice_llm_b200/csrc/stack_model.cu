@@ -16,7 +16,7 @@ namespace {
 
 constexpr uint32_t CHUNK_SMALL = 256, CHUNK = 2048, TRACE_TOKENS = 256;
 constexpr uint32_t DECODE_SPLITS = 128;  // most shares of the context one decoded token's attention is cut into
-constexpr uint32_t FEW_TOKENS = 4;       // up to here attention runs in the latent space also where the tiled form exists
+constexpr uint32_t FEW_TOKENS = 4;       // up to here attention runs in its form for single tokens also where the tiled form exists
 
 struct StackModel;
 
@@ -29,12 +29,13 @@ DenseMat mat_of(const alice_weights* w) {
 // Buffers of one forward call, shared by all layers.
 struct Scratch {
     uint32_t chunk = 0, wp = 0, ldy = 0, ldf = 0, lda = 0;
-    float *x = nullptr, *y = nullptr;
+    float *x = nullptr, *y = nullptr, *r = nullptr;  // stream, projections, a single token's sum ahead of its norm
     void *h = nullptr, *f = nullptr, *a = nullptr;   // activations: f32, or bf16 in tiled products
     // latent
     float *q = nullptr, *ql = nullptr, *part = nullptr, *mix = nullptr;
     void* cqn = nullptr;
     bf16 *k_all = nullptr, *v_all = nullptr, *q_rot = nullptr;   // keys and values of the whole context and rotated queries (tiled prefill)
+    unsigned int* tickets = nullptr;                 // grouped attention
     // delta
     float *qn = nullptr, *kn = nullptr, *pair_inv = nullptr, *pair_b = nullptr, *v = nullptr, *beta = nullptr, *g = nullptr, *gate = nullptr, *o = nullptr;
     bf16* low = nullptr;                             // bf16 copy of the low-rank columns
@@ -56,14 +57,15 @@ struct StackLayer {
     std::unique_ptr<Mixer> mixer;
     DenseMat gu, down;
     uint32_t ff = 0;
-    const float *norm = nullptr, *ls1 = nullptr, *ls2 = nullptr, *gate_b = nullptr, *up_b = nullptr, *down_b = nullptr;
+    const float *norm = nullptr, *norm2 = nullptr, *ls1 = nullptr, *ls2 = nullptr, *gate_b = nullptr, *up_b = nullptr, *down_b = nullptr;
 };
 
 struct StackModel final : alice_model {
     alice_stack_config cfg{};
     std::vector<StackLayer> layers;
-    DenseMat embed;
+    DenseMat embed, out_head;
     const float *final_norm = nullptr, *loop_step = nullptr;
+    const float* pending = nullptr;   // weight of a norm that still stands between s.r and the stream (single tokens, norm after the sum)
     Scratch s;
     uint32_t chunk = 0;
     float* trace = nullptr;
@@ -85,7 +87,16 @@ struct StackModel final : alice_model {
     }
 
     int body(uint32_t n);
-    int layer(uint32_t i, uint32_t n, uint32_t pass);
+    int layer(uint32_t i, uint32_t n, uint32_t pass) { return cfg.block == ALICE_BLOCK_POST ? layer_post(i, n, pass) : layer_parallel(i, n, pass); }
+    int layer_parallel(uint32_t i, uint32_t n, uint32_t pass);
+    int layer_post(uint32_t i, uint32_t n, uint32_t pass);
+    int settle();
+    int norm() const { return cfg.norm == ALICE_NORM_RMS ? NORM_RMS : NORM_LAYER; }
+    NormArgs norm_args(const float* w, bool low) const {
+        NormArgs na;
+        na.x = s.x; na.ldx = s.wp; na.n = cfg.width; na.k = s.wp; na.norm = norm(); na.w = w; na.eps = cfg.eps; na.out = s.h; na.out_bf16 = low;
+        return na;
+    }
     int head(uint32_t n, const uint32_t* rows, uint32_t nrows, bool argmax);
     int product(GemmOp& op) {
         MCU(launch_dense_gemm(op, e->num_sms, e->status, e->stream, e->pdl));
@@ -202,30 +213,67 @@ struct DeltaMixer final : Mixer {
     }
 };
 
+struct GroupedMixer final : Mixer {
+    GroupedShape sh{};
+    const float *sink = nullptr, *freq = nullptr;
+    std::vector<void*> cache;      // per pass, [kv_heads][plane_rows][ld]
+    uint32_t plane_rows = 0;
+    size_t cache_bytes = 0;
+
+    bool recurrent() const override { return false; }
+    bool tiled(const StackModel* m) const { return !m->exact() && grouped_tiled_fits(sh); }
+    uint32_t head_groups() const { return sh.kv_heads * ((sh.group() + 15) / 16); }   // CTAs of a share of the context
+    int clear(cudaStream_t st) override {
+        for (void* c : cache) MCU(cudaMemsetAsync(c, 0, cache_bytes, st));
+        return ALICE_OK;
+    }
+    int run(StackModel* m, uint32_t n, uint32_t pass) override {
+        Scratch& s = m->s;
+        cudaStream_t st = m->e->stream;
+        const bool pdl = m->e->pdl;
+        GroupedArgs a;
+        a.s = sh; a.y = s.y; a.ldy = s.ldy; a.sink = sink; a.freq = freq; a.eps = m->cfg.eps; a.pos = m->d_pos; a.cache = cache[pass]; a.plane_rows = plane_rows;
+        a.cache_bf16 = !m->exact(); a.q = m->exact() ? (void*)s.q : (void*)s.q_rot; a.out = s.a; a.ldo = o.k; a.act_bf16 = m->tiled_bf16(n);
+        a.part = s.part; a.tickets = s.tickets; a.status = m->e->status;
+        const bool few = n <= FEW_TOKENS && tiled(m);
+        a.append = few && n == 1;
+        if (!a.append) MCU(launch_grouped_prepare(a, n, st, pdl));
+        if (few) {
+            // one CTA per SM: shares of the context times heads times tokens
+            a.splits = std::max<uint32_t>(1, std::min(DECODE_SPLITS, (uint32_t)m->e->num_sms / head_groups()) / n);
+            MCU(launch_grouped_decode(a, n, st, pdl));
+        } else if (tiled(m)) {
+            MCU(launch_grouped_prefill(a, n, st, pdl));
+        } else {
+            MCU(launch_grouped_attn(a, n, st, pdl));
+        }
+        return ALICE_OK;
+    }
+};
+
 // ---- the step -------------------------------------------------------------------------------------------
 
-int StackModel::layer(uint32_t i, uint32_t n, uint32_t pass) {
+// x + ls1 * mixer(h) + ls2 * mlp(h), both of the same normalised stream.
+int StackModel::layer_parallel(uint32_t i, uint32_t n, uint32_t pass) {
     StackLayer& L = layers[i];
     Mixer& mx = *L.mixer;
     cudaStream_t st = e->stream;
     const bool low = tiled_bf16(n);
     if (n == 1) {
         RowsIn in;
-        in.x = s.x; in.n_x = cfg.width; in.norm = NORM_LAYER; in.norm_w = L.norm; in.eps = cfg.eps;
+        in.x = s.x; in.n_x = cfg.width; in.norm = norm(); in.norm_w = L.norm; in.eps = cfg.eps;
         in.w0 = mx.in; in.y0 = s.y;
         if (L.ff) { in.gu = L.gu; in.gate_b = L.gate_b; in.up_b = L.up_b; in.y1 = static_cast<float*>(s.f); }
         MCU(launch_rows_in(in, e->num_sms, st, e->pdl));
         const int rc = mx.run(this, n, pass);
         if (rc) return rc;
         RowsOut out;
-        out.w1 = mx.o; out.a = static_cast<const float*>(s.a); out.s1 = L.ls1; out.x = s.x;
+        out.w1 = mx.o; out.a = static_cast<const float*>(s.a); out.s1 = L.ls1; out.x = out.out = s.x;
         if (L.ff) { out.w2 = L.down; out.f = static_cast<const float*>(s.f); out.s2 = L.ls2; out.b2 = L.down_b; }
         MCU(launch_rows_out(out, e->num_sms, st, e->pdl));
         return ALICE_OK;
     }
-    NormArgs na;
-    na.x = s.x; na.ldx = s.wp; na.n = cfg.width; na.k = s.wp; na.w = L.norm; na.eps = cfg.eps; na.out = s.h; na.out_bf16 = low;
-    MCU(launch_layer_norm(na, n, st, e->pdl));
+    MCU(launch_norm(norm_args(L.norm, low), n, st, e->pdl));
     int rc;
     {
         GemmOp op;
@@ -250,17 +298,91 @@ int StackModel::layer(uint32_t i, uint32_t n, uint32_t pass) {
     return ALICE_OK;
 }
 
+// x <- norm1(alpha * x + mixer(x)), x <- norm2(alpha * x + mlp(x)). A single token's sum stays in s.r until the next product
+// takes its norm on the way in and leaves the stream in s.x; of several tokens the stream is also kept in s.h as the products read it.
+int StackModel::layer_post(uint32_t i, uint32_t n, uint32_t pass) {
+    StackLayer& L = layers[i];
+    Mixer& mx = *L.mixer;
+    cudaStream_t st = e->stream;
+    const bool low = tiled_bf16(n);
+    int rc;
+    if (n == 1) {
+        RowsIn in;
+        in.n_x = cfg.width; in.eps = cfg.eps;
+        in.x = pending ? s.r : s.x; in.norm = pending ? norm() : NORM_NONE; in.norm_w = pending; in.h_out = pending ? s.x : nullptr;
+        in.w0 = mx.in; in.y0 = s.y;
+        MCU(launch_rows_in(in, e->num_sms, st, e->pdl));
+        if ((rc = mx.run(this, n, pass))) return rc;
+        RowsOut out;
+        out.w1 = mx.o; out.a = static_cast<const float*>(s.a); out.alpha = cfg.alpha; out.x = s.x; out.out = s.r;
+        MCU(launch_rows_out(out, e->num_sms, st, e->pdl));
+        pending = L.norm;
+        if (!L.ff) return ALICE_OK;
+        in = RowsIn();
+        in.n_x = cfg.width; in.eps = cfg.eps; in.x = s.r; in.norm = norm(); in.norm_w = pending; in.h_out = s.x;
+        in.gu = L.gu; in.gate_b = L.gate_b; in.up_b = L.up_b; in.y1 = static_cast<float*>(s.f);
+        MCU(launch_rows_in(in, e->num_sms, st, e->pdl));
+        out.w1 = L.down; out.a = static_cast<const float*>(s.f);
+        MCU(launch_rows_out(out, e->num_sms, st, e->pdl));
+        pending = L.norm2;
+        return ALICE_OK;
+    }
+    GemmOp op;
+    op.tokens = n; op.a = s.h; op.lda = s.wp; op.a_bf16 = low; op.w = mx.in; op.out = s.y; op.ldo = s.ldy;
+    if (low && mx.low_column() < mx.in.n) { op.out2 = s.low; op.col2 = mx.low_column(); op.ld2 = mx.in.n - op.col2; }
+    if ((rc = product(op))) return rc;
+    if ((rc = mx.run(this, n, pass))) return rc;
+    auto join = [&](const void* a, const DenseMat& w, const float* norm_w) -> int {
+        GemmOp op;
+        op.tokens = n; op.a = a; op.lda = w.k; op.a_bf16 = low; op.w = w; op.epi = EPI_RESID; op.out = s.x; op.ldo = s.wp; op.alpha = cfg.alpha;
+        const int rc = product(op);
+        if (rc) return rc;
+        NormArgs na = norm_args(norm_w, low);
+        na.x_out = s.x;
+        MCU(launch_norm(na, n, st, e->pdl));
+        return ALICE_OK;
+    };
+    if ((rc = join(s.a, mx.o, L.norm)) || !L.ff) return rc;
+    op = GemmOp();
+    op.tokens = n; op.a = s.h; op.lda = s.wp; op.a_bf16 = low; op.w = L.gu; op.epi = EPI_SWIGLU; op.out = s.f; op.ldo = L.down.k; op.out_bf16 = low;
+    op.bias = L.gate_b; op.bias2 = L.up_b;
+    if ((rc = product(op))) return rc;
+    return join(s.f, L.down, L.norm2);
+}
+
+// The stream in s.x, whatever norm still stands before it.
+int StackModel::settle() {
+    if (!pending) return ALICE_OK;
+    NormArgs na = norm_args(pending, false);
+    na.x = s.r; na.x_out = s.x; na.out = nullptr;
+    MCU(launch_norm(na, 1, e->stream, e->pdl));
+    pending = nullptr;
+    return ALICE_OK;
+}
+
 int StackModel::body(uint32_t n) {
     cudaStream_t st = e->stream;
     EnterArgs ea;
     ea.emb = embed.w; ea.tokens = d_token; ea.vocab = vocab; ea.emb_ld = embed.k; ea.n = cfg.width; ea.ld = s.wp; ea.scale = cfg.embed_scale;
     ea.set = true; ea.x = s.x;
     MCU(launch_enter(ea, n, st, e->pdl));
+    pending = nullptr;
+    // with the norm behind the sum, layers read the stream itself: its copy as the products take it
+    auto copy = [&]() -> int {
+        if (cfg.block != ALICE_BLOCK_POST || n == 1) return ALICE_OK;
+        NormArgs na = norm_args(nullptr, tiled_bf16(n));
+        na.norm = NORM_NONE;
+        MCU(launch_norm(na, n, st, e->pdl));
+        return ALICE_OK;
+    };
+    int rc = copy();
+    if (rc) return rc;
     trace_runs = 0; trace_tokens = n;
     auto one = [&](uint32_t i, uint32_t pass) -> int {
-        const int rc = layer(i, n, pass);
+        int rc = layer(i, n, pass);
         if (rc) return rc;
         if (tracing) {
+            if ((rc = settle())) return rc;
             MCU(cudaMemcpy2DAsync(trace + (size_t)trace_runs * n * cfg.width, (size_t)cfg.width * 4, s.x, (size_t)s.wp * 4, (size_t)cfg.width * 4, n,
                                   cudaMemcpyDeviceToDevice, st));
             trace_runs++;
@@ -268,38 +390,38 @@ int StackModel::body(uint32_t n) {
         return ALICE_OK;
     };
     const uint32_t a = cfg.loop_times ? cfg.loop_start : cfg.num_layers, b = cfg.loop_times ? cfg.loop_stop : cfg.num_layers;
-    int rc;
     for (uint32_t i = 0; i < a; i++) if ((rc = one(i, 0))) return rc;
     for (uint32_t t = 0; t < cfg.loop_times; t++) {
         EnterArgs la = ea;
         la.set = false;
         if (t == 0) la.emb = nullptr;
         la.step = loop_step + (size_t)t * cfg.width;
+        if ((rc = settle())) return rc;
         if (b > a) MCU(launch_enter(la, n, st, e->pdl));
+        if (b > a && (rc = copy())) return rc;
         for (uint32_t i = a; i < b; i++) if ((rc = one(i, t))) return rc;
     }
     for (uint32_t i = b; i < cfg.num_layers; i++) if ((rc = one(i, 0))) return rc;
-    return ALICE_OK;
+    return settle();
 }
 
 // Logits of the given rows of the stream (at most MAX_NORM_ROWS).
 int StackModel::head(uint32_t n, const uint32_t* rows, uint32_t nrows, bool argmax) {
     if (nrows == 1) {
         RowsIn in;
-        in.x = s.x + (size_t)rows[0] * s.wp; in.n_x = cfg.width; in.norm = NORM_LAYER; in.norm_w = final_norm; in.eps = cfg.eps;
-        in.w0 = embed; in.y0 = logits;
+        in.x = s.x + (size_t)rows[0] * s.wp; in.n_x = cfg.width; in.norm = norm(); in.norm_w = final_norm; in.eps = cfg.eps;
+        in.w0 = out_head; in.y0 = logits;
         if (argmax) in.argmax_key = argmax_keys;
         MCU(launch_rows_in(in, e->num_sms, e->stream, e->pdl));
         return ALICE_OK;
     }
     const bool low = tiled_bf16(n);
-    NormArgs na;
-    na.x = s.x; na.ldx = s.wp; na.n = cfg.width; na.k = s.wp; na.w = final_norm; na.eps = cfg.eps; na.out = s.h; na.out_bf16 = low;
+    NormArgs na = norm_args(final_norm, low);
     na.gather = true;
     for (uint32_t i = 0; i < nrows; i++) na.idx[i] = rows[i];
-    MCU(launch_layer_norm(na, nrows, e->stream, e->pdl));
+    MCU(launch_norm(na, nrows, e->stream, e->pdl));
     GemmOp op;
-    op.tokens = nrows; op.a = s.h; op.lda = s.wp; op.a_bf16 = low; op.w = embed; op.out = logits; op.ldo = vocab;
+    op.tokens = nrows; op.a = s.h; op.lda = s.wp; op.a_bf16 = low; op.w = out_head; op.out = logits; op.ldo = vocab;
     return product(op);
 }
 
@@ -372,6 +494,26 @@ struct Builder {
 
 uint32_t P(uint32_t v) { return pad_to(v, DENSE_PAD); }
 
+// Frequencies of the rotated pairs, in double and rounded once. With a factor, wavelengths above original / low turn that much
+// slower, those below original / high stay, and between the two the share of the original grows linearly.
+const float* rotation(Builder& b, const alice_stack_layer& L) {
+    std::vector<float> f(std::max<uint32_t>(1, L.rot_dims / 2));
+    for (uint32_t i = 0; i < L.rot_dims / 2; i++) {
+        double x = std::pow(L.rot_base, -2.0 * i / L.rot_dims);
+        if (L.rot_factor != 0.0) {
+            const double wave = 2.0 * 3.14159265358979323846 / x;
+            if (wave > L.rot_original / L.rot_low) {
+                x /= L.rot_factor;
+            } else if (wave >= L.rot_original / L.rot_high && L.rot_high > L.rot_low) {
+                const double keep = (L.rot_original / wave - L.rot_low) / (L.rot_high - L.rot_low);
+                x = (1.0 - keep) * x / L.rot_factor + keep * x;
+            }
+        }
+        f[i] = (float)x;
+    }
+    return b.floats(f.data(), f.size(), "freq");
+}
+
 void build_latent(Builder& b, const alice_stack_layer& L, uint32_t wp, uint32_t passes, LatentMixer& mx) {
     StackModel* m = b.m;
     LatentShape& s = mx.sh;
@@ -389,9 +531,7 @@ void build_latent(Builder& b, const alice_stack_layer& L, uint32_t wp, uint32_t 
     mx.q_norm = b.floats(L.q_norm, L.q_rank, "q_norm");
     mx.kv_norm = b.floats(L.kv_norm, L.kv_rank, "kv_norm");
     mx.sink = b.floats(L.sink, L.heads, "sink");
-    std::vector<float> f(std::max<uint32_t>(1, L.rot_dims / 2));
-    for (uint32_t i = 0; i < L.rot_dims / 2; i++) f[i] = (float)std::pow(L.rot_base, -2.0 * i / L.rot_dims);
-    mx.freq = b.floats(f.data(), f.size(), "freq");
+    mx.freq = rotation(b, L);
     mx.cache_bytes = (size_t)m->max_seq * (s.cp + s.rp) * (m->exact() ? 4 : 2);
     for (uint32_t p = 0; p < passes; p++) mx.cache.push_back(b.zeros<uint8_t>(mx.cache_bytes));
 }
@@ -421,6 +561,26 @@ void build_delta(Builder& b, const alice_stack_layer& L, uint32_t wp, uint32_t p
     }
 }
 
+void build_grouped(Builder& b, const alice_stack_layer& L, uint32_t wp, uint32_t passes, GroupedMixer& mx) {
+    StackModel* m = b.m;
+    GroupedShape& s = mx.sh;
+    if (!L.heads || !L.kv_heads || L.heads % L.kv_heads || !L.dim || !L.vdim) return b.shape("grouped mixer with a zero size, or heads no multiple of kv_heads");
+    if (L.rot_dims % 2 || L.rot_dims > L.dim) return b.shape("rotated dimensions must be even and lie within dim");
+    if (L.dim > GROUPED_MAX_DIM || L.vdim > GROUPED_MAX_DIM) return b.shape("grouped mixer with more than 512 dimensions a head");
+    if (L.softcap < 0.0f) return b.shape("negative softcap");
+    s.heads = L.heads; s.kv_heads = L.kv_heads; s.dim = L.dim; s.vdim = L.vdim; s.rot_dims = L.rot_dims; s.dp = pad_to(L.dim, 16); s.vp = pad_to(L.vdim, 16);
+    s.off_k = P(L.heads * L.dim); s.off_v = s.off_k + P(L.kv_heads * L.dim); s.scale = L.scale; s.softcap = L.softcap; s.unit_qk = L.unit_qk != 0;
+    mx.in = b.matrix(L.in, s.off_v + P(L.kv_heads * L.vdim), wp, "in");
+    mx.o = b.matrix(L.o, m->cfg.width, P(L.heads * L.vdim), "o");
+    const std::vector<float> none(L.heads, -INFINITY);
+    mx.sink = b.floats(L.sink ? L.sink : none.data(), L.heads, "sink");
+    mx.freq = rotation(b, L);
+    mx.plane_rows = pad_to(m->max_seq, 64);
+    static_assert(64 % GROUPED_TILE == 0, "whole tiles in a plane");
+    mx.cache_bytes = (size_t)L.kv_heads * mx.plane_rows * s.ld() * (m->exact() ? 4 : 2);
+    for (uint32_t p = 0; p < passes; p++) mx.cache.push_back(b.zeros<uint8_t>(mx.cache_bytes));
+}
+
 // Scratch for the largest layer of each kind.
 void build_scratch(Builder& b) {
     StackModel* m = b.m;
@@ -431,7 +591,7 @@ void build_scratch(Builder& b) {
         if (const auto* x = dynamic_cast<const LatentMixer*>(L.mixer.get())) small |= !x->tiled(m);
     m->chunk = std::min<uint32_t>(small ? CHUNK_SMALL : CHUNK, pad_to(m->max_seq, 64));
     const uint32_t M = m->chunk, ML = small ? M : std::min(M, FEW_TOKENS);
-    uint32_t k_all = 0, v_all = 0;
+    uint32_t k_all = 0, v_all = 0, q_rot = 0, few = 0, tickets = 0;   // few: partial sums of a share, for FEW_TOKENS at once
     uint32_t ldy = 0, ldf = 0, lda = 0, q = 0, ql = 0, part = 0, mix = 0, qp = 0, kd = 0, v = 0, h = 0, g = 0, o = 0, low = 0;
     for (const auto& L : m->layers) {
         ldy = std::max(ldy, L.mixer->in.n);
@@ -439,9 +599,13 @@ void build_scratch(Builder& b) {
         ldf = std::max(ldf, L.down.k);
         if (const auto* x = dynamic_cast<const LatentMixer*>(L.mixer.get())) {
             const LatentShape& z = x->sh;
-            if (x->tiled(m)) { k_all = std::max(k_all, x->uk.n); v_all = std::max(v_all, x->uv.n); }
+            if (x->tiled(m)) { k_all = std::max(k_all, x->uk.n); v_all = std::max(v_all, x->uv.n); q_rot = std::max(q_rot, x->uq.n); }
             q = std::max(q, x->uq.n); qp = std::max(qp, z.qp);
             ql = std::max(ql, z.heads * (z.cp + z.rp)); part = std::max(part, z.heads * (z.cp + 2)); mix = std::max(mix, z.heads * z.cp);
+        } else if (const auto* x = dynamic_cast<const GroupedMixer*>(L.mixer.get())) {
+            const GroupedShape& z = x->sh;
+            (m->exact() ? q : q_rot) = std::max(m->exact() ? q : q_rot, z.heads * z.dp);
+            if (x->tiled(m)) { few = std::max(few, z.heads * (z.vp + 4)); tickets = std::max(tickets, FEW_TOKENS * x->head_groups()); }
         } else if (const auto* x = dynamic_cast<const DeltaMixer*>(L.mixer.get())) {
             const DeltaShape& z = x->sh;
             kd = std::max(kd, z.kv_heads * z.dp); v = std::max(v, z.heads * z.vp); h = std::max(h, z.heads);
@@ -451,16 +615,18 @@ void build_scratch(Builder& b) {
     s.chunk = M; s.wp = P(m->cfg.width); s.ldy = ldy;
     s.x = b.zeros<float>((size_t)M * s.wp);
     s.y = b.zeros<float>((size_t)M * ldy);
+    s.r = b.zeros<float>(s.wp);
     s.h = b.zeros<float>((size_t)M * s.wp);
     s.f = b.zeros<float>((size_t)M * ldf);
     s.a = b.zeros<float>((size_t)M * lda);     // heads * vdim columns and the padding of each mixer's own stride
     s.q = b.zeros<float>((size_t)M * q);
     s.cqn = b.zeros<float>((size_t)M * qp);
     s.ql = b.zeros<float>((size_t)ML * ql);
-    s.part = b.zeros<float>((size_t)std::max(ML, DECODE_SPLITS) * part);
+    s.part = b.zeros<float>(std::max((size_t)std::max(ML, DECODE_SPLITS) * part, (size_t)std::max(FEW_TOKENS, DECODE_SPLITS) * few));
+    s.tickets = b.zeros<unsigned int>(tickets);
     s.mix = b.zeros<float>((size_t)ML * mix);
     s.k_all = b.zeros<bf16>((size_t)m->max_seq * k_all);
-    s.q_rot = b.zeros<bf16>(k_all ? (size_t)M * q : 0);
+    s.q_rot = b.zeros<bf16>((size_t)M * q_rot);
     s.v_all = b.zeros<bf16>((size_t)m->max_seq * v_all);
     s.qn = b.zeros<float>((size_t)M * kd); s.kn = b.zeros<float>((size_t)M * kd);
     s.pair_inv = b.zeros<float>((size_t)M * h * DELTA_BLOCK); s.pair_b = b.zeros<float>((size_t)M * h * DELTA_BLOCK);
@@ -487,6 +653,7 @@ int32_t alice_stack_create(alice_engine* e, const alice_stack_config* cfg, const
     if (!c.num_layers || !c.width || !c.vocab_size || !c.max_seq_len) return alice_fail(ALICE_E_SHAPE, "%s: zero dimension in config", who);
     if (c.loop_times && (c.loop_start > c.loop_stop || c.loop_stop > c.num_layers || !c.loop_step))
         return alice_fail(ALICE_E_SHAPE, "%s: loop %u .. %u of %u layers", who, c.loop_start, c.loop_stop, c.num_layers);
+    if (c.block > ALICE_BLOCK_POST || c.norm > ALICE_NORM_RMS) return alice_fail(ALICE_E_UNSUPPORTED, "%s: block %u, norm %u", who, c.block, c.norm);
     if (e->tp_world > 1) return alice_fail(ALICE_E_UNSUPPORTED, "%s: layer-stack models run on one GPU", who);
     MCU(cudaSetDevice(e->device));
     auto* m = new StackModel();
@@ -495,6 +662,7 @@ int32_t alice_stack_create(alice_engine* e, const alice_stack_config* cfg, const
     Builder b{m};
     const uint32_t wp = P(c.width);
     m->embed = b.matrix(embed, c.vocab_size, wp, "embed");
+    m->out_head = c.head ? b.matrix(c.head, c.vocab_size, wp, "head") : m->embed;
     m->final_norm = b.floats(final_norm, c.width, "final_norm");
     if (c.loop_times) m->loop_step = b.floats(c.loop_step, (size_t)c.loop_times * c.width, "loop_step");
     for (uint32_t i = 0; i < c.num_layers && !b.rc; i++) {
@@ -509,20 +677,29 @@ int32_t alice_stack_create(alice_engine* e, const alice_stack_config* cfg, const
             auto mx = std::make_unique<DeltaMixer>();
             build_delta(b, L, wp, passes, *mx);
             sl.mixer = std::move(mx);
+        } else if (L.mixer == ALICE_MIX_GROUPED) {
+            auto mx = std::make_unique<GroupedMixer>();
+            build_grouped(b, L, wp, passes, *mx);
+            sl.mixer = std::move(mx);
         } else {
             b.rc = alice_fail(ALICE_E_UNSUPPORTED, "%s: layer %u has an unknown mixer %u", who, i, L.mixer);
             break;
         }
         sl.norm = b.floats(L.norm, c.width, "norm");
-        sl.ls1 = b.floats(L.ls1, c.width, "ls1");
+        const bool post = c.block == ALICE_BLOCK_POST;
+        auto optional = [&](const float* p, size_t n, const char* name) { return p ? b.floats(p, n, name) : nullptr; };
+        if (!post) sl.ls1 = b.floats(L.ls1, c.width, "ls1");
         if (L.ff) {
             sl.ff = L.ff;
             sl.gu = b.matrix(L.gu, 2 * P(L.ff), wp, "gu");
             sl.down = b.matrix(L.down, c.width, P(L.ff), "down");
-            sl.ls2 = b.floats(L.ls2, c.width, "ls2");
-            sl.gate_b = b.floats(L.gate_bias, P(L.ff), "gate_bias");
-            sl.up_b = b.floats(L.up_bias, P(L.ff), "up_bias");
-            sl.down_b = b.floats(L.down_bias, c.width, "down_bias");
+            if (post) sl.norm2 = b.floats(L.norm2, c.width, "norm2");
+            else sl.ls2 = b.floats(L.ls2, c.width, "ls2");
+            if (post && L.down_bias) b.shape("a bias on the way out of a feed-forward whose norm comes behind the sum");
+            if (!L.gate_bias != !L.up_bias) b.shape("gate and up biases come together");
+            sl.gate_b = optional(L.gate_bias, P(L.ff), "gate_bias");
+            sl.up_b = optional(L.up_bias, P(L.ff), "up_bias");
+            if (!post) sl.down_b = b.floats(L.down_bias, c.width, "down_bias");
         }
         m->layers.push_back(std::move(sl));
     }

@@ -1,7 +1,8 @@
 // Small per-token kernels of layer-stack models: the embedding (and what re-enters the stream before a looped pass) and the
-// layer norm ahead of a tiled product.
+// norms ahead of or behind a tiled product.
 #include "dense_dev.cuh"
 #include "mixers.cuh"
+#include "mma_sync.cuh"
 
 namespace alice {
 namespace {
@@ -22,16 +23,67 @@ __global__ void __launch_bounds__(1024) enter_kernel(const __grid_constant__ Ent
     }
 }
 
-template <class OT>
-__global__ void __launch_bounds__(256) layer_norm_kernel(const __grid_constant__ NormArgs a) {
-    extern __shared__ __align__(16) float h[];
+// The row is held in registers: a thread owns every 256th group of four elements (NV groups; rows up to 1024 * NV wide).
+template <class OT, int NV>
+__global__ void __launch_bounds__(256) norm_kernel(const __grid_constant__ NormArgs a) {
     __shared__ float red[8];
     pdl_launch_dependents();
     pdl_wait();
     const uint32_t t = blockIdx.x, src = a.gather ? a.idx[t] : t;
-    load_normed<8>(h, a.x + (size_t)src * a.ldx, a.n, a.k, NORM_LAYER, a.w, a.eps, red);
+    const float* x = a.x + (size_t)src * a.ldx;
+    float v[NV][4];
+    float s = 0.0f;
+#pragma unroll
+    for (int j = 0; j < NV; j++) {
+        const uint32_t c = (threadIdx.x + j * 256) * 4;
+        const float4 u = c < a.k ? *reinterpret_cast<const float4*>(x + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        v[j][0] = u.x; v[j][1] = u.y; v[j][2] = u.z; v[j][3] = u.w;
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            if (c + i >= a.n) v[j][i] = 0.0f;
+            s += a.norm == NORM_LAYER ? v[j][i] : v[j][i] * v[j][i];
+        }
+    }
+    float mean = 0.0f, inv = 1.0f;
+    if (a.norm != NORM_NONE) {
+        s = block_sum<8>(s, red);
+        if (a.norm == NORM_LAYER) {
+            mean = s / (float)a.n;
+            float q = 0.0f;
+#pragma unroll
+            for (int j = 0; j < NV; j++)
+#pragma unroll
+                for (int i = 0; i < 4; i++)
+                    if ((threadIdx.x + j * 256) * 4 + i < a.n) { const float d = v[j][i] - mean; q += d * d; }
+            s = block_sum<8>(q, red);
+        }
+        inv = __frcp_rn(__fsqrt_rn(s / (float)a.n + a.eps));
+    }
     OT* out = static_cast<OT*>(a.out) + (size_t)t * a.k;
-    for (uint32_t i = threadIdx.x; i < a.k; i += 256) put(out + i, h[i]);
+#pragma unroll
+    for (int j = 0; j < NV; j++) {
+        const uint32_t c = (threadIdx.x + j * 256) * 4;
+        if (c >= a.k) break;
+        if (a.norm != NORM_NONE)
+#pragma unroll
+            for (int i = 0; i < 4; i++) v[j][i] = c + i < a.n ? (v[j][i] - mean) * inv * a.w[c + i] : 0.0f;
+        if (a.out) {
+            if constexpr (sizeof(OT) == 2) {
+                *reinterpret_cast<uint2*>(out + c) = make_uint2(pack_bf16(v[j][0], v[j][1]), pack_bf16(v[j][2], v[j][3]));
+            } else {
+                *reinterpret_cast<float4*>(out + c) = make_float4(v[j][0], v[j][1], v[j][2], v[j][3]);
+            }
+        }
+        if (a.x_out) *reinterpret_cast<float4*>(a.x_out + (size_t)t * a.ldx + c) = make_float4(v[j][0], v[j][1], v[j][2], v[j][3]);
+    }
+}
+
+template <class OT>
+cudaError_t norm_type(const NormArgs& a, uint32_t rows, cudaStream_t st, bool pdl) {
+    if (a.k <= 1024) return launch_pdl(norm_kernel<OT, 1>, dim3(rows), dim3(256), 0, st, pdl, a);
+    if (a.k <= 4096) return launch_pdl(norm_kernel<OT, 4>, dim3(rows), dim3(256), 0, st, pdl, a);
+    if (a.k <= 16384) return launch_pdl(norm_kernel<OT, 16>, dim3(rows), dim3(256), 0, st, pdl, a);
+    return launch_pdl(norm_kernel<OT, 56>, dim3(rows), dim3(256), 0, st, pdl, a);
 }
 
 }  // namespace
@@ -40,13 +92,9 @@ cudaError_t launch_enter(const EnterArgs& a, uint32_t tokens, cudaStream_t st, b
     return launch_pdl(enter_kernel, dim3(tokens), dim3(a.n > 512 ? 1024 : 256), 0, st, pdl, a);
 }
 
-cudaError_t launch_layer_norm(const NormArgs& a, uint32_t rows, cudaStream_t st, bool pdl) {
-    if (a.gather && rows > MAX_NORM_ROWS) return cudaErrorInvalidValue;
-    static bool done_f[64] = {}, done_b[64] = {};
-    cudaError_t err = a.out_bf16 ? allow_smem(layer_norm_kernel<bf16>, 224 * 1024, done_b) : allow_smem(layer_norm_kernel<float>, 224 * 1024, done_f);
-    if (err != cudaSuccess) return err;
-    return a.out_bf16 ? launch_pdl(layer_norm_kernel<bf16>, dim3(rows), dim3(256), (size_t)a.k * 4, st, pdl, a)
-                      : launch_pdl(layer_norm_kernel<float>, dim3(rows), dim3(256), (size_t)a.k * 4, st, pdl, a);
+cudaError_t launch_norm(const NormArgs& a, uint32_t rows, cudaStream_t st, bool pdl) {
+    if ((a.gather && rows > MAX_NORM_ROWS) || a.k % 4 || a.ldx % 4 || a.k > 56 * 1024 || a.ldx < a.k || (a.gather && a.x_out)) return cudaErrorInvalidValue;
+    return a.out_bf16 ? norm_type<bf16>(a, rows, st, pdl) : norm_type<float>(a, rows, st, pdl);
 }
 
 }  // namespace alice

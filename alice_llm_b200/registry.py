@@ -21,7 +21,7 @@ def _stack(engine, path, dtype, max_seq_len):
 
 
 # architecture -> (loader, part of the native library it runs on)
-ARCHITECTURES = {"llama": (_llama, "all"), "Zamitar": (_stack, "stack")}
+ARCHITECTURES = {"llama": (_llama, "all"), "Zamitar": (_stack, "stack"), "Suborax": (_stack, "stack")}
 
 
 def architecture_of(path) -> str:

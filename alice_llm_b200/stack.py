@@ -11,9 +11,27 @@ import numpy as np
 from . import _lib
 from .safetensors_file import SafetensorsFile, bf16_to_f32
 
-MIX_LATENT, MIX_DELTA = 1, 2
-MIXERS = {"latent_attention": MIX_LATENT, "channel_delta": MIX_DELTA}
+MIX_LATENT, MIX_DELTA, MIX_GROUPED = 1, 2, 3
+BLOCK_PARALLEL, BLOCK_POST = 0, 1
+NORM_LAYER, NORM_RMS = 0, 1
 PAD = 64          # columns, and row segments of packed matrices, come in multiples of this
+
+
+class Family:
+    """What an architecture fixes, whatever its sizes."""
+
+    def __init__(self, mixers, block, norm, norm_offset=0.0, mlp_bias=False, tied=True, unit_qk=False):
+        self.mixers, self.block, self.norm = mixers, block, norm
+        self.norm_offset = norm_offset      # added to stored norm weights
+        self.mlp_bias = mlp_bias            # gate, up and down have biases
+        self.tied = tied                    # the embedding table is the head
+        self.unit_qk = unit_qk              # rotated queries and keys over their root mean square
+
+
+FAMILIES = {
+    "Zamitar": Family({"latent_attention": MIX_LATENT, "channel_delta": MIX_DELTA}, BLOCK_PARALLEL, NORM_LAYER, mlp_bias=True),
+    "Suborax": Family({"attention": MIX_GROUPED}, BLOCK_POST, NORM_RMS, norm_offset=1.0, tied=False, unit_qk=True),
+}
 
 
 class ConfigError(ValueError):
@@ -50,28 +68,32 @@ def _number(d: dict, key: str, where: str) -> float:
 class LayerSpec:
     """One layer: mixer kind and sizes, feed-forward width (0 = none)."""
 
-    LATENT_SIZES = ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank")
-    DELTA_SIZES = ("heads", "kv_heads", "dim", "vdim")
+    SIZES = {MIX_LATENT: ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank"), MIX_DELTA: ("heads", "kv_heads", "dim", "vdim"),
+             MIX_GROUPED: ("heads", "kv_heads", "dim", "vdim")}
 
-    def __init__(self, d: dict, where: str):
+    def __init__(self, d: dict, where: str, family: Family):
         kind = d.get("type")
-        if kind not in MIXERS:
-            raise ConfigError(f"{where}: mixer {kind!r} (known: {', '.join(MIXERS)})")
-        self.kind, m = MIXERS[kind], d["mixer"]
+        if kind not in family.mixers:
+            raise ConfigError(f"{where}: mixer {kind!r} (known: {', '.join(family.mixers)})")
+        self.kind, m = family.mixers[kind], d["mixer"]
         self.heads = self.kv_heads = self.dim = self.vdim = self.q_rank = self.kv_rank = self.rot_dim = self.rot_dims = 0
         self.conv_taps = self.decay_rank = self.gate_rank = 0
         self.scale = self.rot_base = 1.0
-        for key in self.LATENT_SIZES if self.kind == MIX_LATENT else self.DELTA_SIZES:
+        self.softcap = self.rot_factor = self.rot_low = self.rot_high = self.rot_original = 0.0
+        self.unit_qk = int(family.unit_qk)
+        for key in self.SIZES[self.kind]:
             setattr(self, key, _size(m, key, where))
-        if self.kind == MIX_LATENT:
+        if self.kind != MIX_DELTA:
             self.scale = _number(m, "scale", where)
-            self.rot_dims, self.rot_base = _size(m["rot"], "dims", where), _number(m["rot"], "base", where)
-            if self.rot_dims % 2 or self.rot_dims > self.rot_dim:
-                raise ConfigError(f"{where}: {self.rot_dims} rotated dimensions of {self.rot_dim}")
+            self._rotation(m.get("rot"), self.rot_dim if self.kind == MIX_LATENT else self.dim, where)
         else:
             self.conv_taps = _size(m, "conv", where)
-            if self.heads % self.kv_heads:
-                raise ConfigError(f"{where}: {self.heads} heads do not divide over {self.kv_heads} key heads")
+        if self.kind == MIX_GROUPED and m.get("softcap") is not None:
+            self.softcap = _number(m, "softcap", where)
+            if self.softcap <= 0:
+                raise ConfigError(f"{where}: softcap = {self.softcap}")
+        if self.kind != MIX_LATENT and self.heads % self.kv_heads:
+            raise ConfigError(f"{where}: {self.heads} heads do not divide over {self.kv_heads} key heads")
         self.ff = 0
         mlp = d.get("mlp")
         if mlp:
@@ -79,10 +101,27 @@ class LayerSpec:
                 raise ConfigError(f"{where}: feed-forward {mlp.get('kind')!r} (known: dense)")
             self.ff = _size(mlp, "ff", where)
 
+    def _rotation(self, rot, room: int, where: str):
+        if not isinstance(rot, dict):
+            raise ConfigError(f"{where}: rot = {rot!r}")
+        self.rot_dims, self.rot_base = _size(rot, "dims", where, 0), _number(rot, "base", where)
+        if self.rot_dims % 2 or self.rot_dims > room:
+            raise ConfigError(f"{where}: {self.rot_dims} rotated dimensions of {room}")
+        if self.rot_base <= 0:
+            raise ConfigError(f"{where}: rot base = {self.rot_base}")
+        if rot.get("scaling"):
+            for key in ("factor", "low", "high", "original"):
+                v = _number(rot["scaling"], key, f"{where}: rot scaling")
+                if v <= 0:
+                    raise ConfigError(f"{where}: rot scaling: {key} = {v}")
+                setattr(self, "rot_" + key, v)
+
     # rows of the packed input projection: (tensor, rows), each starting at a multiple of PAD
     def input_segments(self):
         if self.kind == MIX_LATENT:
             return [("dq", self.q_rank), ("dkv", self.kv_rank + self.rot_dim), ("g", self.heads * self.vdim)]
+        if self.kind == MIX_GROUPED:
+            return [("q", self.heads * self.dim), ("k", self.kv_heads * self.dim), ("v", self.kv_heads * self.vdim)]
         return [("q", self.kv_heads * self.dim), ("k", self.kv_heads * self.dim), ("v", self.heads * self.vdim), ("b", self.heads),
                 ("a1", self.decay_rank), ("g1", self.gate_rank)]
 
@@ -92,7 +131,7 @@ class LayerSpec:
         if self.kind == MIX_LATENT:
             out["uq"] = (self.heads * (self.dim + self.rot_dim), pad(self.q_rank))
             out["uk"], out["uv"] = (self.heads * self.dim, pad(self.kv_rank)), (self.heads * self.vdim, pad(self.kv_rank))
-        else:
+        elif self.kind == MIX_DELTA:
             out["a2"] = (self.heads * delta_dim(self.dim), pad(self.decay_rank))
             out["g2"] = (self.heads * self.vdim, pad(self.gate_rank))
         if self.ff:
@@ -106,9 +145,13 @@ class StackConfig:
     def __init__(self, d: dict, max_seq_len: int):
         where = "config"
         self.architecture = d.get("architecture")
+        if self.architecture not in FAMILIES:
+            raise ConfigError(f"config: architecture {self.architecture!r} (known: {', '.join(FAMILIES)})")
+        self.family = FAMILIES[self.architecture]
         self.vocab_size, self.width = _size(d, "vocab", where), _size(d, "width", where)
         self.eps, self.embed_scale = _number(d["norm"], "eps", "norm"), _number(d["embedding"], "scale", "embedding")
-        self.layers = [LayerSpec(l, f"layer {i}") for i, l in enumerate(d["layers"])]
+        self.alpha = _number(d, "postln_alpha", where) if self.family.block == BLOCK_POST else 1.0
+        self.layers = [LayerSpec(l, f"layer {i}", self.family) for i, l in enumerate(d["layers"])]
         if not self.layers:
             raise ConfigError("config: no layers")
         self.loop_start = self.loop_stop = self.loop_times = 0
@@ -183,20 +226,24 @@ class Checkpoint:
         return bf16_to_f32(a) if a.dtype == np.uint16 else np.asarray(a, np.float32)
 
 
-def pack_layer(ck: Checkpoint, i: int, L: LayerSpec, width: int):
+def pack_layer(ck: Checkpoint, i: int, L: LayerSpec, cfg: "StackConfig"):
     """-> ({matrix name: uint16 array}, {vector name: float32 array}); fills in the ranks only the tensors tell."""
-    p, m = f"l{i}.", f"l{i}.mix."
+    p, m, width, family = f"l{i}.", f"l{i}.mix.", cfg.width, cfg.family
     if L.kind == MIX_DELTA:
         L.decay_rank, L.gate_rank = len(ck.raw(m + "a1")), len(ck.raw(m + "g1"))
     shapes = L.packed_shapes(width)
     H, V = L.heads, L.vdim
     mats = {"in": _rows([ck.matrix(m + n, r, width) for n, r in L.input_segments()], pad(width)),
             "o": _cols(ck.matrix(m + "o", width, H * V), shapes["o"][1])}
-    vecs = {"norm": ck.floats(p + "norm1", width), "ls1": ck.floats(p + "ls1", width)}
+    vecs = {"norm": ck.floats(p + "norm1", width) + np.float32(family.norm_offset)}
+    if family.block == BLOCK_PARALLEL:
+        vecs["ls1"] = ck.floats(p + "ls1", width)
     if L.kind == MIX_LATENT:
         for n, src in (("uq", L.q_rank), ("uk", L.kv_rank), ("uv", L.kv_rank)):
             mats[n] = _cols(ck.matrix(m + n, shapes[n][0], src), shapes[n][1])
         vecs.update(q_norm=ck.floats(m + "dq.norm", L.q_rank), kv_norm=ck.floats(m + "dkv.norm", L.kv_rank), sink=ck.floats(m + "sink", H))
+    elif L.kind == MIX_GROUPED:
+        vecs["sink"] = ck.floats(m + "sink", H)
     else:
         D, dp, K = L.dim, delta_dim(L.dim), L.conv_taps
         a2 = np.zeros((H, dp, L.decay_rank), np.uint16)
@@ -216,15 +263,21 @@ def pack_layer(ck: Checkpoint, i: int, L: LayerSpec, width: int):
         q = f"l{i}.mlp."
         mats["gu"] = _interleave(ck.matrix(q + "gate", L.ff, width), ck.matrix(q + "up", L.ff, width), pad(width))
         mats["down"] = _cols(ck.matrix(q + "down", width, L.ff), shapes["down"][1])
-        vecs.update(ls2=ck.floats(p + "ls2", width), gate_bias=_vec(ck.floats(q + "gate.b", L.ff), pad(L.ff)),
-                    up_bias=_vec(ck.floats(q + "up.b", L.ff), pad(L.ff)), down_bias=ck.floats(q + "down.b", width))
+        if family.block == BLOCK_POST:
+            vecs["norm2"] = ck.floats(p + "norm2", width) + np.float32(family.norm_offset)
+        else:
+            vecs["ls2"] = ck.floats(p + "ls2", width)
+        if family.mlp_bias:
+            vecs.update(gate_bias=_vec(ck.floats(q + "gate.b", L.ff), pad(L.ff)), up_bias=_vec(ck.floats(q + "up.b", L.ff), pad(L.ff)),
+                        down_bias=ck.floats(q + "down.b", width))
     for n, a in mats.items():
         assert a.shape == shapes[n], (n, a.shape, shapes[n])
     return mats, vecs
 
 
-def create(engine, cfg: StackConfig, packed_layers, embed, final_norm, loop_step, exact: bool):
-    """alice_stack_create over packed layers: [(matrices, vectors)]; a matrix is a uint16 array or a ready weight handle.
+def create(engine, cfg: StackConfig, packed_layers, embed, final_norm, loop_step, exact: bool, head=None):
+    """alice_stack_create over packed layers: [(matrices, vectors)]; a matrix is a uint16 array or a ready weight handle
+    (head None: the embedding table).
     -> (handle, objects that must outlive it)."""
     from .gpu import GpuQuantType, GpuWeightBuffer
     keep = []
@@ -244,14 +297,15 @@ def create(engine, cfg: StackConfig, packed_layers, embed, final_norm, loop_step
     for spec, dst, (mats, vecs) in zip(cfg.layers, arr, packed_layers):
         dst.mixer = spec.kind
         for n in ("heads", "kv_heads", "dim", "vdim", "q_rank", "kv_rank", "rot_dim", "rot_dims", "conv_taps", "decay_rank", "gate_rank", "ff",
-                  "scale", "rot_base"):
+                  "unit_qk", "scale", "softcap", "rot_base", "rot_factor", "rot_low", "rot_high", "rot_original"):
             setattr(dst, n, getattr(spec, n))
         for n, a in mats.items():
             setattr(dst, n if n != "in" else "in_", up(a))
         for n, a in vecs.items():
             setattr(dst, n, vec(a))
     c = _lib.StackConfig(len(cfg.layers), cfg.width, cfg.vocab_size, cfg.max_seq_len, cfg.loop_start, cfg.loop_stop, cfg.loop_times, int(exact),
-                         cfg.eps, cfg.embed_scale, vec(loop_step) if cfg.loop_times else None)
+                         cfg.family.block, cfg.family.norm, cfg.eps, cfg.embed_scale, cfg.alpha, vec(loop_step) if cfg.loop_times else None,
+                         None if head is None else up(head))
     h = C.c_void_p()
     _lib.check(engine._lib.alice_stack_create(engine._h, C.byref(c), arr, up(embed), C.c_void_p(vec(final_norm)), C.byref(h)))
     return h, keep
@@ -262,10 +316,12 @@ def load_tensors(engine, config: dict, tensors: dict, dtype: str = "bfloat16", m
     if dtype not in ("bfloat16", "float32"):
         raise ConfigError(f"dtype {dtype!r} (bfloat16 or float32)")
     cfg, ck = StackConfig(config, max_seq_len), Checkpoint(tensors)
-    packed = [pack_layer(ck, i, L, cfg.width) for i, L in enumerate(cfg.layers)]
+    packed = [pack_layer(ck, i, L, cfg) for i, L in enumerate(cfg.layers)]
     embed = _cols(ck.matrix("embed", cfg.vocab_size, cfg.width), pad(cfg.width))
     step = ck.floats("loop.step", cfg.loop_times, cfg.width) if cfg.loop_times else None
-    h, keep = create(engine, cfg, packed, embed, ck.floats("final.norm", cfg.width), step, dtype == "float32")
+    head = None if cfg.family.tied else _cols(ck.matrix("head", cfg.vocab_size, cfg.width), pad(cfg.width))
+    final = ck.floats("final.norm", cfg.width) + np.float32(cfg.family.norm_offset)
+    h, keep = create(engine, cfg, packed, embed, final, step, dtype == "float32", head)
     return h, cfg, keep
 
 

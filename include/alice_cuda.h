@@ -267,9 +267,11 @@ int32_t alice_model_set_position(alice_model* m, uint32_t pos);
 
 /* ---- layer-stack models ------------------------------------------------------------------------ */
 /* A decoder whose layers are listed one by one, each with its own token mixer, as another kind of alice_model: the same
- * step, greedy-decode, logits and reset calls drive it. No counterpart in the reference. Each layer adds
- *   ls1 * mixer(h) + ls2 * mlp(h),   h = layer_norm(x) (weight, no bias),
- * to a 32-bit residual stream; the head is the embedding table behind a last layer norm. Layers loop_start .. loop_stop - 1
+ * step, greedy-decode, logits and reset calls drive it. No counterpart in the reference. The residual stream x is in 32 bits.
+ *   ALICE_BLOCK_PARALLEL  x <- x + ls1 * mixer(h) + ls2 * mlp(h),   h = norm(x)
+ *   ALICE_BLOCK_POST      x <- norm(alpha * x + mixer(x)), then x <- norm2(alpha * x + mlp(x))
+ * Norms are layer norms (weight, no bias) or root-mean-square norms, one kind per model; the head (the embedding table if it
+ * has no matrix of its own) stands behind a last one. Layers loop_start .. loop_stop - 1
  * run loop_times times in a row with the same weights and a state or cache per pass; ahead of pass t the embedding output
  * (t > 0) and loop_step[t] join the stream. loop_times == 0: no loop.
  *
@@ -279,38 +281,55 @@ int32_t alice_model_set_position(alice_model* m, uint32_t pos);
  *                     sigmoid output gate.
  *   ALICE_MIX_DELTA   gated delta rule with one decay per key channel, short causal convolutions on q, k, v, root-mean-square
  *                     norm and sigmoid gate on the output; recurrent state in 32 bits.
+ *   ALICE_MIX_GROUPED attention with kv_heads key / value heads, each serving heads / kv_heads consecutive query heads; half-split
+ *                     rotation of the first rot_dims of q and k, with unit_qk then both over their root mean square; scores
+ *                     times scale, capped as softcap * tanh(s / softcap); a sink per head.
  *
  * Matrices are ALICE_TYPE_BF16 handles whose columns are zero-padded to a multiple of 64 (P() below), and whose row segments
  * start at multiples of 64 rows (zero rows between):
  *   in    latent: [P(q_rank) query latent | P(kv_rank + rot_dim) key latent, key part | P(heads * vdim) gate]
  *         delta:  [P(kv_heads * dim) q | same k | P(heads * vdim) v | P(heads) step | P(decay_rank) | P(gate_rank)]
+ *         grouped: [P(heads * dim) q | P(kv_heads * dim) k | P(kv_heads * vdim) v]
  *   uq    [heads * (dim + rot_dim)][P(q_rank)]       uk [heads * dim][P(kv_rank)]      uv [heads * vdim][P(kv_rank)]
  *   a2    [heads * D][P(decay_rank)] with dim padded to D = 64, 128 or 256 per head; dt_bias likewise [heads * D]
  *   g2    [heads * vdim][P(gate_rank)]               o  [width][P(heads * vdim)]
  *   gu    64 gate rows, 64 up rows, 64 gate rows, ... of P(ff) each [2 P(ff)][P(width)]; down [width][P(ff)]
- *   embed [vocab][P(width)]
+ *   embed, head [vocab][P(width)]
  * and gate_bias / up_bias hold P(ff) floats. conv [conv_taps][columns of q | k | v in `in`]. Float arrays are copied. */
 #define ALICE_MIX_LATENT 1u
 #define ALICE_MIX_DELTA 2u
+#define ALICE_MIX_GROUPED 3u
+#define ALICE_BLOCK_PARALLEL 0u
+#define ALICE_BLOCK_POST 1u
+#define ALICE_NORM_LAYER 0u
+#define ALICE_NORM_RMS 1u
 typedef struct {
     uint32_t mixer;
     uint32_t heads, kv_heads, dim, vdim;
     uint32_t q_rank, kv_rank, rot_dim, rot_dims;     /* latent */
     uint32_t conv_taps, decay_rank, gate_rank;       /* delta */
     uint32_t ff;                                     /* 0: no feed-forward */
-    float scale;                                     /* latent: factor on the scores */
-    double rot_base;
+    uint32_t unit_qk;                                /* grouped */
+    float scale;                                     /* latent, grouped: factor on the scores */
+    float softcap;                                   /* grouped: 0 = none */
+    /* latent, grouped: frequencies rot_base^(-2i / rot_dims); rot_factor 0: as they are, else wavelengths above rot_original /
+     * rot_low are rot_factor times longer, those below rot_original / rot_high stay, linear in 1 / wavelength between */
+    double rot_base, rot_factor, rot_low, rot_high, rot_original;
     const alice_weights *in, *uq, *uk, *uv, *a2, *g2, *o, *gu, *down;
-    const float *norm, *ls1, *ls2, *gate_bias, *up_bias, *down_bias;
-    const float *q_norm, *kv_norm, *sink;            /* latent */
+    const float *norm, *norm2, *ls1, *ls2;           /* parallel: norm, ls1, ls2; post: norm, norm2 */
+    const float *gate_bias, *up_bias, *down_bias;    /* post: may be null */
+    const float *q_norm, *kv_norm;                   /* latent */
+    const float *sink;                               /* latent, grouped (null: none) */
     const float *conv, *a_log, *dt_bias, *head_norm; /* delta */
 } alice_stack_layer;
 typedef struct {
     uint32_t num_layers, width, vocab_size, max_seq_len;
     uint32_t loop_start, loop_stop, loop_times;
     uint32_t exact;                                  /* 1: every activation, product and cache in 32 bits */
-    float eps, embed_scale;
+    uint32_t block, norm;
+    float eps, embed_scale, alpha;                   /* alpha: post */
     const float* loop_step;                          /* [loop_times][width] */
+    const alice_weights* head;                       /* null: the embedding table */
 } alice_stack_config;
 int32_t alice_stack_create(alice_engine* e, const alice_stack_config* cfg, const alice_stack_layer* layers, const alice_weights* embed,
                            const float* final_norm, alice_model** out);

@@ -302,7 +302,7 @@ def test_position_limits_and_rollback(eng):
 def test_weight_handles_of_the_wrong_shape_are_refused(eng):
     cfg = stack.StackConfig(zm.ODD, 16)
     w = zm.weights(zm.ODD)
-    packed = [stack.pack_layer(stack.Checkpoint(w), i, L, cfg.width) for i, L in enumerate(cfg.layers)]
+    packed = [stack.pack_layer(stack.Checkpoint(w), i, L, cfg) for i, L in enumerate(cfg.layers)]
     packed[1][0]["uk"] = packed[1][0]["uk"][:-1]
     embed = np.zeros((cfg.vocab_size, 64), np.uint16)
     with pytest.raises(AliceError, match="uk"):

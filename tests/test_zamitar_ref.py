@@ -199,7 +199,7 @@ def test_tensor_shapes_are_checked():
             del t[name]
         with pytest.raises(stack.ConfigError, match=name.replace(".", r"\.")):
             for i, L in enumerate(cfg.layers):
-                stack.pack_layer(stack.Checkpoint(t), i, L, cfg.width)
+                stack.pack_layer(stack.Checkpoint(t), i, L, cfg)
 
 
 @pytest.mark.parametrize("name", zm.MODELS)
@@ -208,7 +208,7 @@ def test_packed_layers_hold_every_weight(name):
     d = zm.MODELS[name]
     cfg, w = stack.StackConfig(d, 8), zm.weights(d)
     for i, L in enumerate(cfg.layers):
-        mats, vecs = stack.pack_layer(stack.Checkpoint(w), i, L, cfg.width)
+        mats, vecs = stack.pack_layer(stack.Checkpoint(w), i, L, cfg)
         at, seen = 0, 0
         for n, rows in L.input_segments():
             seg = mats["in"][at:at + rows, :cfg.width]
