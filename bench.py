@@ -820,15 +820,24 @@ def run_ours(args, rank, world, local_rank):
 
 
 # ---- layer-stack models (--stack) -------------------------------------------------------------------------
-# width, feed-forward, heads and layer count of each size; half of the layers are latent attention, half delta rule. The
-# compared Llama has the same width, feed-forward, heads, layer count and vocabulary, in the Q4_K_M mix.
+# width, feed-forward, heads and layer count of each size. w*: Zamitar, half of the layers latent attention, half delta rule,
+# beside a Llama of the same width, feed-forward, heads, layer count and vocabulary in the Q4_K_M mix. s*: Suborax, all layers
+# grouped attention, beside the Zamitar of the same sizes.
 STACK_SIZES = {
     "w2048": dict(width=2048, ff=8192, heads=16, q_rank=768, kv_rank=512, rank=128, layers=8, vocab=32000),
     "w4096": dict(width=4096, ff=14336, heads=32, q_rank=1536, kv_rank=512, rank=128, layers=8, vocab=32000),
+    "s2048": dict(width=2048, ff=8192, heads=16, kv_heads=4, layers=8, vocab=32000, beside="w2048"),
+    "s4096": dict(width=4096, ff=14336, heads=32, kv_heads=8, layers=8, vocab=32000, beside="w4096"),
 }
 
 
 def stack_config(z):
+    if "kv_heads" in z:
+        grouped = {"type": "attention", "mlp": {"kind": "dense", "ff": z["ff"]},
+                   "mixer": dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0,
+                                 rot=dict(base=10000.0, dims=128, scaling=dict(factor=4.0, low=1.0, high=4.0, original=4096)))}
+        return {"architecture": "Suborax", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+                "postln_alpha": 2.0, "layers": [grouped] * z["layers"]}
     latent = {"type": "latent_attention", "mlp": {"kind": "dense", "ff": z["ff"]},
               "mixer": dict(heads=z["heads"], dim=128, rot_dim=64, vdim=128, q_rank=z["q_rank"], kv_rank=z["kv_rank"], scale=192 ** -0.5,
                             rot=dict(base=10000.0, dims=64))}
@@ -839,7 +848,7 @@ def stack_config(z):
 
 
 def build_stack(eng, z, max_seq_len, seed=0):
-    """-> (GpuModel, weight bytes one token reads, matrix FLOPs per token). Weights drawn on the device."""
+    """-> (GpuModel, weight bytes one token reads, matrix FLOPs of a prompt token, the head aside). Weights drawn on the device."""
     import torch
     from alice_llm_b200 import stack
     from alice_llm_b200.gpu import GpuModel, GpuQuantType
@@ -864,6 +873,9 @@ def build_stack(eng, z, max_seq_len, seed=0):
         L.decay_rank = L.gate_rank = z["rank"] if L.kind == stack.MIX_DELTA else 0
         mats = {n: mat(*shape) for n, shape in L.packed_shapes(cfg.width).items()}
         w, ff = cfg.width, stack.pad(L.ff)
+        if L.kind == stack.MIX_GROUPED:
+            packed.append((mats, dict(norm=one(w), norm2=one(w), sink=small(L.heads))))
+            continue
         vecs = dict(norm=one(w), ls1=small(w), ls2=small(w), gate_bias=small(ff), up_bias=small(ff), down_bias=small(w))
         if L.kind == stack.MIX_LATENT:
             vecs.update(q_norm=one(L.q_rank), kv_norm=one(L.kv_rank), sink=small(L.heads))
@@ -872,8 +884,13 @@ def build_stack(eng, z, max_seq_len, seed=0):
                         dt_bias=small(L.heads * stack.delta_dim(L.dim)) - 2.0, head_norm=one(L.vdim))
         packed.append((mats, vecs))
     embed = mat(cfg.vocab_size, stack.pad(cfg.width))
-    h, more = stack.create(eng, cfg, packed, embed, one(cfg.width), None, False)
-    return GpuModel(eng, h, cfg, [keep, more]), nbytes, nbytes      # two FLOPs per weight = its two bytes
+    keep.append(embed)
+    head = None
+    if not cfg.family.tied:
+        nbytes -= cfg.vocab_size * stack.pad(cfg.width) * 2   # of the embedding table a token reads one row
+        head = mat(cfg.vocab_size, stack.pad(cfg.width))
+    h, more = stack.create(eng, cfg, packed, embed, one(cfg.width), None, False, head)
+    return GpuModel(eng, h, cfg, [keep, more]), nbytes, nbytes - cfg.vocab_size * stack.pad(cfg.width) * 2      # two FLOPs per weight = its two bytes
 
 
 def llama_like(z, context):
@@ -884,7 +901,7 @@ def llama_like(z, context):
 
 
 def run_stack(args):
-    """Prefill and greedy decode of layer-stack models beside a quantized Llama of the same size, on one GPU."""
+    """Prefill and greedy decode of layer-stack models beside another model of the same size, on one GPU."""
     import torch
     from alice_llm_b200.gpu import GpuEngine
     torch.cuda.set_device(0)
@@ -914,7 +931,8 @@ def run_stack(args):
     clocks = ClockSampler(0)
     clocks.start()
     out = {}
-    for name in args.stack.split(","):
+
+    def one(name):
         z = STACK_SIZES[name]
         rng = np.random.default_rng(1)
         prompt = rng.integers(0, z["vocab"], ctx).astype(np.uint32)
@@ -928,15 +946,29 @@ def run_stack(args):
         pf = timed(prefill, 5)
         gm.decode_greedy(1, 8)
         dec = timed(lambda: gm.decode_greedy(1, tokens)) / tokens
-        half = z["layers"] // 2
-        extra = half * (2 * z["heads"] * 128 * 128 * 4) + half * ctx * (z["kv_rank"] + 64) * 2   # states read and written, latent rows read
-        # attention: scores and sums over half of the context on average, keys and values made from the latent once
-        aflops = half * (2 * z["heads"] * (192 + 128) * ctx / 2)
-        out[name] = {"prefill_tokens_per_s": round(ctx / pf * 1e3), "prefill_ms": round(pf, 3),
-                     "prefill_tflops": round((flops + aflops) * ctx / pf / 1e9, 1), "prefill_of_bf16_peak": round((flops + aflops) * ctx / pf / 1e9 / tflops, 3),
-                     "decode_ms_per_token": round(dec, 4), "decode_gbs": round((nbytes + extra) / dec / 1e6), "decode_of_hbm_peak": round((nbytes + extra) / dec / 1e6 / peak, 3)}
+        # attention: scores and sums over half of the context on average
+        if "kv_heads" in z:
+            extra = z["layers"] * ctx * z["kv_heads"] * 256 * 2   # keys and values read
+            aflops = z["layers"] * (2 * z["heads"] * 256 * ctx / 2)
+        else:
+            half = z["layers"] // 2
+            extra = half * (2 * z["heads"] * 128 * 128 * 4) + half * ctx * (z["kv_rank"] + 64) * 2   # states read and written, latent rows read
+            aflops = half * (2 * z["heads"] * (192 + 128) * ctx / 2)   # keys and values made from the latent once are not counted
         gm.free()
-        if not args.stack_only:
+        torch.cuda.empty_cache()
+        return {"prefill_tokens_per_s": round(ctx / pf * 1e3), "prefill_ms": round(pf, 3),
+                "prefill_tflops": round((flops + aflops) * ctx / pf / 1e9, 1), "prefill_of_bf16_peak": round((flops + aflops) * ctx / pf / 1e9 / tflops, 3),
+                "decode_ms_per_token": round(dec, 4), "decode_gbs": round((nbytes + extra) / dec / 1e6),
+                "decode_of_hbm_peak": round((nbytes + extra) / dec / 1e6 / peak, 3)}
+
+    for name in args.stack.split(","):
+        z = STACK_SIZES[name]
+        out[name] = one(name)
+        rng = np.random.default_rng(1)
+        prompt = rng.integers(0, z["vocab"], ctx).astype(np.uint32)
+        if not args.stack_only and "beside" in z:
+            out[name]["zamitar_equal_size"] = dict(out[z["beside"]]) if z["beside"] in out else one(z["beside"])
+        elif not args.stack_only:
             DECODE_CONFIGS["llama_" + name] = llama_like(z, ctx)
             lm, info = build_model(eng, "llama_" + name)
 
@@ -982,10 +1014,10 @@ def main():
     ap.add_argument("--decode-tokens", type=int, default=128)
     ap.add_argument("--decode-seconds", type=float, default=300.0, help="time limit of the whole-model section")
     ap.add_argument("--stack", nargs="?", const=",".join(STACK_SIZES), default="",
-                    help="instead of the default workload: prefill and decode of layer-stack models beside a Llama of equal size (comma list of " +
+                    help="instead of the default workload: prefill and decode of layer-stack models beside another model of equal size (comma list of " +
                          ", ".join(STACK_SIZES) + ")")
     ap.add_argument("--stack-context", type=int, default=2048, help="prompt length of --stack")
-    ap.add_argument("--stack-only", action="store_true", help="--stack without the compared Llama")
+    ap.add_argument("--stack-only", action="store_true", help="--stack without the compared model")
     args = ap.parse_args()
     if args.stack:
         return run_stack(args)

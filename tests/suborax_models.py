@@ -20,7 +20,7 @@ def config(layers, width=80, vocab=131, eps=1e-5, scale=0.8, alpha=1.7):
             "layers": layers}
 
 
-def weights(cfg, seed=0, sink=1.5):
+def weights(cfg, seed=0, sink=2.5):
     """{name: uint16 bfloat16 bits}."""
     rng = np.random.default_rng(seed)
     w = {}
@@ -60,11 +60,11 @@ def row_errors(got, want):
 
 
 # Sizes chosen to differ from one another and to be no multiples of what the kernels tile by. "odd" has head sizes that are odd,
-# one key head per query head, a layer without a feed-forward first; "wide" groups above sixteen heads and larger sizes.
+# one key head per query head, a layer without a feed-forward first, a large eps; "wide" groups above sixteen heads and larger sizes.
 MIXED = config([attention(), attention(heads=6, kv_heads=1, dim=40, vdim=16, rot=40, softcap=3.0, ff=0), attention(heads=3, kv_heads=3, dim=8, vdim=56, rot=4, ff=48),
                 attention(heads=10, kv_heads=5, dim=16, vdim=24, rot=10, base=50.0, scaled=None, ff=130)])
-ODD = config([attention(heads=2, kv_heads=2, dim=7, vdim=5, rot=6, ff=0, softcap=20.0), attention(heads=5, kv_heads=1, dim=33, vdim=65, rot=2, scale=0.3, ff=33),
-              attention(heads=1, kv_heads=1, dim=10, vdim=3, rot=10, softcap=1.0, ff=1, scaled=scaling(2.0, 1.0, 8.0, 100))], width=50, vocab=77, eps=1e-3, scale=0.35, alpha=0.9)
+ODD = config([attention(heads=6, kv_heads=6, dim=7, vdim=9, rot=6, ff=0, softcap=20.0), attention(heads=5, kv_heads=1, dim=33, vdim=65, rot=2, scale=0.3, ff=33),
+              attention(heads=4, kv_heads=2, dim=10, vdim=21, rot=10, softcap=1.0, ff=65, scaled=scaling(2.0, 1.0, 8.0, 100))], width=50, vocab=77, eps=0.3, scale=0.35, alpha=0.9)
 WIDE = config([attention(heads=20, kv_heads=1, dim=64, vdim=72, rot=32, scale=0.2, ff=300), attention(heads=8, kv_heads=2, dim=128, vdim=128, rot=128, scale=0.15, softcap=12.0, ff=260),
                attention(heads=4, kv_heads=2, dim=200, vdim=130, rot=64, scale=0.12, ff=100)], width=272, vocab=515, scale=1.4, alpha=3.1)
 MODELS = {"mixed": MIXED, "odd": ODD, "wide": WIDE}
