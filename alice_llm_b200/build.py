@@ -16,7 +16,7 @@ LIB = os.path.join(HERE, "libalice_cuda.so")
 # What a layer-stack model needs, as a library of its own; the whole library is these and the quantized-matvec path.
 LIB_STACK = os.path.join(HERE, "libalice_stack.so")
 STACK_SOURCES = ["engine.cu", "tp.cu", "step.cu", "model_api.cu", "stack_model.cu", "stack_ops.cu", "dense_rows.cu", "dense_gemm.cu", "delta.cu",
-                 "latent.cu", "latent_decode.cu", "latent_prefill.cu", "grouped.cu", "grouped_decode.cu"]
+                 "latent.cu", "latent_decode.cu", "latent_prefill.cu", "grouped.cu", "grouped_decode.cu", "grouped_prefill.cu"]
 SOURCES = STACK_SOURCES + ["abi.cu", "gemv_launch.cu", "q8k.cu", "dequant.cu", "ternarize.cu", "glue.cu", "model.cu"]
 # never --use_fast_math: dequantization and the Q8_K quantizer must round like the reference
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",

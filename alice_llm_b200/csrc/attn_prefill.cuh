@@ -1,7 +1,7 @@
 // Causal attention of many tokens over rows of keys and values in global memory, on the tensor cores: bf16 queries, keys and
 // values, f32 scores, softmax and sums. The softmax weights enter the weighted sum as a bf16 pair (value and remainder), so
 // they are not cut to eight bits. The sink of a head is the state the online softmax starts from: a key that scores `sink`
-// and has no value (-inf: no sink). Shared by the mixers that attend (latent_prefill.cu, grouped.cu).
+// and has no value (-inf: no sink). Shared by the mixers that attend (latent_prefill.cu, grouped_prefill.cu).
 #pragma once
 #include "dense_dev.cuh"
 #include "mixers.cuh"
@@ -13,7 +13,8 @@ namespace alice {
 // which all heads share. Column counts are multiples of 8, rows 16-byte aligned.
 struct PrefillArgs {
     uint32_t heads = 0, group = 1, vdim = 0, v_cols = 0;      // v_cols: vdim as the rows hold it
-    const bf16* q = nullptr;                                  // [t][heads][k1_cols + k2_cols]
+    const bf16* q = nullptr;                                  // rows of k1_cols + k2_cols, those of a group one behind the other
+    size_t q_row = 0, q_group = 0;                            // elements between tokens and between groups
     const bf16 *k1 = nullptr, *k2 = nullptr, *v = nullptr;
     uint32_t k1_cols = 0, k2_cols = 0;
     size_t k1_row = 0, k1_head = 0, k2_row = 0, v_row = 0, v_head = 0;   // elements between rows and between heads
@@ -76,7 +77,7 @@ __global__ void __launch_bounds__(PF_THREADS, 2) attn_prefill_kernel(const __gri
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     for (uint32_t r = fr; r < PF_ROWS; r += PF_KEYS) {   // queries, part of the first copy group
-        const bf16* q = a.q + ((size_t)(t0 + min(r, rows - 1)) * a.heads + h) * qd;
+        const bf16* q = a.q + (t0 + min(r, rows - 1)) * a.q_row + (h / a.group) * a.q_group + (h % a.group) * qd;
         for (uint32_t c = fc; c < DQ / 8; c += TPR) cp16(q_sm + r * G::LQ * 2 + c * 16, q + min(c * 8, qd - 8), r < rows && c * 8 < qd);
     }
     fetch(0, 0);

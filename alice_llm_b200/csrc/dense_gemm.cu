@@ -80,26 +80,6 @@ cudaError_t launch_f32(const GemmOp& op, cudaStream_t st, bool pdl) {
     }
 }
 
-using EncodeFn = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
-                              const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-EncodeFn encode_fn() {
-    static EncodeFn fn = [] {
-        void* p = nullptr;
-        cudaDriverEntryPointQueryResult q;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q) != cudaSuccess || q != cudaDriverEntryPointSuccess) p = nullptr;
-        return reinterpret_cast<EncodeFn>(p);
-    }();
-    return fn;
-}
-
-// rows x cols bf16, ld elements between rows, copied as tiles of box_rows x 64 (rows past the end read as zero)
-bool tile_map(CUtensorMap* map, const void* base, uint32_t rows, uint32_t cols, uint32_t ld, uint32_t box_rows) {
-    const cuuint64_t dims[2] = {cols, rows}, strides[1] = {(cuuint64_t)ld * 2};
-    const cuuint32_t box[2] = {TC_BK, box_rows}, step[2] = {1, 1};
-    return encode_fn()(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, step, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                       CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
-}
-
 template <int BN, int EPI>
 cudaError_t tc_inst(const TcArgs& a, uint32_t grid, cudaStream_t st, bool pdl) {
     static bool done[64] = {};

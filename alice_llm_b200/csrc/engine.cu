@@ -181,10 +181,10 @@ int32_t alice_sync(alice_engine* e) {
     if (st != 0) {
         cudaMemset(e->status, 0, sizeof(int));
         static const char* const what[] = {"?", "unspecified wait", "weights did not land in shared memory", "partial sums of a row", "stage release",
-                                           "grid barrier", "rows from a tensor-parallel peer", "operands or accumulators of a tensor-core product", "a tile of cached keys and values"};
+                                           "grid barrier", "rows from a tensor-parallel peer", "operands or accumulators of a tensor-core product", "a tile of cached keys and values", "operands or weights of tensor-core attention"};
         const int code = st & 0xff;
         return fail(ALICE_E_KERNEL, "alice_sync: a kernel wait ran out of its cycle budget (status %d: %s); results of the queued work are void",
-                    st, code >= 1 && code <= 8 ? what[code] : what[0]);
+                    st, code >= 1 && code <= 9 ? what[code] : what[0]);
     }
     return ALICE_OK;
 }

@@ -1,6 +1,5 @@
 // Attention whose key / value heads serve groups of query heads (a plain key / value cache): rotation and norm of queries and
-// keys into place, the f32 form for any number of tokens, and the tensor-core form for many.
-#include "attn_prefill.cuh"
+// keys into place, and the f32 form for any number of tokens.
 #include "grouped_dev.cuh"
 
 namespace alice {
@@ -11,7 +10,7 @@ template <class CT>
 __global__ void __launch_bounds__(256) grouped_prepare_kernel(const __grid_constant__ GroupedArgs a) {
     __shared__ float2 cs[GROUPED_PAIRS];
     const GroupedShape& s = a.s;
-    const uint32_t t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const uint32_t t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, group = s.heads / s.kv_heads;
     pdl_launch_dependents();
     pdl_wait();
     const uint32_t p = (uint32_t)*a.pos + t;
@@ -20,7 +19,7 @@ __global__ void __launch_bounds__(256) grouped_prepare_kernel(const __grid_const
     const float* y = a.y + (size_t)t * a.ldy;
     for (uint32_t i = warp; i < s.heads + 2 * s.kv_heads; i += 8) {
         if (i < s.heads) {
-            rotate_norm(y + (size_t)i * s.dim, static_cast<CT*>(a.q) + ((size_t)t * s.heads + i) * s.dp, s, cs, a.eps, lane);
+            rotate_norm(y + (size_t)i * s.dim, static_cast<CT*>(a.q) + ((size_t)(i / group * gridDim.x + t) * group + i % group) * s.dp, s, cs, a.eps, lane);
             continue;
         }
         const bool key = i < s.heads + s.kv_heads;
@@ -47,7 +46,7 @@ __global__ void __launch_bounds__(256) grouped_attn_kernel(const __grid_constant
     const uint32_t p0 = (uint32_t)*a.pos, last = min(r0 + GA_ROWS, rows) - 1, keys = p0 + last / group + 1;
     for (uint32_t i = threadIdx.x; i < GA_ROWS * s.dp; i += 256) {
         const uint32_t r = r0 + i / s.dp;
-        qs[i] = r < rows ? get(static_cast<const CT*>(a.q) + ((size_t)(r / group) * s.heads + kh * group + r % group) * s.dp + i % s.dp) * s.scale : 0.0f;
+        qs[i] = r < rows ? get(static_cast<const CT*>(a.q) + ((size_t)kh * rows + r) * s.dp + i % s.dp) * s.scale : 0.0f;
     }
     float m[GA_RW], l[GA_RW], o[GA_RW][NC];
     uint32_t see[GA_RW];                             // keys the row sees
@@ -153,17 +152,6 @@ cudaError_t launch_grouped_prepare(const GroupedArgs& a, uint32_t tokens, cudaSt
 cudaError_t launch_grouped_attn(const GroupedArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
     if (a.cache_bf16) return a.act_bf16 ? attn_type<bf16, bf16>(a, tokens, st, pdl) : attn_type<bf16, float>(a, tokens, st, pdl);
     return a.act_bf16 ? cudaErrorInvalidValue : attn_type<float, float>(a, tokens, st, pdl);
-}
-cudaError_t launch_grouped_prefill(const GroupedArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
-    if (!grouped_tiled_fits(a.s) || !a.cache_bf16 || !a.act_bf16) return cudaErrorInvalidValue;
-    const GroupedShape& z = a.s;
-    const auto* cache = static_cast<const bf16*>(a.cache);
-    PrefillArgs p;
-    p.heads = z.heads; p.group = z.group(); p.vdim = z.vdim; p.v_cols = z.vp; p.pos = a.pos; p.sink = a.sink; p.scale = z.scale; p.softcap = z.softcap;
-    p.q = static_cast<const bf16*>(a.q); p.k1 = cache; p.k1_cols = z.dp; p.v = cache + z.dp;
-    p.k1_row = p.v_row = z.ld(); p.k1_head = p.v_head = (size_t)a.plane_rows * z.ld();
-    p.out = static_cast<bf16*>(a.out); p.ldo = a.ldo;
-    return launch_attn_prefill<true>(p, tokens, st, pdl);
 }
 
 }  // namespace alice

@@ -45,7 +45,7 @@ cudaError_t launch_latent_prefill(const LatentArgs& a, uint32_t tokens, cudaStre
     if (err != cudaSuccess) return err;
     const LatentShape& z = a.s;
     PrefillArgs p;
-    p.heads = z.heads; p.vdim = p.v_cols = z.vdim; p.q = a.q_rot; p.pos = a.pos; p.sink = a.sink; p.scale = z.scale;
+    p.heads = z.heads; p.vdim = p.v_cols = z.vdim; p.q = a.q_rot; p.q_group = z.dim + z.rot; p.q_row = z.heads * p.q_group; p.pos = a.pos; p.sink = a.sink; p.scale = z.scale;
     p.k1 = a.k_all; p.k1_cols = z.dim; p.k1_row = (size_t)z.heads * z.dim; p.k1_head = z.dim;
     p.k2 = static_cast<const bf16*>(a.cache) + z.cp; p.k2_cols = z.rot; p.k2_row = z.cp + z.rp;
     p.v = a.v_all; p.v_row = (size_t)z.heads * z.vdim; p.v_head = z.vdim;

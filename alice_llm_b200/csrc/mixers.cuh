@@ -1,6 +1,8 @@
 // Token mixers of layer-stack models (csrc/delta.cu, csrc/latent.cu, csrc/grouped.cu) and the small per-token kernels around them
 // (csrc/stack_ops.cu). Sizes are run-time values; positions come from device memory so that a captured step can be replayed.
 #pragma once
+#include <cmath>
+
 #include "dense.cuh"
 
 namespace alice {
@@ -145,7 +147,7 @@ struct GroupedArgs {
     void* cache = nullptr;            // [kv_heads][plane_rows][ld]
     uint32_t plane_rows = 0;
     bool cache_bf16 = false;
-    void* q = nullptr;                // prepared queries [t][heads][dp], of the cache's type
+    void* q = nullptr;                // prepared queries [kv_heads][t][group][dp], of the cache's type
     void* out = nullptr;              // [t][ldo]
     uint32_t ldo = 0;
     bool act_bf16 = false;            // type of out
@@ -162,6 +164,11 @@ cudaError_t launch_grouped_prepare(const GroupedArgs& a, uint32_t tokens, cudaSt
 cudaError_t launch_grouped_attn(const GroupedArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 // On the tensor cores, bf16 cache: many tokens (prepared queries), few tokens (queries straight from the projections).
 inline bool grouped_tiled_fits(const GroupedShape& s) { return s.dp <= 256 && s.vp <= 256; }
+// What no score exceeds: unit queries and keys meet in at most dim, and a cap is one.
+inline float grouped_bound(const GroupedShape& s) {
+    const float unit = s.unit_qk ? 1.01f * std::fabs(s.scale) * s.dim : INFINITY;   // a little more for their rounding
+    return s.softcap > 0.0f ? std::fmin(s.softcap, unit) : unit;
+}
 cudaError_t launch_grouped_prefill(const GroupedArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 cudaError_t launch_grouped_decode(const GroupedArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 
