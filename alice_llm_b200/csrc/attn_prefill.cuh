@@ -27,9 +27,6 @@ struct PrefillArgs {
     uint32_t ldo = 0;
 };
 
-// tanh(x / (2 log2(e))), from the exponential: exact to an ulp or two of 1
-__device__ __forceinline__ float tanh_of_pow2(float x) { return 1.0f - __fdividef(2.0f, 1.0f + exp2f(x)); }
-
 constexpr int PF_KEYS = 32, PF_ROWS = 128, PF_THREADS = 128;   // keys per tile; queries per CTA, 32 per warp: each key fragment serves two row tiles
 
 // DQ, DV: query / key and value dimensions the tiles have room for (multiples of 16, zero beyond the true sizes). Values wider

@@ -7,6 +7,8 @@ namespace alice {
 
 __device__ __forceinline__ float sigmoid_f(float z) { return __fdiv_rn(1.0f, 1.0f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
+// tanh(x / (2 log2(e))), from the exponential: exact to an ulp or two of 1
+__device__ __forceinline__ float tanh_of_pow2(float x) { return 1.0f - __fdividef(2.0f, 1.0f + exp2f(x)); }
 __device__ __forceinline__ float2 bf2(uint32_t u) { return make_float2(__uint_as_float(u << 16), __uint_as_float(u & 0xffff0000u)); }
 __device__ __forceinline__ float dot8(uint4 v, float4 x0, float4 x1, float acc) {
     const float2 a = bf2(v.x), b = bf2(v.y), d = bf2(v.z), e = bf2(v.w);

@@ -5,29 +5,48 @@
 namespace alice {
 namespace {
 
-// One CTA per token; a warp per row of a head: queries, then keys, then values.
-template <class CT>
+// One CTA per token; a warp per row of a head: queries, then keys, then values. The next row is loaded while one is finished.
+template <class CT, int E>
 __global__ void __launch_bounds__(256) grouped_prepare_kernel(const __grid_constant__ GroupedArgs a) {
     __shared__ float2 cs[GROUPED_PAIRS];
     const GroupedShape& s = a.s;
-    const uint32_t t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, group = s.heads / s.kv_heads;
+    const uint32_t t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, group = s.heads / s.kv_heads, rows = s.heads + 2 * s.kv_heads;
     pdl_launch_dependents();
     pdl_wait();
+    const float* y = a.y + (size_t)t * a.ldy;
+    HeadRow<E> row[2];
+    auto load = [&](uint32_t i, HeadRow<E>& r) {
+        if (i < s.heads) r.load(y + (size_t)i * s.dim, s.dim, s.rot_dims, lane);
+        else if (i < s.heads + s.kv_heads) r.load(y + s.off_k + (size_t)(i - s.heads) * s.dim, s.dim, s.rot_dims, lane);
+        else if (i < rows) r.load(y + s.off_v + (size_t)(i - s.heads - s.kv_heads) * s.vdim, s.vdim, 0, lane);
+    };
+    load(warp, row[0]);
     const uint32_t p = (uint32_t)*a.pos + t;
     rotation_table(cs, a.freq, s.rot_dims / 2, p, 256);
     __syncthreads();
-    const float* y = a.y + (size_t)t * a.ldy;
-    for (uint32_t i = warp; i < s.heads + 2 * s.kv_heads; i += 8) {
+    auto store = [&](uint32_t i, HeadRow<E>& r) {
         if (i < s.heads) {
-            rotate_norm(y + (size_t)i * s.dim, static_cast<CT*>(a.q) + ((size_t)(i / group * gridDim.x + t) * group + i % group) * s.dp, s, cs, a.eps, lane);
-            continue;
+            r.store(static_cast<CT*>(a.q) + ((size_t)(i / group * gridDim.x + t) * group + i % group) * s.dp, s.dp, s.unit_qk, cs, a.eps, lane);
+        } else {
+            const bool key = i < s.heads + s.kv_heads;
+            CT* out = static_cast<CT*>(a.cache) + ((size_t)(i - s.heads - (key ? 0 : s.kv_heads)) * a.plane_rows + p) * s.ld();
+            r.store(key ? out : out + s.dp, key ? s.dp : s.vp, key && s.unit_qk, cs, a.eps, lane);
         }
-        const bool key = i < s.heads + s.kv_heads;
-        const uint32_t g = i - s.heads - (key ? 0 : s.kv_heads);
-        CT* row = static_cast<CT*>(a.cache) + ((size_t)g * a.plane_rows + p) * s.ld();
-        if (key) rotate_norm(y + s.off_k + (size_t)g * s.dim, row, s, cs, a.eps, lane);
-        else value_row(y + s.off_v + (size_t)g * s.vdim, row + s.dp, s, lane);
+    };
+    for (uint32_t i = warp; i < rows; i += 16) {
+        load(i + 8, row[1]);
+        store(i, row[0]);
+        load(i + 16, row[0]);
+        if (i + 8 < rows) store(i + 8, row[1]);
     }
+}
+template <class CT>
+cudaError_t prepare_type(const GroupedArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
+    const uint32_t n = std::max(a.s.dp, a.s.vp);
+    if (n <= 64) return launch_pdl(grouped_prepare_kernel<CT, 2>, dim3(tokens), dim3(256), 0, st, pdl, a);
+    if (n <= 128) return launch_pdl(grouped_prepare_kernel<CT, 4>, dim3(tokens), dim3(256), 0, st, pdl, a);
+    if (n <= 256) return launch_pdl(grouped_prepare_kernel<CT, 8>, dim3(tokens), dim3(256), 0, st, pdl, a);
+    return launch_pdl(grouped_prepare_kernel<CT, 16>, dim3(tokens), dim3(256), 0, st, pdl, a);
 }
 
 // f32 arithmetic. grid (blocks of rows, kv_heads), 8 warps of RW rows; a row is one (token, head of the group), a lane one of the
@@ -146,8 +165,7 @@ cudaError_t attn_type(const GroupedArgs& a, uint32_t tokens, cudaStream_t st, bo
 
 cudaError_t launch_grouped_prepare(const GroupedArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
     if (a.s.dp > GROUPED_MAX_DIM || a.s.vp > GROUPED_MAX_DIM) return cudaErrorInvalidValue;
-    return a.cache_bf16 ? launch_pdl(grouped_prepare_kernel<bf16>, dim3(tokens), dim3(256), 0, st, pdl, a)
-                        : launch_pdl(grouped_prepare_kernel<float>, dim3(tokens), dim3(256), 0, st, pdl, a);
+    return a.cache_bf16 ? prepare_type<bf16>(a, tokens, st, pdl) : prepare_type<float>(a, tokens, st, pdl);
 }
 cudaError_t launch_grouped_attn(const GroupedArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
     if (a.cache_bf16) return a.act_bf16 ? attn_type<bf16, bf16>(a, tokens, st, pdl) : attn_type<bf16, float>(a, tokens, st, pdl);

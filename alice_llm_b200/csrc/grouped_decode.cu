@@ -52,6 +52,14 @@ __global__ void __launch_bounds__(GD_WARPS * 32, 1) grouped_decode_kernel(const 
     }
     __syncwarp();
     pdl_wait();
+    // rows that need no position travel together with it
+    const float* y = a.y + (size_t)t * a.ldy;
+    HeadRow<8> query, key, value;
+    if (warp < rows) query.load(y + (size_t)(h0 + warp) * s.dim, s.dim, s.rot_dims, lane);
+    if (a.append && warp == W - 1) {
+        key.load(y + s.off_k + (size_t)kh * s.dim, s.dim, s.rot_dims, lane);
+        value.load(y + s.off_v + (size_t)kh * s.vdim, s.vdim, 0, lane);
+    }
     const uint32_t pos = (uint32_t)*a.pos + t, ctx = pos + 1, tiles = (ctx + GD_KEYS - 1) / GD_KEYS;
     const uint32_t per = ((tiles + gridDim.y - 1) / gridDim.y + W - 1) / W * W, shares = (tiles + per - 1) / per;
     const uint32_t lo = blockIdx.y * per, hi = min(tiles, lo + per);
@@ -75,25 +83,32 @@ __global__ void __launch_bounds__(GD_WARPS * 32, 1) grouped_decode_kernel(const 
     const uint32_t half = s.rot_dims / 2;
     rotation_table(cs, a.freq, half, pos, blockDim.x);
     __syncthreads();
-    const float* y = a.y + (size_t)t * a.ldy;
     if (fresh && warp == W - 1) {
-        bf16* row = static_cast<bf16*>(a.cache) + plane + (size_t)pos * ld;
-        rotate_norm(y + s.off_k + (size_t)kh * s.dim, row, s, cs, a.eps, lane);   // further head groups of these keys write the same bits
-        value_row(y + s.off_v + (size_t)kh * s.vdim, row + s.dp, s, lane);
+        bf16* out = static_cast<bf16*>(a.cache) + plane + (size_t)pos * ld;
+        key.store(out, s.dp, s.unit_qk, cs, a.eps, lane);   // further head groups of these keys write the same bits
+        value.store(out + s.dp, s.vp, false, cs, a.eps, lane);
         __threadfence();
         asm volatile("fence.proxy.async.global;" ::: "memory");   // the bulk copy below reads what this warp has written
     }
     for (uint32_t r = warp; r < GD_HEADS; r += W) {
-        if (r < rows) rotate_norm(y + (size_t)(h0 + r) * s.dim, qs + r * ldq, s, cs, a.eps, lane);
-        else for (uint32_t i = lane; i < s.dp; i += 32) put(qs + r * ldq + i, 0.0f);
+        if (r < rows) {
+            if (r >= W) query.load(y + (size_t)(h0 + r) * s.dim, s.dim, s.rot_dims, lane);
+            query.store(qs + r * ldq, s.dp, s.unit_qk, cs, a.eps, lane);
+        } else {
+            for (uint32_t i = lane; i < s.dp; i += 32) put(qs + r * ldq + i, 0.0f);
+        }
     }
     __syncthreads();
     for (; issued < min(stages, mine); issued++) issue(issued);
 
     constexpr float LOG2E = 1.4426950408889634f;
-    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f}, o[NT][4];
+    // scores in powers of two; bounded ones need no running maximum
+    const bool bounded = a.bounded;
+    const float scale = s.softcap > 0.0f ? s.scale / s.softcap * 2.0f * LOG2E : s.scale * LOG2E, cap = s.softcap * LOG2E;
+    float m[2], l[2] = {0.0f, 0.0f}, o[NT][4];
 #pragma unroll
     for (int i = 0; i < NT; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
+    m[0] = m[1] = bounded ? 0.0f : -INFINITY;
     const uint32_t q_addr = q_sm + ((lane % 16) * ldq + lane / 16 * 8) * 2;
     uint32_t done = 0;
     for (; done < mine; done++) {
@@ -115,27 +130,29 @@ __global__ void __launch_bounds__(GD_WARPS * 32, 1) grouped_decode_kernel(const 
         for (int n = 0; n < 2; n++) {
 #pragma unroll
             for (int e = 0; e < 4; e++) {
-                float v = (d[0][n][e] + d[1][n][e]) * s.scale;
-                if (s.softcap > 0.0f) v = s.softcap * tanhf(v / s.softcap);
-                sc[n][e] = k0 + n * 8 + (lane & 3) * 2 + (e & 1) < ctx ? v * LOG2E : -INFINITY;
+                float v = (d[0][n][e] + d[1][n][e]) * scale;
+                if (s.softcap > 0.0f) v = cap * tanh_of_pow2(v);
+                sc[n][e] = k0 + n * 8 + (lane & 3) * 2 + (e & 1) < ctx ? v : -INFINITY;
             }
             top0 = fmaxf(top0, fmaxf(sc[n][0], sc[n][1]));
             top1 = fmaxf(top1, fmaxf(sc[n][2], sc[n][3]));
         }
+        if (!bounded) {
 #pragma unroll
-        for (int x = 1; x <= 2; x *= 2) {
-            top0 = fmaxf(top0, __shfl_xor_sync(0xffffffffu, top0, x));
-            top1 = fmaxf(top1, __shfl_xor_sync(0xffffffffu, top1, x));
+            for (int x = 1; x <= 2; x *= 2) {
+                top0 = fmaxf(top0, __shfl_xor_sync(0xffffffffu, top0, x));
+                top1 = fmaxf(top1, __shfl_xor_sync(0xffffffffu, top1, x));
+            }
+            const float f0 = exp2f(m[0] - top0), f1 = exp2f(m[1] - top1);   // a tile holds at least one key: the tops are finite
+            m[0] = top0; m[1] = top1;
+            l[0] *= f0; l[1] *= f1;
+#pragma unroll
+            for (int i = 0; i < NT; i++) { o[i][0] *= f0; o[i][1] *= f0; o[i][2] *= f1; o[i][3] *= f1; }
         }
-        const float f0 = exp2f(m[0] - top0), f1 = exp2f(m[1] - top1);   // a tile holds at least one key: the tops are finite
-        m[0] = top0; m[1] = top1;
-        l[0] *= f0; l[1] *= f1;
-#pragma unroll
-        for (int i = 0; i < NT; i++) { o[i][0] *= f0; o[i][1] *= f0; o[i][2] *= f1; o[i][3] *= f1; }
         uint32_t hi4[4], lo4[4];
 #pragma unroll
         for (int e = 0; e < 4; e++) {
-            const float tp = e & 1 ? top1 : top0;
+            const float tp = m[e & 1];
             const float x = exp2f(sc[e / 2][(e & 1) * 2] - tp), z = exp2f(sc[e / 2][(e & 1) * 2 + 1] - tp);
             l[e & 1] += x + z;
             hi4[e] = pack_bf16(x, z);
@@ -226,7 +243,7 @@ __global__ void __launch_bounds__(GD_WARPS * 32, 1) grouped_decode_kernel(const 
         const float* p = part + (size_t)(h0 + r) * stride + 4 + c;
         const size_t step = (size_t)s.heads * stride;
         float v = 0.0f;
-#pragma unroll 8
+#pragma unroll 16
         for (uint32_t k = 0; k < shares; k++) v = fmaf(wt[r][k], __ldcg(p + k * step), v);
         put(out + (size_t)r * s.vdim + c, v);
     }

@@ -16,7 +16,6 @@ namespace {
 
 constexpr uint32_t GP_KEYS = 128, GP_ROWS = 128, GP_THREADS = 320, GP_STAGES = 2, GP_BOX = GP_ROWS * 128;
 constexpr uint32_t GP_O_COL = 256;          // tensor memory: scores of the two tiles at 0 and 128, sums at 256 and 384
-constexpr float GP_BOUND = 60.0f;           // exp of more would leave too little room in f32
 constexpr int KERR_ATTN_WAIT = 9;           // a wait inside the tensor-core attention
 constexpr int CAP_NONE = 0, CAP_EXP = -1;   // otherwise: terms of the odd series of tanh
 
@@ -278,7 +277,7 @@ cudaError_t prefill_inst(const GpArgs& a, uint32_t kv_heads, cudaStream_t st, bo
     return launch_pdl(grouped_prefill_kernel<CAP>, dim3(kv_heads, (a.tokens * a.group + 2 * GP_ROWS - 1) / (2 * GP_ROWS)), dim3(GP_THREADS), smem, st, pdl, a);
 }
 
-bool tc_fits(const GroupedShape& s) { return s.dp <= 128 && s.vp <= 128 && grouped_bound(s) <= GP_BOUND; }
+bool tc_fits(const GroupedArgs& a) { return a.s.dp <= 128 && a.s.vp <= 128 && a.bounded; }
 
 cudaError_t prefill_tc(const GroupedArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
     if (!encode_fn()) return cudaErrorNotSupported;
@@ -319,7 +318,7 @@ cudaError_t prefill_sync(const GroupedArgs& a, uint32_t tokens, cudaStream_t st,
 
 cudaError_t launch_grouped_prefill(const GroupedArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
     if (!grouped_tiled_fits(a.s) || !a.cache_bf16 || !a.act_bf16) return cudaErrorInvalidValue;
-    return tc_fits(a.s) ? prefill_tc(a, tokens, st, pdl) : prefill_sync(a, tokens, st, pdl);
+    return tc_fits(a) ? prefill_tc(a, tokens, st, pdl) : prefill_sync(a, tokens, st, pdl);
 }
 
 }  // namespace alice

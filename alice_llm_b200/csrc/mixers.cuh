@@ -8,7 +8,7 @@
 namespace alice {
 
 // ---- stack_ops.cu -------------------------------------------------------------------------------
-// x[t] <- (set ? 0 : x[t]) + (emb ? emb[tokens[t]] * scale : 0) + (step ? step : 0), columns [0, n); [n, ld) untouched.
+// x[t] <- (set ? 0 : x[t]) + (emb ? emb[tokens[t]] * scale : 0) + (step ? step : 0); columns [n, ld) are zero there and stay so.
 struct EnterArgs {
     const bf16* emb = nullptr;
     const int* tokens = nullptr;
@@ -17,6 +17,8 @@ struct EnterArgs {
     const float* step = nullptr;
     bool set = false;
     float* x = nullptr;
+    void* h = nullptr;                // a copy of the result, rows ld apart
+    bool h_bf16 = false;
 };
 cudaError_t launch_enter(const EnterArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 
@@ -151,6 +153,7 @@ struct GroupedArgs {
     void* out = nullptr;              // [t][ldo]
     uint32_t ldo = 0;
     bool act_bf16 = false;            // type of out
+    bool bounded = false;             // no score exceeds GROUPED_BOUND: exp needs no running maximum
     // grouped_decode.cu
     bool append = false;              // one token: its cache row is made here too
     uint32_t splits = 1;
@@ -164,6 +167,7 @@ cudaError_t launch_grouped_prepare(const GroupedArgs& a, uint32_t tokens, cudaSt
 cudaError_t launch_grouped_attn(const GroupedArgs& a, uint32_t tokens, cudaStream_t st, bool pdl);
 // On the tensor cores, bf16 cache: many tokens (prepared queries), few tokens (queries straight from the projections).
 inline bool grouped_tiled_fits(const GroupedShape& s) { return s.dp <= 256 && s.vp <= 256; }
+constexpr float GROUPED_BOUND = 60.0f;   // exp of more would leave too little room in f32
 // What no score exceeds: unit queries and keys meet in at most dim, and a cap is one.
 inline float grouped_bound(const GroupedShape& s) {
     const float unit = s.unit_qk ? 1.01f * std::fabs(s.scale) * s.dim : INFINITY;   // a little more for their rounding

@@ -234,7 +234,7 @@ struct GroupedMixer final : Mixer {
         GroupedArgs a;
         a.s = sh; a.y = s.y; a.ldy = s.ldy; a.sink = sink; a.freq = freq; a.eps = m->cfg.eps; a.pos = m->d_pos; a.cache = cache[pass]; a.plane_rows = plane_rows;
         a.cache_bf16 = !m->exact(); a.q = m->exact() ? (void*)s.q : (void*)s.q_rot; a.out = s.a; a.ldo = o.k; a.act_bf16 = m->tiled_bf16(n);
-        a.part = s.part; a.tickets = s.tickets; a.status = m->e->status;
+        a.bounded = grouped_bound(sh) <= GROUPED_BOUND; a.part = s.part; a.tickets = s.tickets; a.status = m->e->status;
         const bool few = n <= FEW_TOKENS && tiled(m);
         a.append = few && n == 1;
         if (!a.append) MCU(launch_grouped_prepare(a, n, st, pdl));
@@ -365,18 +365,10 @@ int StackModel::body(uint32_t n) {
     EnterArgs ea;
     ea.emb = embed.w; ea.tokens = d_token; ea.vocab = vocab; ea.emb_ld = embed.k; ea.n = cfg.width; ea.ld = s.wp; ea.scale = cfg.embed_scale;
     ea.set = true; ea.x = s.x;
+    if (cfg.block == ALICE_BLOCK_POST && n > 1) { ea.h = s.h; ea.h_bf16 = tiled_bf16(n); }   // layers read the stream itself: its copy as the products take it
     MCU(launch_enter(ea, n, st, e->pdl));
     pending = nullptr;
-    // with the norm behind the sum, layers read the stream itself: its copy as the products take it
-    auto copy = [&]() -> int {
-        if (cfg.block != ALICE_BLOCK_POST || n == 1) return ALICE_OK;
-        NormArgs na = norm_args(nullptr, tiled_bf16(n));
-        na.norm = NORM_NONE;
-        MCU(launch_norm(na, n, st, e->pdl));
-        return ALICE_OK;
-    };
-    int rc = copy();
-    if (rc) return rc;
+    int rc;
     trace_runs = 0; trace_tokens = n;
     auto one = [&](uint32_t i, uint32_t pass) -> int {
         int rc = layer(i, n, pass);
@@ -398,7 +390,6 @@ int StackModel::body(uint32_t n) {
         la.step = loop_step + (size_t)t * cfg.width;
         if ((rc = settle())) return rc;
         if (b > a) MCU(launch_enter(la, n, st, e->pdl));
-        if (b > a && (rc = copy())) return rc;
         for (uint32_t i = a; i < b; i++) if ((rc = one(i, t))) return rc;
     }
     for (uint32_t i = b; i < cfg.num_layers; i++) if ((rc = one(i, 0))) return rc;

@@ -7,7 +7,11 @@
 namespace alice {
 namespace {
 
-__global__ void __launch_bounds__(1024) enter_kernel(const __grid_constant__ EnterArgs a) {
+__device__ __forceinline__ void put4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void put4(bf16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w)); }
+
+template <class HT>
+__global__ void __launch_bounds__(256) enter_kernel(const __grid_constant__ EnterArgs a) {
     pdl_launch_dependents();
     pdl_wait();
     const uint32_t t = blockIdx.x;
@@ -15,11 +19,21 @@ __global__ void __launch_bounds__(1024) enter_kernel(const __grid_constant__ Ent
     if (tok >= a.vocab) tok = 0;
     const bf16* e = a.emb ? a.emb + (size_t)tok * a.emb_ld : nullptr;
     float* x = a.x + (size_t)t * a.ld;
-    for (uint32_t i = threadIdx.x; i < a.n; i += blockDim.x) {
-        float v = a.set ? 0.0f : x[i];
-        if (e) v += __fmul_rn(__bfloat162float(e[i]), a.scale);
-        if (a.step) v += a.step[i];
-        x[i] = v;
+    for (uint32_t c = threadIdx.x * 4; c < a.ld; c += 1024) {   // rows are padded with zeros to a multiple of 64
+        float4 v = a.set ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(x + c);
+        if (e) {
+            const uint2 u = __ldg(reinterpret_cast<const uint2*>(e + c));
+            const float2 p = bf2(u.x), q = bf2(u.y);
+            v.x += __fmul_rn(p.x, a.scale); v.y += __fmul_rn(p.y, a.scale); v.z += __fmul_rn(q.x, a.scale); v.w += __fmul_rn(q.y, a.scale);
+        }
+        if (a.step) {
+            if (c < a.n) v.x += a.step[c];
+            if (c + 1 < a.n) v.y += a.step[c + 1];
+            if (c + 2 < a.n) v.z += a.step[c + 2];
+            if (c + 3 < a.n) v.w += a.step[c + 3];
+        }
+        *reinterpret_cast<float4*>(x + c) = v;
+        if (a.h) put4(static_cast<HT*>(a.h) + (size_t)t * a.ld + c, v);
     }
 }
 
@@ -67,14 +81,9 @@ __global__ void __launch_bounds__(256) norm_kernel(const __grid_constant__ NormA
         if (a.norm != NORM_NONE)
 #pragma unroll
             for (int i = 0; i < 4; i++) v[j][i] = c + i < a.n ? (v[j][i] - mean) * inv * a.w[c + i] : 0.0f;
-        if (a.out) {
-            if constexpr (sizeof(OT) == 2) {
-                *reinterpret_cast<uint2*>(out + c) = make_uint2(pack_bf16(v[j][0], v[j][1]), pack_bf16(v[j][2], v[j][3]));
-            } else {
-                *reinterpret_cast<float4*>(out + c) = make_float4(v[j][0], v[j][1], v[j][2], v[j][3]);
-            }
-        }
-        if (a.x_out) *reinterpret_cast<float4*>(a.x_out + (size_t)t * a.ldx + c) = make_float4(v[j][0], v[j][1], v[j][2], v[j][3]);
+        const float4 u = make_float4(v[j][0], v[j][1], v[j][2], v[j][3]);
+        if (a.out) put4(out + c, u);
+        if (a.x_out) put4(a.x_out + (size_t)t * a.ldx + c, u);
     }
 }
 
@@ -89,7 +98,8 @@ cudaError_t norm_type(const NormArgs& a, uint32_t rows, cudaStream_t st, bool pd
 }  // namespace
 
 cudaError_t launch_enter(const EnterArgs& a, uint32_t tokens, cudaStream_t st, bool pdl) {
-    return launch_pdl(enter_kernel, dim3(tokens), dim3(a.n > 512 ? 1024 : 256), 0, st, pdl, a);
+    if (a.ld % 4 || a.ld < a.n || (a.emb && a.emb_ld < a.ld)) return cudaErrorInvalidValue;
+    return a.h_bf16 ? launch_pdl(enter_kernel<bf16>, dim3(tokens), dim3(256), 0, st, pdl, a) : launch_pdl(enter_kernel<float>, dim3(tokens), dim3(256), 0, st, pdl, a);
 }
 
 cudaError_t launch_norm(const NormArgs& a, uint32_t rows, cudaStream_t st, bool pdl) {
